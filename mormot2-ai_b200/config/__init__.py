@@ -5,6 +5,7 @@ from .busavik import BusavikConfig
 from .fimudra import FimudraConfig
 from .sezopel import SezopelConfig
 from .laralix import LaralixConfig
+from .lotirax import LotiraxConfig
 from .registry import (architectures, config_of_folder, family_of, read_config_json,
                        register_architecture)
 
@@ -13,7 +14,9 @@ register_architecture(BusavikConfig, BusavikConfig.ARCHITECTURE, BusavikConfig.M
 register_architecture(FimudraConfig, FimudraConfig.ARCHITECTURE, FimudraConfig.MODEL_TYPE)
 register_architecture(SezopelConfig, SezopelConfig.ARCHITECTURE, SezopelConfig.MODEL_TYPE)
 register_architecture(LaralixConfig, LaralixConfig.ARCHITECTURE, LaralixConfig.MODEL_TYPE)
+register_architecture(LotiraxConfig, LotiraxConfig.ARCHITECTURE, LotiraxConfig.MODEL_TYPE)
 
 __all__ = ["LayerSpec", "ModelSpec", "PartSpec", "Run", "Qwen3Config", "BusavikConfig", "FimudraConfig", "SezopelConfig", "LaralixConfig",
+           "LotiraxConfig",
            "architectures",
            "config_of_folder", "family_of", "read_config_json", "register_architecture"]

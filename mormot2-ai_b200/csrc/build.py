@@ -53,6 +53,7 @@ SOURCES = {
     "streams": "streams.cu",
     "recurrent": "recurrent.cu",
     "linear_state": "linear_state.cu",
+    "attention_diff": "attention_diff.cu",
 }
 HEADERS = ["common.cuh"]
 EXTRA_HEADERS = {"gemm_tc": ["tc_common.cuh"],

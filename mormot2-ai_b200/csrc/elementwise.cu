@@ -460,6 +460,209 @@ MB_EXPORT int mb_pass_input(float* x, const float* x0, const void* b, int b_dtyp
   MB_CHECK_LAUNCH("mb_pass_input");
 }
 
+// ------------------------------------------------------------------ scaled sums of sublayers
+// What several sublayers left for the residual (their products' split sums, the rows of a
+// token's experts, a stored output), each with a factor and a vector over the columns:
+//   v[t, c] = x[t, c] + sum over the terms of scale[c] * factor * (p0 + p1 + ...)[t, c]
+// in the order of the terms and of their parts. CONCAT false: x = v and, with y, the RMS norm
+// y[t] = w * v / sqrt(mean(v^2) + eps). CONCAT true: y[t] = [v ; x0[t]] (2 H values) and
+// x[t] = w (float32), what the product of y is then added onto.
+// A thread holds 4 * VEC columns (V4; 16-byte accesses) or walks them one by one.
+struct BranchTerm {
+  const float* p;
+  const float* scale;      // [H] or null
+  long long part_stride;
+  long long row_stride;
+  int parts;
+  float factor;
+};
+#define BRANCH_TERMS 4
+struct BranchTerms {
+  BranchTerm t[BRANCH_TERMS];
+  int n;
+};
+
+template <typename TO, int VEC, int THREADS, bool CONCAT>
+__global__ void __launch_bounds__(THREADS)
+branch_vec_kernel(float* __restrict__ x, const __grid_constant__ BranchTerms terms,
+                  const void* __restrict__ w, int w_bf16, float eps, TO* __restrict__ y,
+                  const float* __restrict__ x0, int H) {
+  __shared__ float red[33];
+  const int r = blockIdx.x;
+  float* xr = x + (size_t)r * H;
+  // Ahead of the wait for the kernel before: the norm's weights (or the pass's vector), and,
+  // where a product has left terms, the residual row, which that product did not write (kernels
+  // further back are complete once this one runs)
+  float wv[VEC][4];
+  float4 v[VEC];
+#pragma unroll
+  for (int i = 0; i < VEC; ++i) {
+    const int c = (i * THREADS + threadIdx.x) * 4;
+    v[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+    wv[i][0] = wv[i][1] = wv[i][2] = wv[i][3] = 0.f;
+    if (c >= H) continue;
+    if (terms.n > 0) v[i] = *(const float4*)(xr + c);
+    if (CONCAT || y != nullptr) {
+      const float4 raw = !CONCAT && w_bf16 ? load4<__nv_bfloat16>((const __nv_bfloat16*)w + c)
+                                           : *(const float4*)((const float*)w + c);
+      wv[i][0] = raw.x; wv[i][1] = raw.y; wv[i][2] = raw.z; wv[i][3] = raw.w;
+    }
+  }
+  mb_grid_wait();
+  mb_grid_launch_next();
+  float sum = 0.f;
+#pragma unroll
+  for (int i = 0; i < VEC; ++i) {
+    const int c = (i * THREADS + threadIdx.x) * 4;
+    if (c >= H) continue;
+    if (terms.n == 0) v[i] = *(const float4*)(xr + c);
+    for (int k = 0; k < terms.n; ++k) {
+      const BranchTerm& t = terms.t[k];
+      const float* pp = t.p + (size_t)r * t.row_stride + c;
+      float4 s = make_float4(1.f, 1.f, 1.f, 1.f), u = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (t.scale) s = __ldg((const float4*)(t.scale + c));
+      for (int p0 = 0; p0 < t.parts; p0 += 8) {       // up to eight loads in flight
+        float4 a[8];
+#pragma unroll
+        for (int j = 0; j < 8; ++j)
+          if (p0 + j < t.parts) a[j] = __ldg((const float4*)(pp + (size_t)(p0 + j) * t.part_stride));
+#pragma unroll
+        for (int j = 0; j < 8; ++j)
+          if (p0 + j < t.parts) { u.x += a[j].x; u.y += a[j].y; u.z += a[j].z; u.w += a[j].w; }
+      }
+      v[i].x = fmaf(s.x * t.factor, u.x, v[i].x);
+      v[i].y = fmaf(s.y * t.factor, u.y, v[i].y);
+      v[i].z = fmaf(s.z * t.factor, u.z, v[i].z);
+      v[i].w = fmaf(s.w * t.factor, u.w, v[i].w);
+    }
+    if (CONCAT) {
+      TO* yr = y + (size_t)r * 2 * H + c;
+      store4<TO>(yr, v[i]);
+      store4<TO>(yr + H, *(const float4*)(x0 + (size_t)r * H + c));
+      *(float4*)(xr + c) = make_float4(wv[i][0], wv[i][1], wv[i][2], wv[i][3]);
+    } else {
+      if (terms.n > 0) *(float4*)(xr + c) = v[i];
+      sum = fmaf(v[i].x, v[i].x, fmaf(v[i].y, v[i].y, fmaf(v[i].z, v[i].z, fmaf(v[i].w, v[i].w, sum))));
+    }
+  }
+  if (CONCAT || y == nullptr) return;
+  sum = block_sum(sum, red);
+  const float inv = 1.0f / sqrtf(sum / (float)H + eps);
+#pragma unroll
+  for (int i = 0; i < VEC; ++i) {
+    const int c = (i * THREADS + threadIdx.x) * 4;
+    if (c >= H) continue;
+    store4<TO>(y + (size_t)r * H + c,
+               make_float4(wv[i][0] * (v[i].x * inv), wv[i][1] * (v[i].y * inv),
+                           wv[i][2] * (v[i].z * inv), wv[i][3] * (v[i].w * inv)));
+  }
+}
+
+template <typename TO, bool CONCAT>
+__global__ void __launch_bounds__(256)
+branch_kernel(float* __restrict__ x, const __grid_constant__ BranchTerms terms,
+              const void* __restrict__ w, int w_bf16, float eps, TO* __restrict__ y,
+              const float* __restrict__ x0, int H) {
+  mb_grid_wait();
+  mb_grid_launch_next();
+  __shared__ float red[33];
+  const int r = blockIdx.x;
+  float* xr = x + (size_t)r * H;
+  float sum = 0.f;
+  for (int c = threadIdx.x; c < H; c += blockDim.x) {
+    float v = xr[c];
+    for (int k = 0; k < terms.n; ++k) {
+      const BranchTerm& t = terms.t[k];
+      const float u = sum_parts(t.p + (size_t)r * t.row_stride + c, t.parts, (size_t)t.part_stride);
+      v = fmaf((t.scale ? t.scale[c] : 1.0f) * t.factor, u, v);
+    }
+    if (CONCAT) {
+      y[(size_t)r * 2 * H + c] = from_f32<TO>(v);
+      y[(size_t)r * 2 * H + H + c] = from_f32<TO>(x0[(size_t)r * H + c]);
+      xr[c] = ((const float*)w)[c];
+    } else {
+      if (terms.n > 0) xr[c] = v;
+      sum = fmaf(v, v, sum);
+    }
+  }
+  if (CONCAT || y == nullptr) return;
+  sum = block_sum(sum, red);
+  const float inv = 1.0f / sqrtf(sum / (float)H + eps);
+  for (int c = threadIdx.x; c < H; c += blockDim.x) {   // a thread reads what it has written
+    const float wc = w_bf16 ? __bfloat162float(((const __nv_bfloat16*)w)[c]) : ((const float*)w)[c];
+    y[(size_t)r * H + c] = from_f32<TO>(wc * (xr[c] * inv));
+  }
+}
+
+template <typename TO, bool CONCAT>
+static int branch_launch(float* x, const BranchTerms& terms, const void* w, int w_bf16, float eps,
+                         void* y, const float* x0, int R, int H, cudaStream_t s) {
+  uintptr_t bits = (uintptr_t)x | (uintptr_t)w | (uintptr_t)y | (uintptr_t)x0;
+  long long strides = 0;
+  for (int k = 0; k < terms.n; ++k) {
+    bits |= (uintptr_t)terms.t[k].p | (uintptr_t)terms.t[k].scale;
+    strides |= terms.t[k].part_stride | terms.t[k].row_stride;
+  }
+  if (H % 4 == 0 && H <= 4 * 1024 * 4 && (bits & 15) == 0 && (strides & 3) == 0) {
+#define BR_GO(V_, T_)                                                                        \
+  mb_launch(branch_vec_kernel<TO, V_, T_, CONCAT>, dim3(R), dim3(T_), 0, s, x, terms, w,     \
+            w_bf16, eps, (TO*)y, x0, H)
+    if ((R <= 256 && H > 1024) || H > 4 * 256 * 4) {
+      const int vec = (H + 4 * 1024 - 1) / (4 * 1024);
+      if (vec <= 1) { BR_GO(1, 1024); }
+      else if (vec <= 2) { BR_GO(2, 1024); }
+      else { BR_GO(4, 1024); }
+    } else {
+      const int vec = (H + 4 * 256 - 1) / (4 * 256);
+      if (vec <= 1) { BR_GO(1, 256); }
+      else if (vec <= 2) { BR_GO(2, 256); }
+      else { BR_GO(4, 256); }
+    }
+#undef BR_GO
+    return 0;
+  }
+  mb_launch(branch_kernel<TO, CONCAT>, dim3(R), dim3(256), 0, s, x, terms, w, w_bf16, eps, (TO*)y,
+            x0, H);
+  return 0;
+}
+
+static bool branch_terms(const BranchTerm* list, int n, BranchTerms* out) {
+  if (n < 0 || n > BRANCH_TERMS) return false;
+  *out = BranchTerms{};
+  for (int k = 0; k < n; ++k) {
+    if (list[k].p == nullptr || list[k].parts < 1) return false;
+    out->t[k] = list[k];
+  }
+  out->n = n;
+  return true;
+}
+
+MB_EXPORT int mb_branch_norm(float* x, const BranchTerm* list, int n, const void* w, int w_dtype,
+                             float eps, void* y, int y_dtype, int R, int H, void* stream) {
+  if (R <= 0) return 0;
+  BranchTerms terms;
+  if (!branch_terms(list, n, &terms)) MB_FAIL("mb_branch_norm: %d terms", n);
+  if (y != nullptr && w == nullptr) MB_FAIL("mb_branch_norm: a norm without weights");
+  cudaStream_t s = (cudaStream_t)stream;
+  if (y_dtype == MB_F32)
+    branch_launch<float, false>(x, terms, w, w_dtype == MB_BF16, eps, y, nullptr, R, H, s);
+  else
+    branch_launch<__nv_bfloat16, false>(x, terms, w, w_dtype == MB_BF16, eps, y, nullptr, R, H, s);
+  MB_CHECK_LAUNCH("mb_branch_norm");
+}
+
+MB_EXPORT int mb_pass_concat(float* x, const BranchTerm* list, int n, const float* x0,
+                             const float* vector, void* y, int y_dtype, int R, int H,
+                             void* stream) {
+  if (R <= 0) return 0;
+  BranchTerms terms;
+  if (!branch_terms(list, n, &terms)) MB_FAIL("mb_pass_concat: %d terms", n);
+  cudaStream_t s = (cudaStream_t)stream;
+  if (y_dtype == MB_F32) branch_launch<float, true>(x, terms, vector, 0, 0.f, y, x0, R, H, s);
+  else branch_launch<__nv_bfloat16, true>(x, terms, vector, 0, 0.f, y, x0, R, H, s);
+  MB_CHECK_LAUNCH("mb_pass_concat");
+}
+
 // ------------------------------------------------------------------ q and k normed as whole rows
 // Rows [q (qw) | k (kw) | room (kw)] of ld values: q <- wq * q / rms(q) over all qw values at
 // once, k likewise with wk; with copy_k the k values as they came are first copied behind k

@@ -201,6 +201,8 @@ MB_EXPORT int mb_moe_route(const float* z, int ldz, int parts, long long part_st
 // plan (int32): [0] number of tiles, [1 .. 1+E] first list row of every expert (E + 1 values),
 // then perm[A] (the assignment a = t·top + k at every list row), then tile_expert[max_tiles]
 // and tile_row0[max_tiles]. One block.
+// With `table` given the choices come from it: token t's k-th expert is
+// table[tok_ids[t] * top + k] (A = T * top; an id outside the table counts as 0).
 // With z given (a step of at most 64 tokens) the block first routes the tokens itself, a warp a
 // token, and writes ids, w and sg as moe_route does: one kernel instead of two.
 __global__ void __launch_bounds__(1024)
@@ -208,7 +210,8 @@ moe_plan_kernel(int* __restrict__ ids, int A, int E, int bm, int max_tiles,
                 int* __restrict__ plan, const float* __restrict__ z, int ldz, int parts,
                 size_t part_stride, int top, int shared_col, float* __restrict__ w,
                 float* __restrict__ sg, int mode, const float* __restrict__ corr, float wscale,
-                int E_route) {
+                int E_route, const int* __restrict__ table, const int* __restrict__ tok_ids,
+                int V) {
   mb_grid_wait();
   mb_grid_launch_next();
   extern __shared__ int counts[];  // E counters, then E cursors
@@ -224,6 +227,11 @@ moe_plan_kernel(int* __restrict__ ids, int A, int E, int bm, int max_tiles,
     }
     __syncthreads();  // the block's own writes of ids are visible to it
   }
+  auto choice = [&](int a) {
+    if (table == nullptr) return ids[a];
+    const int t = a / top, id = tok_ids[t];
+    return table[(size_t)(id < 0 || id >= V ? 0 : id) * top + (a - t * top)];
+  };
   int* cursor = counts + E;
   int* offsets = plan + 1;
   int* perm = offsets + E + 1;
@@ -232,7 +240,7 @@ moe_plan_kernel(int* __restrict__ ids, int A, int E, int bm, int max_tiles,
   for (int e = threadIdx.x; e < E; e += blockDim.x) counts[e] = 0;
   __syncthreads();
   for (int a = threadIdx.x; a < A; a += blockDim.x) {
-    const int e = ids[a];
+    const int e = choice(a);
     if (e >= 0 && e < E) atomicAdd(&counts[e], 1);
   }
   __syncthreads();
@@ -253,7 +261,7 @@ moe_plan_kernel(int* __restrict__ ids, int A, int E, int bm, int max_tiles,
   }
   __syncthreads();
   for (int a = threadIdx.x; a < A; a += blockDim.x) {
-    const int e = ids[a];
+    const int e = choice(a);
     if (e >= 0 && e < E) perm[atomicAdd(&cursor[e], 1)] = a;
   }
 }
@@ -265,8 +273,23 @@ MB_EXPORT int mb_moe_plan(int* ids, int A, int E, int bm, int max_tiles, int* pl
   if (max_tiles < (A + bm - 1) / bm + E) MB_FAIL("mb_moe_plan: room for %d tiles", max_tiles);
   mb_launch(moe_plan_kernel, dim3(1), dim3(1024), (size_t)2 * E * sizeof(int),
             (cudaStream_t)stream, ids, A, E, bm, max_tiles, plan, (const float*)nullptr, 0, 1,
-            (size_t)0, 1, -1, (float*)nullptr, (float*)nullptr, 0, (const float*)nullptr, 1.0f, E);
+            (size_t)0, 1, -1, (float*)nullptr, (float*)nullptr, 0, (const float*)nullptr, 1.0f, E,
+            (const int*)nullptr, (const int*)nullptr, 0);
   MB_CHECK_LAUNCH("mb_moe_plan");
+}
+
+// The same for choices that a table [V, top] names by token id.
+MB_EXPORT int mb_moe_table_plan(const int* table, int V, int top, const int* tok_ids, int A, int E,
+                                int bm, int max_tiles, int* plan, void* stream) {
+  if (A <= 0) return 0;
+  if (E > 4096 || top <= 0 || top > E || A % top || V <= 0)
+    MB_FAIL("mb_moe_table_plan: %d choices of %d experts, %d ids", top, E, V);
+  if (max_tiles < (A + bm - 1) / bm + E) MB_FAIL("mb_moe_table_plan: room for %d tiles", max_tiles);
+  mb_launch(moe_plan_kernel, dim3(1), dim3(1024), (size_t)2 * E * sizeof(int),
+            (cudaStream_t)stream, (int*)nullptr, A, E, bm, max_tiles, plan, (const float*)nullptr, 0,
+            1, (size_t)0, top, -1, (float*)nullptr, (float*)nullptr, 0, (const float*)nullptr, 1.0f,
+            E, table, tok_ids, V);
+  MB_CHECK_LAUNCH("mb_moe_table_plan");
 }
 
 // moe_route and moe_plan in one kernel, for a step of at most 64 tokens.
@@ -286,7 +309,8 @@ MB_EXPORT int mb_moe_route_plan(const float* z, int ldz, int parts, long long pa
   if (max_tiles < (A + bm - 1) / bm + E) MB_FAIL("mb_moe_route_plan: room for %d tiles", max_tiles);
   mb_launch(moe_plan_kernel, dim3(1), dim3(1024), (size_t)2 * E * sizeof(int),
             (cudaStream_t)stream, ids, A, E, bm, max_tiles, plan, z, ldz, parts,
-            (size_t)part_stride, top, shared_col, w, sg, mode, corr, wscale, E_route);
+            (size_t)part_stride, top, shared_col, w, sg, mode, corr, wscale, E_route,
+            (const int*)nullptr, (const int*)nullptr, 0);
   MB_CHECK_LAUNCH("mb_moe_route_plan");
 }
 
@@ -304,20 +328,42 @@ __device__ __forceinline__ float moe_gated(float z, float u, int act, float limi
   return z / (1.0f + expf(-z)) * u;
 }
 
+// An activation of one input, for experts without a gate (the codes of the elementwise kernels).
+// 0: SiLU; 1: the tanh form of GELU; 3: the square of relu.
+__device__ __forceinline__ float moe_plain(float z, int act) {
+  if (act == 3) {
+    z = fmaxf(z, 0.f);
+    return z * z;
+  }
+  if (act == 1)
+    return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
+  return z / (1.0f + expf(-z));
+}
+
+// What a product of the experts is: the second one, the first with gate and up rows, or the first
+// of experts without a gate (W [E][N][K]).
+enum { MOE_DOWN = 0, MOE_GATED_UP = 1, MOE_PLAIN_UP = 2 };
+
+template <int MODE>
+__device__ __forceinline__ float moe_act(float z, float u, int act, float limit) {
+  return MODE == MOE_GATED_UP ? moe_gated(z, u, act, limit) : moe_plain(z, act);
+}
+
 #define MG_BN 64
 #define MG_BK 16
 // UP:   in = h [T, K] (row of list row r: perm[r] / top), W [E][2N][K] (gate rows, then up
-//       rows), out = act [A, N] at list row r.
+//       rows; without a gate [E][N][K]), out = act [A, N] at list row r.
 // DOWN: in = act [A, K] at list row r, W [E][N][K], out = y [A, N] float32 at row perm[r],
-//       multiplied by weight[perm[r]].
-template <typename T, typename TW, int BM, bool UP>
+//       multiplied by weight[perm[r]] (null: by one).
+template <typename T, typename TW, int BM, int MODE>
 __global__ void __launch_bounds__(256)
 moe_gemm_kernel(const T* __restrict__ in, const TW* __restrict__ W, void* __restrict__ out,
                 const int* __restrict__ plan, int A, int E, int max_tiles, int top, int N, int K,
                 int act, const float* __restrict__ weight, float limit) {
   mb_grid_wait();
   mb_grid_launch_next();
-  constexpr int NW = UP ? 2 : 1;
+  constexpr bool UP = MODE != MOE_DOWN;
+  constexpr int NW = MODE == MOE_GATED_UP ? 2 : 1;
   constexpr int TM = BM / 16;
   const int tile = blockIdx.y;
   if (tile >= plan[0]) return;
@@ -389,10 +435,10 @@ moe_gemm_kernel(const T* __restrict__ in, const TW* __restrict__ W, void* __rest
       if (gn >= N) continue;
       if (UP) {
         ((T*)out)[(size_t)(r0 + r) * N + gn] =
-            from_f32<T>(moe_gated(acc[0][i][j], acc[NW - 1][i][j], act, limit));
+            from_f32<T>(moe_act<MODE>(acc[0][i][j], acc[NW - 1][i][j], act, limit));
       } else {
         const int a = src[r];
-        ((float*)out)[(size_t)a * N + gn] = weight[a] * acc[0][i][j];
+        ((float*)out)[(size_t)a * N + gn] = (weight ? weight[a] : 1.0f) * acc[0][i][j];
       }
     }
   }
@@ -401,7 +447,7 @@ moe_gemm_kernel(const T* __restrict__ in, const TW* __restrict__ W, void* __rest
 // The same two products on the tensor cores for bfloat16 operands (mma_tile.cuh); the plan's
 // tiles have 128 rows. The first product multiplies the gathered rows with the gate and the up
 // rows of the expert at once.
-template <bool UP>
+template <int MODE>
 __global__ void __launch_bounds__(MT_THREADS)
 moe_gemm_mma_kernel(const __nv_bfloat16* __restrict__ in, const __nv_bfloat16* __restrict__ W,
                     void* __restrict__ out, const int* __restrict__ plan, int A, int E,
@@ -409,7 +455,8 @@ moe_gemm_mma_kernel(const __nv_bfloat16* __restrict__ in, const __nv_bfloat16* _
                     const float* __restrict__ weight, float limit) {
   mb_grid_wait();
   mb_grid_launch_next();
-  constexpr int NB = UP ? 2 : 1;
+  constexpr bool UP = MODE != MOE_DOWN;
+  constexpr int NB = MODE == MOE_GATED_UP ? 2 : 1;
   constexpr int MT_BN = 128 / NB;
   const int tile = blockIdx.y;
   if (tile >= plan[0]) return;
@@ -439,10 +486,10 @@ moe_gemm_mma_kernel(const __nv_bfloat16* __restrict__ in, const __nv_bfloat16* _
     if (r >= rows || gn >= N) return;
     if (UP) {
       ((__nv_bfloat16*)out)[(size_t)(r0 + r) * N + gn] =
-          __float2bfloat16_rn(moe_gated(acc[0][mi][ni][el], acc[NB - 1][mi][ni][el], act, limit));
+          __float2bfloat16_rn(moe_act<MODE>(acc[0][mi][ni][el], acc[NB - 1][mi][ni][el], act, limit));
     } else {
       const int a = src[r];
-      ((float*)out)[(size_t)a * N + gn] = weight[a] * acc[0][mi][ni][el];
+      ((float*)out)[(size_t)a * N + gn] = (weight ? weight[a] : 1.0f) * acc[0][mi][ni][el];
     }
   });
 }
@@ -456,7 +503,7 @@ moe_gemm_mma_kernel(const __nv_bfloat16* __restrict__ in, const __nv_bfloat16* _
 // holds values 8t .. 8t+7 of both operands: the products pair them up in another order than
 // the instruction's own, which is the same sum. K must be a multiple of 32.
 #define MR_WARPS 4
-template <bool UP>
+template <int MODE>
 __global__ void __launch_bounds__(MR_WARPS * 32)
 moe_rows_mma_kernel(const __nv_bfloat16* __restrict__ in, const __nv_bfloat16* __restrict__ W,
                     void* __restrict__ out, const int* __restrict__ plan, int A, int E,
@@ -464,7 +511,8 @@ moe_rows_mma_kernel(const __nv_bfloat16* __restrict__ in, const __nv_bfloat16* _
                     const float* __restrict__ weight, float limit) {
   mb_grid_wait();
   mb_grid_launch_next();
-  constexpr int NB = UP ? 2 : 1;
+  constexpr bool UP = MODE != MOE_DOWN;
+  constexpr int NB = MODE == MOE_GATED_UP ? 2 : 1;
   const int tile = blockIdx.y;
   if (tile >= plan[0]) return;
   const int* offsets = plan + 1;
@@ -501,7 +549,7 @@ moe_rows_mma_kernel(const __nv_bfloat16* __restrict__ in, const __nv_bfloat16* _
   float acc[NB][4];
 #pragma unroll
   for (int nb = 0; nb < NB; ++nb) acc[nb][0] = acc[nb][1] = acc[nb][2] = acc[nb][3] = 0.f;
-  constexpr int UNROLL = UP ? 4 : 8;
+  constexpr int UNROLL = NB == 2 ? 4 : 8;
   for (int k0 = 0; k0 < K; k0 += 32 * UNROLL) {
     uint4 a[UNROLL][NB], b[UNROLL][NB];
 #pragma unroll
@@ -535,10 +583,10 @@ moe_rows_mma_kernel(const __nv_bfloat16* __restrict__ in, const __nv_bfloat16* _
     if (gn >= N || r >= rows) continue;
     if (UP) {
       ((__nv_bfloat16*)out)[(size_t)(r0 + r) * N + gn] =
-          __float2bfloat16_rn(moe_gated(acc[0][el], acc[NB - 1][el], act, limit));
+          __float2bfloat16_rn(moe_act<MODE>(acc[0][el], acc[NB - 1][el], act, limit));
     } else {
       const int a_ = src[r];
-      ((float*)out)[(size_t)a_ * N + gn] = weight[a_] * acc[0][el];
+      ((float*)out)[(size_t)a_ * N + gn] = (weight ? weight[a_] : 1.0f) * acc[0][el];
     }
   }
 }
@@ -548,7 +596,9 @@ MB_EXPORT int mb_moe_gemm(const void* in, int dtype, const void* W, int w_dtype,
                           int K, int up, int act, const float* weight, float limit, void* stream) {
   if (A <= 0) return 0;
   if (bm != 8 && bm != 16 && bm != 64 && bm != 128) MB_FAIL("mb_moe_gemm: tiles of %d rows", bm);
-  if (!up && weight == nullptr) MB_FAIL("mb_moe_gemm: the second product needs the weights");
+  if (up < 0 || up > 2) MB_FAIL("mb_moe_gemm: product %d", up);
+  if (up == MOE_PLAIN_UP && act != 0 && act != 1 && act != 3)
+    MB_FAIL("mb_moe_gemm: activation %d of one input", act);
   cudaStream_t s = (cudaStream_t)stream;
   dim3 grid((N + MG_BN - 1) / MG_BN, max_tiles);
   if (bm == 8) {
@@ -558,19 +608,21 @@ MB_EXPORT int mb_moe_gemm(const void* in, int dtype, const void* W, int w_dtype,
     const size_t smem = (size_t)8 * (K + 8) * 2;
     if (smem > 160 * 1024) MB_FAIL("mb_moe_gemm: rows of %d values", K);
     dim3 g8((N + 16 * MR_WARPS - 1) / (16 * MR_WARPS), max_tiles);
-#define GO8(UP_)                                                                              \
+#define GO8(M_)                                                                               \
   {                                                                                           \
     static bool configured = false;                                                           \
     if (!configured) {                                                                        \
-      cudaFuncSetAttribute(moe_rows_mma_kernel<UP_>, cudaFuncAttributeMaxDynamicSharedMemorySize, \
+      cudaFuncSetAttribute(moe_rows_mma_kernel<M_>, cudaFuncAttributeMaxDynamicSharedMemorySize, \
                            160 * 1024);                                                       \
       configured = true;                                                                      \
     }                                                                                         \
-    mb_launch(moe_rows_mma_kernel<UP_>, g8, dim3(MR_WARPS * 32), smem, s,                     \
+    mb_launch(moe_rows_mma_kernel<M_>, g8, dim3(MR_WARPS * 32), smem, s,                     \
               (const __nv_bfloat16*)in, (const __nv_bfloat16*)W, out, plan, A, E, max_tiles,  \
               top, N, K, act, weight, limit);                                                 \
   }
-    if (up) GO8(true) else GO8(false)
+    if (up == MOE_GATED_UP) GO8(MOE_GATED_UP)
+    else if (up == MOE_PLAIN_UP) GO8(MOE_PLAIN_UP)
+    else GO8(MOE_DOWN)
 #undef GO8
     MB_CHECK_LAUNCH("mb_moe_gemm");
   }
@@ -578,23 +630,32 @@ MB_EXPORT int mb_moe_gemm(const void* in, int dtype, const void* W, int w_dtype,
     if (!(dtype == MB_BF16 && w_dtype == MB_BF16 && K % 8 == 0 &&
           (((uintptr_t)in | (uintptr_t)W) & 15) == 0))
       MB_FAIL("mb_moe_gemm: tiles of 128 rows are the tensor-core kernel's (bfloat16, K %% 8 == 0)");
-    if (up)
-      mb_launch(moe_gemm_mma_kernel<true>, dim3((N + 63) / 64, max_tiles), dim3(MT_THREADS), 0, s,
-                (const __nv_bfloat16*)in, (const __nv_bfloat16*)W, out, plan, A, E, max_tiles, top,
-                N, K, act, weight, limit);
+    if (up == MOE_GATED_UP)
+      mb_launch(moe_gemm_mma_kernel<MOE_GATED_UP>, dim3((N + 63) / 64, max_tiles),
+                dim3(MT_THREADS), 0, s, (const __nv_bfloat16*)in, (const __nv_bfloat16*)W, out,
+                plan, A, E, max_tiles, top, N, K, act, weight, limit);
+    else if (up == MOE_PLAIN_UP)
+      mb_launch(moe_gemm_mma_kernel<MOE_PLAIN_UP>, dim3((N + 127) / 128, max_tiles),
+                dim3(MT_THREADS), 0, s, (const __nv_bfloat16*)in, (const __nv_bfloat16*)W, out,
+                plan, A, E, max_tiles, top, N, K, act, weight, limit);
     else
-      mb_launch(moe_gemm_mma_kernel<false>, dim3((N + 127) / 128, max_tiles), dim3(MT_THREADS), 0,
+      mb_launch(moe_gemm_mma_kernel<MOE_DOWN>, dim3((N + 127) / 128, max_tiles), dim3(MT_THREADS), 0,
                 s, (const __nv_bfloat16*)in, (const __nv_bfloat16*)W, out, plan, A, E, max_tiles,
                 top, N, K, act, weight, limit);
     MB_CHECK_LAUNCH("mb_moe_gemm");
   }
-#define GO(T_, TW_, BM_, UP_)                                                                \
-  mb_launch(moe_gemm_kernel<T_, TW_, BM_, UP_>, grid, dim3(256), 0, s, (const T_*)in,        \
+#define GO(T_, TW_, BM_, M_)                                                                 \
+  mb_launch(moe_gemm_kernel<T_, TW_, BM_, M_>,  grid, dim3(256), 0, s, (const T_*)in,        \
             (const TW_*)W, out, plan, A, E, max_tiles, top, N, K, act, weight, limit)
+#define GO2(T_, TW_, BM_)                                             \
+  {                                                                   \
+    if (up == MOE_GATED_UP) GO(T_, TW_, BM_, MOE_GATED_UP);           \
+    else if (up == MOE_PLAIN_UP) GO(T_, TW_, BM_, MOE_PLAIN_UP);      \
+    else GO(T_, TW_, BM_, MOE_DOWN);                                  \
+  }
 #define GO3(T_, TW_)                                                  \
   {                                                                   \
-    if (bm == 16) { if (up) GO(T_, TW_, 16, true); else GO(T_, TW_, 16, false); } \
-    else { if (up) GO(T_, TW_, 64, true); else GO(T_, TW_, 64, false); }          \
+    if (bm == 16) GO2(T_, TW_, 16) else GO2(T_, TW_, 64)              \
   }
   if (dtype == MB_F32) {
     if (w_dtype == MB_F32) GO3(float, float) else GO3(float, __nv_bfloat16)
@@ -602,6 +663,7 @@ MB_EXPORT int mb_moe_gemm(const void* in, int dtype, const void* W, int w_dtype,
     if (w_dtype == MB_F32) GO3(__nv_bfloat16, float) else GO3(__nv_bfloat16, __nv_bfloat16)
   }
 #undef GO3
+#undef GO2
 #undef GO
   MB_CHECK_LAUNCH("mb_moe_gemm");
 }

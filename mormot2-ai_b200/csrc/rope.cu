@@ -469,3 +469,178 @@ MB_EXPORT int mb_qk_norm_rope_store(void* qkv, const float* partial, int parts,
   MB_CHECK_LAUNCH("mb_qk_norm_rope_store");
 }
 
+
+// ------------------------------------------------------------------ heads of several maps
+// Rows [q | k | v] of a product (or its float32 split sums [parts][T][ld], added up in split
+// order) for attention whose heads have `maps` queries and keys each: q holds nh * maps vectors
+// of `dim`, k nkv * maps, v nkv of `vd`. A warp takes one vector at a time: the bias is added
+// (float32, may be null), a map of q or k is normed (x / sqrt(mean(x^2) + eps) * w, one weight
+// for all) and its first rot_dim values turn, pair (i, i + rot_dim / 2), cosine and sine times
+// `amp`. q goes to q_out [T][nh * maps * dim]; the maps of a key head lie one after the other
+// in the head's cache row of maps * dim values. A lane holds two neighbouring values of every
+// 64 (PAIRS; the sizes and row pitches are then even) or one of every 32. A block takes
+// `per_block` vectors of one token and forms the token's sines and cosines once.
+#define MP_WARPS 4
+#define MP_MAX 8    // rounds of a lane over a vector: 512 values in pairs, 256 single ones
+
+template <typename T> __device__ __forceinline__ float2 load2(const T* p);
+template <> __device__ __forceinline__ float2 load2<float>(const float* p) { return *(const float2*)p; }
+template <> __device__ __forceinline__ float2 load2<__nv_bfloat16>(const __nv_bfloat16* p) {
+  return __bfloat1622float2(*(const __nv_bfloat162*)p);
+}
+__device__ __forceinline__ void store2(float* p, float2 v) { *(float2*)p = v; }
+__device__ __forceinline__ void store2(__nv_bfloat16* p, float2 v) {
+  *(__nv_bfloat162*)p = __floats2bfloat162_rn(v.x, v.y);
+}
+
+template <typename TI, typename TO, bool PAIRS>
+__global__ void __launch_bounds__(MP_WARPS * 32)
+maps_norm_rope_store_kernel(const TI* __restrict__ rows, int parts, size_t part_stride, int ld,
+                            const float* __restrict__ bias, const float* __restrict__ q_norm,
+                            const float* __restrict__ k_norm, float eps,
+                            const float* __restrict__ inv_freq, int rot_dim, float amp,
+                            const int* __restrict__ tok_slot, const int* __restrict__ tok_pos,
+                            const int* __restrict__ page_table, int max_pages, int ring_pages,
+                            TO* __restrict__ kpool, TO* __restrict__ vpool, TO* __restrict__ q_out,
+                            int nh, int nkv, int maps, int dim, int vd, int per_block) {
+  constexpr int PER = PAIRS ? 2 : 1, STEP = 32 * PER;
+  extern __shared__ float mp_smem[];   // [rot_dim / 2] cosines, then sines, then [warps][dim]
+  const int half = rot_dim >> 1;
+  float* cs = mp_smem;
+  float* sn = cs + half;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  float* buf = sn + half + warp * dim;
+  const int t = blockIdx.x;
+  // before the wait: what does not depend on the kernel before
+  const int pos = tok_pos[t], slot = tok_slot[t];
+  for (int i = threadIdx.x; i < half; i += MP_WARPS * 32) {
+    float s, c;
+    sincosf(inv_freq[i] * (float)pos, &s, &c);
+    cs[i] = c * amp;
+    sn[i] = s * amp;
+  }
+  __syncthreads();
+  mb_grid_wait();
+  mb_grid_launch_next();
+  const int nq = nh * maps, nk = nkv * maps, total = nq + nk + nkv;
+  const int first = blockIdx.y * per_block, last = min(first + per_block, total);
+  for (int n = first + warp; n < last; n += MP_WARPS) {
+    const bool is_q = n < nq, is_k = !is_q && n < nq + nk;
+    const int size = is_q || is_k ? dim : vd;
+    const int col = is_q || is_k ? n * dim : (nq + nk) * dim + (n - nq - nk) * vd;
+    const TI* src = rows + (size_t)t * ld + col;
+    float2 v[MP_MAX];
+    float sum = 0.f;
+#pragma unroll
+    for (int j = 0; j < MP_MAX; ++j) {
+      v[j] = make_float2(0.f, 0.f);
+      const int i = STEP * j + PER * lane;
+      if (i >= size) continue;
+      for (int p0 = 0; p0 < parts; p0 += 8) {
+        float2 a[8];
+#pragma unroll
+        for (int p = 0; p < 8; ++p) {
+          if (p0 + p >= parts) continue;
+          const TI* at = src + (size_t)(p0 + p) * part_stride + i;
+          a[p] = PAIRS ? load2<TI>(at) : make_float2(to_f32<TI>(*at), 0.f);
+        }
+#pragma unroll
+        for (int p = 0; p < 8; ++p)
+          if (p0 + p < parts) { v[j].x += a[p].x; v[j].y += a[p].y; }
+      }
+      if (bias) {
+        v[j].x += bias[col + i];
+        if (PAIRS) v[j].y += bias[col + i + 1];
+      }
+      sum = fmaf(v[j].x, v[j].x, fmaf(v[j].y, v[j].y, sum));
+    }
+    TO* dst;
+    if (is_q) {
+      dst = q_out + (size_t)t * nq * dim + col;
+    } else {
+      const int m = n - nq, g = is_k ? m / maps : m - nk;
+      const size_t row = kv_row(page_table, max_pages, ring_pages, slot, pos, nkv, g);
+      dst = is_k ? kpool + (row * maps + (m - g * maps)) * dim : vpool + row * vd;
+    }
+    if (is_q || is_k) {
+      const float* w = is_q ? q_norm : k_norm;
+      const float inv = 1.0f / sqrtf(warp_sum(sum) / (float)dim + eps);
+#pragma unroll
+      for (int j = 0; j < MP_MAX; ++j) {
+        const int i = STEP * j + PER * lane;
+        if (i >= size) continue;
+        v[j].x = w[i] * (v[j].x * inv);
+        buf[i] = v[j].x;
+        if (PAIRS) {
+          v[j].y = w[i + 1] * (v[j].y * inv);
+          buf[i + 1] = v[j].y;
+        }
+      }
+      __syncwarp();
+      auto turn = [&](int i, float x) {
+        if (i >= rot_dim) return x;
+        return i < half ? x * cs[i] - buf[i + half] * sn[i]
+                        : x * cs[i - half] + buf[i - half] * sn[i - half];
+      };
+#pragma unroll
+      for (int j = 0; j < MP_MAX; ++j) {
+        const int i = STEP * j + PER * lane;
+        if (i >= size) continue;
+        v[j].x = turn(i, v[j].x);
+        if (PAIRS) v[j].y = turn(i + 1, v[j].y);
+      }
+      __syncwarp();      // buf is written again by the warp's next vector
+    }
+#pragma unroll
+    for (int j = 0; j < MP_MAX; ++j) {
+      const int i = STEP * j + PER * lane;
+      if (i >= size) continue;
+      if (PAIRS) store2(dst + i, v[j]);
+      else dst[i] = from_f32<TO>(v[j].x);
+    }
+  }
+}
+
+MB_EXPORT int mb_maps_norm_rope_store(const void* rows, int in_dtype, int parts,
+                                      long long part_stride, int ld, const float* bias,
+                                      const float* q_norm, const float* k_norm, float eps,
+                                      const float* inv_freq, int rot_dim, float amp,
+                                      const int* tok_slot, const int* tok_pos,
+                                      const int* page_table, int max_pages, int ring_pages,
+                                      void* kpool, void* vpool, void* q_out, int dtype, int T,
+                                      int nh, int nkv, int maps, int dim, int vd, void* stream) {
+  if (T <= 0) return 0;
+  if (rot_dim < 0 || rot_dim > dim || (rot_dim & 1))
+    MB_FAIL("mb_maps_norm_rope_store: %d of %d values rotate", rot_dim, dim);
+  if (nh <= 0 || nkv <= 0 || maps <= 0 || nh % nkv || parts < 1)
+    MB_FAIL("mb_maps_norm_rope_store: %d heads on %d KV heads, %d maps, %d parts", nh, nkv, maps, parts);
+  if (ld < (nh + nkv) * maps * dim + nkv * vd)
+    MB_FAIL("mb_maps_norm_rope_store: a row pitch of %d", ld);
+  if (in_dtype == MB_BF16 && dtype != MB_BF16)
+    MB_FAIL("mb_maps_norm_rope_store: bfloat16 rows for float32 activations");
+  const uintptr_t in_bytes = in_dtype == MB_F32 ? 8 : 4, out_bytes = dtype == MB_F32 ? 8 : 4;
+  const bool pairs = !(dim & 1) && !(vd & 1) && !(ld & 1) && !(part_stride & 1) &&
+                     ((uintptr_t)rows % in_bytes) == 0 &&
+                     (((uintptr_t)kpool | (uintptr_t)vpool | (uintptr_t)q_out) % out_bytes) == 0;
+  const int most = (pairs ? 64 : 32) * MP_MAX;
+  if (dim <= 0 || vd <= 0 || dim > most || vd > most)
+    MB_FAIL("mb_maps_norm_rope_store: vectors of %d and %d values (at most %d)", dim, vd, most);
+  const size_t smem = (size_t)(rot_dim + MP_WARPS * dim) * sizeof(float);
+  const int total = (nh + nkv) * maps + nkv;
+  // few tokens: a vector a warp; many: four a warp, so that a block's angles serve sixteen
+  const int per_block = T < 256 ? MP_WARPS : 4 * MP_WARPS;
+  dim3 grid(T, (total + per_block - 1) / per_block);
+  cudaStream_t s = (cudaStream_t)stream;
+#define GO(TI_, TO_, P_)                                                                        \
+  mb_launch(maps_norm_rope_store_kernel<TI_, TO_, P_>, grid, dim3(MP_WARPS * 32), smem, s,      \
+            (const TI_*)rows, parts, (size_t)part_stride, ld, bias, q_norm, k_norm, eps,        \
+            inv_freq, rot_dim, amp, tok_slot, tok_pos, page_table, max_pages, ring_pages,       \
+            (TO_*)kpool, (TO_*)vpool, (TO_*)q_out, nh, nkv, maps, dim, vd, per_block)
+#define GO_P(TI_, TO_) { if (pairs) GO(TI_, TO_, true); else GO(TI_, TO_, false); }
+  if (dtype == MB_F32) GO_P(float, float)
+  else if (in_dtype == MB_F32) GO_P(float, __nv_bfloat16)
+  else GO_P(__nv_bfloat16, __nv_bfloat16)
+#undef GO_P
+#undef GO
+  MB_CHECK_LAUNCH("mb_maps_norm_rope_store");
+}

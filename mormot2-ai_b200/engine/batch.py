@@ -7,7 +7,7 @@ device buffer that is filled by one copy from pinned host memory.
 """
 from __future__ import annotations
 
-from dataclasses import dataclass
+from dataclasses import dataclass, field
 from typing import List, Sequence, Tuple
 
 import numpy as np
@@ -42,6 +42,8 @@ class StepContext:
     host_new: List[int]
     host_past: List[int]
     host_slots: List[int]
+    # what a part keeps for a later run in the same pass of the model (emptied at its start)
+    memo: dict = field(default_factory=dict)
 
     @property
     def long(self) -> bool:

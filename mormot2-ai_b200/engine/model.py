@@ -125,6 +125,7 @@ class DecoderModel:
         if self.spec.streams:
             shape = (self.spec.streams,) + shape
         x = torch.empty(shape, dtype=torch.float32, device=self.rt.device)
+        step.memo = {}      # what a part keeps for a later run of this pass of the model
         self.embedding.forward(step.tok_ids, x)
         x0 = None
         if self.keeps_embedding:     # a later pass adds the embedding's output once more
@@ -139,10 +140,14 @@ class DecoderModel:
             state = cache.states.get(run.cache_line) if run.cache_line is not None else None
             block = self.layers[run.layer].block
             if i in self.entries:
-                if pending is not None:
-                    settle(x, pending)
-                    pending = None
-                self.entries[i].forward(x, x0)
+                entry = self.entries[i]
+                if getattr(entry, "accepts_pending", False):
+                    pending = entry.forward(x, x0, pending=pending)
+                else:
+                    if pending is not None:
+                        settle(x, pending)
+                        pending = None
+                    entry.forward(x, x0)
             if getattr(block, "accepts_pending", False):
                 pending = block.forward(x, step, line, state, run.writes_cache, pending=pending)
             else:

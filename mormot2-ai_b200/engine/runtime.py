@@ -158,6 +158,12 @@ class Runtime:
             return
         K.latent_attention(q, out, step, line, nh, kv_rank, rot_dim, window, scale)
 
+    def differential_attention(self, q, out, step, line, nh, nkv, dim, vd, window, scale, lam,
+                               factor, eps) -> None:
+        """Differential attention: the tensor-core kernels for bfloat16 and the sizes they take,
+        else the float32 kernel."""
+        K.attention_diff(q, out, step, line, nh, nkv, dim, vd, window, scale, lam, factor, eps)
+
     def attention(self, q, q_stride, out, step, line, nh, nkv, hd, window, scale, vd=0,
                   sink=None, softcap=0.0, gate=None, gate_stride=0, slopes=None,
                   keep_first=0) -> None:

@@ -73,7 +73,11 @@ CLASS_OF = {"mb_gemm_tc": "products", "mb_gemm_simt": "products",
             "mb_heads_gemm": "products", "mb_latent_attention": "attention",
             "mb_latent_attention_mma": "attention",
             "mb_moe_route": "routing", "mb_moe_plan": "routing", "mb_moe_route_plan": "routing", "mb_moe_gemm": "products",
-            "mb_moe_combine": "routing", "mb_stream_step": "norms", "mb_add_scaled": "norms",
+            "mb_moe_combine": "routing", "mb_moe_table_plan": "routing",
+            "mb_branch_norm": "norms", "mb_pass_concat": "norms",
+            "mb_maps_norm_rope_store": "rotary", "mb_attention_diff": "attention",
+            "mb_attention_diff_decode": "attention", "mb_attention_diff_prefill": "attention",
+            "mb_attention_diff_prefill_tc": "attention", "mb_stream_step": "norms", "mb_add_scaled": "norms",
             "mb_token_shift": "recurrence", "mb_wkv_scan": "recurrence",
             "mb_mlstm_scan": "recurrence", "mb_tanh": "recurrence",
             "mb_retention_scan": "recurrence", "mb_retention_chunked": "recurrence",
@@ -394,6 +398,61 @@ def pass_input(x: torch.Tensor, b: torch.Tensor, x0: Optional[torch.Tensor] = No
         assert x0.dtype == torch.float32 and x0.shape == x.shape and x0.is_contiguous()
     _call("elementwise", "mb_pass_input", [_vp, _vp, _vp, _i, _i, _i, _vp],
           _ptr(x), _ptr(x0), _ptr(b), code_of(b.dtype), x.shape[0], x.shape[1], _stream())
+
+
+class BranchTerm(_c.Structure):
+    """One term of the kernels below (BranchTerm in csrc/elementwise.cu)."""
+    _fields_ = [("p", _vp), ("scale", _vp), ("part_stride", _ll), ("row_stride", _ll),
+                ("parts", _i), ("factor", _f)]
+
+
+MAX_BRANCH_TERMS = 4
+
+
+def _branch_terms(terms, T: int, H: int):
+    if len(terms) > MAX_BRANCH_TERMS:
+        raise KernelError(f"{len(terms)} terms of a sum into the residual (at most "
+                          f"{MAX_BRANCH_TERMS})")
+    out = (BranchTerm * MAX_BRANCH_TERMS)()
+    for i, (y, factor, scale) in enumerate(terms):
+        assert y.dtype == torch.float32 and y.shape[-2:] == (T, H) and y.stride(-1) == 1
+        assert scale is None or (scale.dtype == torch.float32 and scale.numel() == H
+                                 and scale.is_contiguous())
+        parts, part_stride = (1, 0) if y.dim() == 2 else (y.shape[0], y.stride(0))
+        out[i] = BranchTerm(_ptr(y), _ptr(scale), part_stride, y.stride(-2), parts, float(factor))
+    return out, len(terms)
+
+
+def branch_norm(x: torch.Tensor, terms, w: Optional[torch.Tensor] = None, eps: float = 0.0,
+                out: Optional[torch.Tensor] = None) -> None:
+    """x[t, c] += sum over the terms (y, factor, scale) of scale[c] * factor * (the sum of y's
+    parts), in the order of the terms and of their parts; y float32 [T, H] or [parts, T, H]
+    with any strides between parts and rows, scale float32 [H] or None. With ``out``:
+    out[t] = w * x[t] / rms(x[t])."""
+    T, H = x.shape
+    assert x.dtype == torch.float32
+    _contig(x, "x")
+    arr, n = _branch_terms(terms, T, H)
+    if out is not None:
+        assert out.shape == (T, H) and out.is_contiguous() and w.numel() == H
+    _call("elementwise", "mb_branch_norm", [_vp, _vp, _i, _vp, _i, _f, _vp, _i, _i, _i, _vp],
+          _ptr(x), _c.cast(arr, _vp), n, _ptr(w), code_of(w.dtype) if w is not None else F32,
+          float(eps), _ptr(out), code_of(out.dtype) if out is not None else F32, T, H, _stream())
+
+
+def pass_concat(x: torch.Tensor, terms, x0: torch.Tensor, vector: torch.Tensor,
+                both: torch.Tensor) -> None:
+    """both[t] = [x[t] + the terms (as in ``branch_norm``) ; x0[t]] in both's type, and then
+    x[t] = vector."""
+    T, H = x.shape
+    assert x.dtype == x0.dtype == vector.dtype == torch.float32 and x0.shape == x.shape
+    assert both.shape == (T, 2 * H) and vector.numel() == H
+    for t, what in ((x, "x"), (x0, "x0"), (vector, "the pass's vector"), (both, "the rows")):
+        _contig(t, what)
+    arr, n = _branch_terms(terms, T, H)
+    _call("elementwise", "mb_pass_concat", [_vp, _vp, _i, _vp, _vp, _vp, _i, _i, _i, _vp],
+          _ptr(x), _c.cast(arr, _vp), n, _ptr(x0), _ptr(vector), _ptr(both),
+          code_of(both.dtype), T, H, _stream())
 
 
 def wide_qk_norm(qkv: torch.Tensor, qw: int, kw: int, wq: torch.Tensor, wk: torch.Tensor,
@@ -801,6 +860,19 @@ def moe_plan(ids: torch.Tensor, experts: int, bm: int, max_tiles: int,
           _ptr(ids), ids.numel(), experts, bm, max_tiles, _ptr(plan), _stream())
 
 
+def moe_table_plan(table: torch.Tensor, tok_ids: torch.Tensor, experts: int, bm: int,
+                   max_tiles: int, plan: torch.Tensor) -> None:
+    """``moe_plan`` for choices that a table names: token t's k-th expert is
+    table[tok_ids[t], k]."""
+    V, top = table.shape
+    A = tok_ids.numel() * top
+    assert table.dtype == torch.int32 and tok_ids.dtype == torch.int32
+    _contig(table, "the experts' table")
+    assert plan.dtype == torch.int32 and plan.numel() >= 2 + experts + A + 2 * max_tiles
+    _call("moe", "mb_moe_table_plan", [_vp, _i, _i, _vp, _i, _i, _i, _i, _vp, _vp],
+          _ptr(table), V, top, _ptr(tok_ids), A, experts, bm, max_tiles, _ptr(plan), _stream())
+
+
 def moe_route_plan(z: torch.Tensor, experts: int, top: int, shared_col: int, ids: torch.Tensor,
                    w: torch.Tensor, sg: Optional[torch.Tensor], bm: int, max_tiles: int,
                    plan: torch.Tensor, mode: int = 0, correction: Optional[torch.Tensor] = None,
@@ -820,12 +892,14 @@ def moe_route_plan(z: torch.Tensor, experts: int, top: int, shared_col: int, ids
 
 def moe_gemm(src: torch.Tensor, w: torch.Tensor, out: torch.Tensor, plan: torch.Tensor,
              assignments: int, max_tiles: int, bm: int, top: int, up: bool, act: int = ACT_SILU,
-             weight: Optional[torch.Tensor] = None, limit: float = 0.0) -> None:
+             weight: Optional[torch.Tensor] = None, limit: float = 0.0,
+             gated: bool = True) -> None:
     """One of the experts' two products over the planned tiles. ``up``: w [E, 2N, K] (gate
-    rows, then up rows), rows of ``src`` [T, K] gathered, out [A, N]. Else w [E, N, K], src
-    [A, K], out [A, N] float32 at the assignment's own row, times ``weight`` [A]."""
+    rows, then up rows; without ``gated`` [E, N, K] and an activation of one input), rows of
+    ``src`` [T, K] gathered, out [A, N]. Else w [E, N, K], src [A, K], out [A, N] float32 at the
+    assignment's own row, times ``weight`` [A] (None: times one)."""
     E = w.shape[0]
-    N = w.shape[1] // (2 if up else 1)
+    N = w.shape[1] // (2 if up and gated else 1)
     Kd = w.shape[2]
     _contig(src, "src"), _contig(out, "out"), _contig(w, "the experts' weight")
     assert src.shape[1] == Kd and out.shape[1] == N
@@ -833,7 +907,8 @@ def moe_gemm(src: torch.Tensor, w: torch.Tensor, out: torch.Tensor, plan: torch.
     _call("moe", "mb_moe_gemm",
           [_vp, _i, _vp, _i, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _i, _i, _vp, _f, _vp],
           _ptr(src), code_of(src.dtype), _ptr(w), code_of(w.dtype), _ptr(out), _ptr(plan),
-          assignments, E, max_tiles, bm, top, N, Kd, 1 if up else 0, act, _ptr(weight),
+          assignments, E, max_tiles, bm, top, N, Kd, (1 if gated else 2) if up else 0, act,
+          _ptr(weight),
           float(limit), _stream())
 
 
@@ -860,6 +935,70 @@ def moe_combine(x: torch.Tensor, y: torch.Tensor, top: int, shared: Optional[tor
           _ptr(x), _ptr(y), top, _ptr(shared), parts, stride, _ptr(sg), T, H, _ptr(ids), _ptr(w),
           experts, _ptr(h), code_of(h.dtype) if h is not None else F32, 1 if store else 0,
           _stream())
+
+
+# ------------------------------------------------------------------------------ differential attention
+DIFF_MAX_DIM, DIFF_MAX_VDIM = 256, 512      # of the general kernels
+
+
+def maps_norm_rope_store(rows: torch.Tensor, bias: Optional[torch.Tensor], q_norm: torch.Tensor,
+                         k_norm: torch.Tensor, eps: float, inv_freq: Optional[torch.Tensor],
+                         rot_dim: int, amplitude: float, step, line, nh: int, nkv: int,
+                         maps: int, dim: int, vd: int, q_out: torch.Tensor) -> None:
+    """From the rows [q | k | v] of a product (``rows`` [T, width], or float32 [parts, T, width]:
+    its split sums) with ``maps`` queries a head and ``maps`` keys a key head: the bias (float32
+    [width]) is added, every map of q and k is normed (weights float32 [dim]) and rotated
+    (cosine and sine times ``amplitude``), q goes to ``q_out``, keys (all maps of a head one
+    after the other) and values into the cache line."""
+    T = q_out.shape[0]
+    parts, stride = (1, 0) if rows.dim() == 2 else (rows.shape[0], rows.stride(0))
+    assert rows.shape[-2] == T and rows.stride(-1) == 1
+    assert rows.dim() == 2 or rows.dtype == torch.float32
+    ld = rows.stride(-2)
+    assert ld >= (nh + nkv) * maps * dim + nkv * vd
+    assert q_out.is_contiguous() and q_out.shape[1] == nh * maps * dim
+    assert line.head_dim == maps * dim and line.kv_heads == nkv
+    assert q_out.dtype == line.k.dtype == line.v.dtype
+    for t in (q_norm, k_norm):
+        assert t.dtype == torch.float32 and t.numel() == dim
+    assert bias is None or (bias.dtype == torch.float32 and bias.is_contiguous())
+    if rot_dim > 0 and (inv_freq is None or inv_freq.dtype != torch.float32
+                        or inv_freq.numel() < rot_dim // 2):
+        raise KernelError(f"a rotation of {rot_dim} values without its frequencies")
+    _call("rope", "mb_maps_norm_rope_store",
+          [_vp, _i, _i, _ll, _i, _vp, _vp, _vp, _f, _vp, _i, _f, _vp, _vp, _vp, _i, _i, _vp, _vp,
+           _vp, _i, _i, _i, _i, _i, _i, _i, _vp],
+          _ptr(rows), code_of(rows.dtype), parts, stride, ld, _ptr(bias), _ptr(q_norm),
+          _ptr(k_norm), float(eps), _ptr(inv_freq), rot_dim, float(amplitude),
+          _ptr(step.tok_slot), _ptr(step.tok_pos), _ptr(line.page_table), line.max_pages,
+          line.ring_pages, _ptr(line.k), _ptr(line.v), _ptr(q_out), code_of(q_out.dtype), T, nh,
+          nkv, maps, dim, vd, _stream())
+
+
+def _diff_args(q, out, step, line, nh, nkv, dim, vd):
+    T = out.shape[0]
+    _contig(out, "out"), _contig(q, "q")
+    assert q.shape == (T, nh * 2 * dim) and out.shape == (T, nh * vd)
+    assert q.dtype == out.dtype == line.k.dtype == line.v.dtype
+    assert line.head_dim == 2 * dim and (line.v_dim or line.head_dim) == vd
+    assert line.kv_heads == nkv
+    return T
+
+
+def attention_diff(q: torch.Tensor, out: torch.Tensor, step, line, nh: int, nkv: int, dim: int,
+                   vd: int, window: int, scale: float, lam: float, factor: float,
+                   eps: float) -> None:
+    """Causal differential attention of the step's tokens over the cache line, in float32:
+    o = a_1 - lam a_2 of head h's two maps, out = factor * o / sqrt(mean(o^2) + eps).
+    q [T, nh * 2 * dim] (a head's two maps one after the other), out [T, nh * vd]."""
+    T = _diff_args(q, out, step, line, nh, nkv, dim, vd)
+    _call("attention_diff", "mb_attention_diff",
+          [_vp, _vp, _vp, _vp, _i, _vp, _i, _i, _vp, _vp, _i, _i, _i, _i, _i, _i, _f, _f, _f, _f,
+           _vp],
+          _ptr(q), _ptr(out), _ptr(line.k), _ptr(line.v), code_of(q.dtype),
+          _ptr(line.page_table), line.max_pages, line.ring_pages, _ptr(step.tok_slot),
+          _ptr(step.tok_pos), T, nh, nkv, dim, vd, window, float(scale), float(lam),
+          float(factor), float(eps), _stream())
 
 
 # ------------------------------------------------------------------------------ products

@@ -40,7 +40,8 @@ from ..errors import ConfigError
 class TensorNeed:
     """A tensor that a part binds: its name in the model folder, its shape and its role
     (``matrix``: a projection, drawn N(0, std) by the random-weights mode; ``vector``: a norm
-    weight, drawn 1 + N(0, norm_std); ``table``: an embedding, drawn like a matrix).
+    weight, drawn 1 + N(0, norm_std); ``table``: an embedding, drawn like a matrix;
+    ``choices``: int32 rows of different numbers below ``choices``).
     ``optional``: may be absent; ``must_equal``: if present it must hold the same bytes as the
     tensor of that name (a tied head's stored copy, ``model.qwen3.pas:555-567`` of the
     reference)."""
@@ -49,6 +50,7 @@ class TensorNeed:
     role: str = "matrix"
     optional: bool = False
     must_equal: Optional[str] = None
+    choices: int = 0
 
 
 @dataclass(frozen=True)

@@ -22,6 +22,12 @@ into x also writes that rounding of the new x, which the next sublayer (or the n
 which it is handed on as pending) reads. With ``side`` the block then adds an input of its own
 from the token: e = columns [col0, col0 + dim) of the row of a second embedding table,
 t = P (act(G x) * e), x += norm_side(t).
+
+``parallel_residual``: both sublayers read one norm of the residual and are added at once, each
+times a vector and all times a constant:
+h = norm_input(x); x += factor * (scales_mixer * mixer(h) + scales_ff * feed_forward(h)). The
+sublayers leave their outputs (stored, or as split sums) as terms of a ``BranchSums``, which the
+next norm, the next pass's entry or ``settle`` adds into x.
 """
 from __future__ import annotations
 
@@ -57,13 +63,18 @@ class PreNormResidualBlock(Part):
         return self.feed_forward.forward(h, x, step)
 
     def _norm(self, which, x, pending, **more):
-        norm = self.norms[which]
-        if pending is None:
-            return norm.forward(x, **more)
-        if getattr(norm, "accepts_pending", False):
-            return norm.forward(x, pending=pending, **more)
-        settle(x, pending)             # a norm that knows nothing of pending sums
+        return normed(self.norms[which], x, pending, **more)
+
+
+def normed(norm, x, pending, **more):
+    """norm(x) with what is pending added into x first: by the norm's own kernel where it can."""
+    if pending is None:
         return norm.forward(x, **more)
+    if getattr(norm, "accepts_branches" if isinstance(pending, BranchSums) else "accepts_pending",
+               False):
+        return norm.forward(x, pending=pending, **more)
+    settle(x, pending)             # a norm that knows nothing of pending sums
+    return norm.forward(x, **more)
 
 
 def settle(x, pending) -> None:
@@ -73,6 +84,20 @@ def settle(x, pending) -> None:
         pending.settle(x)
         return
     K.add_partials(x, pending.partial)
+
+
+class BranchSums:
+    """What is still to be added into the residual: x += sum over ``terms`` of
+    scale[c] * factor * (the sum of the term's parts). A term is (y, factor, scale): y float32
+    [T, H] or [parts, T, H] (the parts may lie in any order in memory), scale float32 [H] or
+    None."""
+
+    def __init__(self, terms):
+        self.terms = terms
+
+    def settle(self, x) -> None:
+        from .. import kernels as K
+        K.branch_norm(x, self.terms)
 
 
 class StreamUpdate:
@@ -279,6 +304,57 @@ class OutputNormResidualBlock(Part):
         return ReadyInput(h) if h is not x else None
 
 
+class ParallelResidualBlock(Part):
+    capturable = True
+    accepts_pending = True
+
+    def __init__(self, spec, prefix: str = "", mixer=None, feed_forward=None, norms=None):
+        super().__init__(spec, prefix)
+        self.mixer, self.feed_forward, self.norm = mixer, feed_forward, norms["input"]
+        p = spec.params
+        self.hidden = int(p["hidden_size"])
+        self.factor = float(p.get("factor", 1.0))
+        # the sublayers that this layer has, with the names of their scales (None: no scale)
+        self.names = {q: (prefix + n if n else None) for q, n in p["scales"].items()}
+        self.spare = [prefix + n for n in p.get("spare", [])]
+
+    def libraries(self, rt):
+        return ["elementwise"]
+
+    def tensors(self):
+        return ([TensorNeed(n, (self.hidden,), "vector") for n in self.names.values() if n]
+                + [TensorNeed(n, (self.hidden,), "vector", optional=True) for n in self.spare])
+
+    def bind(self, weights, rt) -> None:
+        self.rt = rt
+        # the layer's scale and the model's factor as one float32 vector
+        self.scale = {q: ((weights[n].to(torch.float32) * self.factor).contiguous() if n else None)
+                      for q, n in self.names.items()}
+
+    def _terms(self, which, part, h, args):
+        scale = self.scale[which]
+        rest = 1.0 if scale is not None else self.factor
+        if hasattr(part, "forward_terms"):
+            return [(y, f * rest, scale) for y, f in part.forward_terms(h, *args)]
+        y = torch.empty((h.shape[0], self.hidden), dtype=torch.float32, device=h.device)
+        if getattr(part, "can_store", False):
+            pending = part.forward(h, y, *args, store=True)
+            return [(pending.partial if pending is not None else y, rest, scale)]
+        y.zero_()
+        pending = part.forward(h, y, *args)
+        if pending is not None:
+            settle(y, pending)
+        return [(y, rest, scale)]
+
+    def forward(self, x, step, line, state, writes_cache: bool, pending=None):
+        h = normed(self.norm, x, pending)
+        terms = self._terms("mixer", self.mixer, h, (step, line, state, writes_cache))
+        if "feed_forward" in self.names:
+            terms += self._terms("feed_forward", self.feed_forward, h, (step,))
+        return BranchSums(terms)
+
+
 BLOCKS.register("prenorm_residual", PreNormResidualBlock)
+BLOCKS.register("parallel_residual", ParallelResidualBlock)
 BLOCKS.register("output_norm_residual", OutputNormResidualBlock)
 BLOCKS.register("hyper_connections", HyperConnectionsBlock)

@@ -11,7 +11,7 @@ import torch
 
 from .. import kernels as K
 from .base import EMBEDDINGS, ENTRIES, HEADS, Part, TensorNeed
-from .linear import Linear
+from .linear import Linear, Pending
 
 
 class TokenEmbedding(Part):
@@ -89,6 +89,42 @@ class PassInput(Part):
         K.pass_input(x, self.vector, x0 if self.add_embedding else None)
 
 
+class PassProjection(Part):
+    """What a pass through looped layers starts from: x = W_in [x ; x0] + step[row], x0 the
+    embedding's output (``names``: ``in`` [size, 2 size], x's columns first, and ``step`` [rows,
+    size]). One kernel adds what is still pending into x, writes [x ; x0] in the activation type
+    and puts step[row] in x's place; the product is added onto that."""
+    capturable = True
+    add_embedding = True        # the model keeps a copy of the embedding's output
+    accepts_pending = True      # forward(..., pending=) -> what is pending afterwards
+
+    def __init__(self, spec, prefix: str = ""):
+        super().__init__(spec, prefix)
+        p = spec.params
+        self.names = {k: prefix + v for k, v in p["names"].items()}
+        self.rows, self.row, self.size = int(p["rows"]), int(p["row"]), int(p["size"])
+
+    def tensors(self) -> List[TensorNeed]:
+        return [TensorNeed(self.names["in"], (self.size, 2 * self.size)),
+                TensorNeed(self.names["step"], (self.rows, self.size), "bias")]
+
+    def bind(self, weights: Dict[str, torch.Tensor], rt) -> None:
+        self.rt = rt
+        self.linear = Linear(weights[self.names["in"]], rt)
+        self.vector = weights[self.names["step"]][self.row].to(torch.float32).contiguous()
+
+    def forward(self, x: torch.Tensor, x0, pending=None):
+        from .block import BranchSums, settle
+        if pending is not None and not isinstance(pending, BranchSums):
+            settle(x, pending)
+            pending = None
+        both = torch.empty((x.shape[0], 2 * self.size), dtype=self.rt.dtype, device=x.device)
+        K.pass_concat(x, pending.terms if pending is not None else [], x0, self.vector, both)
+        y = self.linear(both, out_dtype=torch.float32, defer="any")
+        return BranchSums([(y.partial if isinstance(y, Pending) else y, 1.0, None)])
+
+
 EMBEDDINGS.register("token_embedding", TokenEmbedding)
 ENTRIES.register("pass_input", PassInput)
+ENTRIES.register("pass_projection", PassProjection)
 HEADS.register("lm_head", LmHead)

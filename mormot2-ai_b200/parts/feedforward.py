@@ -29,6 +29,7 @@ from .linear import Linear
 
 class SwiGluFfn(Part):
     capturable = True
+    can_store = True      # forward(..., store=True) writes its output into x instead of adding
 
     def __init__(self, spec, prefix: str = ""):
         super().__init__(spec, prefix)
@@ -56,12 +57,15 @@ class SwiGluFfn(Part):
             weights.pop(n["up"], None)
         self.down = Linear(weights[n["down"]], rt)
 
-    def forward(self, h, x, step):
-        """Adds the feed-forward's output into x, or returns it as ``Pending`` split sums for
-        the next norm to add."""
+    def forward(self, h, x, step, store: bool = False):
+        """Adds the feed-forward's output into x (``store``: writes it there), or returns it as
+        ``Pending`` split sums for whoever reads it next (x is then not touched)."""
         from .linear import Pending
         act = self.gate_up(h)
-        out = self.down(act, add_into=x, defer=True)
+        if store:
+            out = self.down(act, out=x, defer="any")
+        else:
+            out = self.down(act, add_into=x, defer=True)
         return out if isinstance(out, Pending) else None
 
 

@@ -19,6 +19,11 @@ are identity experts without tensors, whose output is the input h times the weig
 ``activation = "clamped_swish"`` with ``limit``: g = min(W_g h, limit),
 u = clamp(W_u h, −limit, limit), g · sigmoid(1.702 g) · (u + 1) (the shared expert has a
 ``shared_limit`` of its own). ``shared_gate = False``: the shared expert is added as it is.
+
+``table_experts``: experts without a router. A table [vocab, top] names every token id's
+experts, each with the weight 1 / top; an expert is W_d act(W_u h) without a gate, and so is the
+shared one, which runs for every token. The lists of a step depend on its token ids only: they
+are made once in a pass of the model, however often its layer runs.
 """
 from __future__ import annotations
 
@@ -27,7 +32,7 @@ from typing import Dict, List
 import torch
 
 from .. import kernels as K
-from ..errors import ConfigError
+from ..errors import ConfigError, WeightsError
 from .base import FEED_FORWARDS, Part, TensorNeed
 from .linear import Linear, Pending
 
@@ -35,6 +40,16 @@ from .linear import Linear, Pending
 def _sums(result):
     """A product's float32 result [T, N], or its pending split sums as [parts, T, N]."""
     return result.partial if isinstance(result, Pending) else result
+
+
+def tile_rows(rt, w_up, T: int, A: int, E: int, hidden: int, inter: int) -> int:
+    """Rows per tile of an expert's list: 128 where the tensor-core kernel runs (bfloat16; 8
+    for a decode step of at most 8 tokens, the form that reads weights into registers), else
+    64, or 16 while an expert has few rows, so that few multiply-adds are wasted."""
+    fast = rt.fast_kernels and w_up.dtype == torch.bfloat16 and hidden % 8 == 0 and inter % 8 == 0
+    if fast and T <= 8 and hidden % 32 == 0 and inter % 32 == 0:
+        return 8        # a decode step: no expert has more rows, its weights stream once
+    return 128 if fast else (64 if A > 16 * E else 16)
 
 
 class RoutedExperts(Part):
@@ -157,14 +172,7 @@ class RoutedExperts(Part):
         w = torch.empty((T, top), dtype=torch.float32, device=dev)
         sg = (torch.empty((T,), dtype=torch.float32, device=dev)
               if self.shared_size and self.shared_gate else None)
-        # rows per tile of an expert's list: 128 where the tensor-core kernel runs (bfloat16; 8
-        # for a decode step of at most 8 tokens, the form that reads weights into registers),
-        # else 64, or 16 while an expert has few rows, so that few multiply-adds are wasted
-        fast = self.rt.fast_kernels and self.w_up.dtype == torch.bfloat16 and self.hidden % 8 == 0 \
-            and self.inter % 8 == 0
-        bm = 128 if fast else (64 if A > 16 * E else 16)
-        if fast and T <= 8 and self.hidden % 32 == 0 and self.inter % 32 == 0:
-            bm = 8      # a decode step: no expert has more rows, its weights stream once
+        bm = tile_rows(self.rt, self.w_up, T, A, E, self.hidden, self.inter)
         max_tiles = (A + bm - 1) // bm + E
         plan = torch.empty((2 + E + A + 2 * max_tiles,), dtype=torch.int32, device=dev)
         R = self.routed
@@ -197,4 +205,102 @@ class RoutedExperts(Part):
         return None
 
 
+class TableExperts(Part):
+    capturable = True
+
+    def __init__(self, spec, prefix: str = ""):
+        super().__init__(spec, prefix)
+        p = spec.params
+        self.hidden, self.vocab = int(p["hidden_size"]), int(p["vocab_size"])
+        self.experts, self.top = int(p["experts"]), int(p["top"])
+        self.inter, self.shared_size = int(p["intermediate_size"]), int(p.get("shared_size", 0))
+        if not 0 < self.top <= self.experts:
+            raise ConfigError(f"{self.top} of {self.experts} experts per token")
+        if p["activation"] not in K.UNARY_ACTIVATIONS:
+            raise ConfigError(f"activation \"{p['activation']}\" is not known "
+                              f"(known: {', '.join(sorted(K.UNARY_ACTIVATIONS))})")
+        self.act = K.UNARY_ACTIVATIONS[p["activation"]]
+        names = p["names"]
+        self.n_table = prefix + names["table"]
+        self.n_expert = [prefix + names["expert"].format(e) for e in range(self.experts)]
+        self.n_shared = prefix + names["shared"]
+        self.up, self.down = names["up"], names["down"]
+
+    def libraries(self, rt) -> List[str]:
+        return ["moe"]
+
+    def tensors(self) -> List[TensorNeed]:
+        out = [TensorNeed(self.n_table, (self.vocab, self.top), "choices", choices=self.experts)]
+        pairs = [(e, self.inter) for e in self.n_expert]
+        if self.shared_size:
+            pairs.append((self.n_shared, self.shared_size))
+        for name, size in pairs:
+            out += [TensorNeed(name + self.up, (size, self.hidden)),
+                    TensorNeed(name + self.down, (self.hidden, size))]
+        return out
+
+    def bind(self, weights: Dict[str, torch.Tensor], rt) -> None:
+        self.rt = rt
+        consume = getattr(rt, "consume_weights", False)
+        take = (lambda name: weights.pop(name)) if consume else (lambda name: weights[name])
+        self.table = weights[self.n_table].contiguous()
+        if self.table.dtype != torch.int32:
+            raise WeightsError(f"{self.n_table} holds {self.table.dtype}, not integers")
+        lo, hi = int(self.table.min()), int(self.table.max())
+        if lo < 0 or hi >= self.experts:
+            raise WeightsError(f"{self.n_table} names experts {lo} to {hi} of {self.experts}")
+        ws = [take(e + k) for e in self.n_expert for k in (self.up, self.down)]
+        kind = ws[0].dtype if len({w.dtype for w in ws}) == 1 else torch.float32
+        # all experts' weights in two tensors: [E, ff, hidden] and [E, hidden, ff]
+        self.w_up = torch.empty((self.experts, self.inter, self.hidden), dtype=kind,
+                                device=ws[0].device)
+        self.w_down = torch.empty((self.experts, self.hidden, self.inter), dtype=kind,
+                                  device=ws[0].device)
+        for e in range(self.experts):
+            self.w_up[e].copy_(ws[2 * e])
+            self.w_down[e].copy_(ws[2 * e + 1])
+            ws[2 * e] = ws[2 * e + 1] = None
+        self.shared_up = self.shared_down = None
+        if self.shared_size:
+            self.shared_up = Linear(weights[self.n_shared + self.up], rt, unary=self.act)
+            self.shared_down = Linear(weights[self.n_shared + self.down], rt)
+
+    def plan(self, step, T: int):
+        """(rows per tile, most tiles, the device's lists), made at the layer's first run in a
+        pass of the model."""
+        have = step.memo.get(id(self))
+        if have is None:
+            A = T * self.top
+            bm = tile_rows(self.rt, self.w_up, T, A, self.experts, self.hidden, self.inter)
+            max_tiles = (A + bm - 1) // bm + self.experts
+            plan = torch.empty((2 + self.experts + A + 2 * max_tiles,), dtype=torch.int32,
+                               device=self.table.device)
+            K.moe_table_plan(self.table, step.tok_ids, self.experts, bm, max_tiles, plan)
+            have = step.memo[id(self)] = (bm, max_tiles, plan)
+        return have
+
+    def forward_terms(self, h, step):
+        """The output as terms [(y, factor)]: the experts' rows as one part per choice, and the
+        shared expert's product."""
+        T, dev = h.shape[0], h.device
+        A = T * self.top
+        bm, max_tiles, plan = self.plan(step, T)
+        act = torch.empty((A, self.inter), dtype=self.rt.dtype, device=dev)
+        K.moe_gemm(h, self.w_up, act, plan, A, max_tiles, bm, self.top, True, self.act,
+                   gated=False)
+        y = torch.empty((A, self.hidden), dtype=torch.float32, device=dev)
+        K.moe_gemm(act, self.w_down, y, plan, A, max_tiles, bm, self.top, False, self.act)
+        # row t * top + k is token t's k-th choice
+        terms = [(y.view(T, self.top, self.hidden).transpose(0, 1), 1.0 / self.top)]
+        if self.shared_size:
+            sa = self.shared_up(h)
+            terms.append((_sums(self.shared_down(sa, out_dtype=torch.float32, defer="any")), 1.0))
+        return terms
+
+    def forward(self, h, x, step):
+        K.branch_norm(x, [(y, f, None) for y, f in self.forward_terms(h, step)])
+        return None
+
+
 FEED_FORWARDS.register("routed_experts", RoutedExperts)
+FEED_FORWARDS.register("table_experts", TableExperts)

@@ -21,6 +21,7 @@ from .base import NORMS, Part, TensorNeed
 class RmsNorm(Part):
     capturable = True
     accepts_pending = True      # forward(..., pending=) adds split sums into x before it norms
+    accepts_branches = True     # ... or scaled sums of several sublayers (block.BranchSums)
 
     def __init__(self, spec, prefix: str = ""):
         super().__init__(spec, prefix)
@@ -51,6 +52,9 @@ class RmsNorm(Part):
         are first added into x."""
         R = n_rows if n_rows is not None else (rows.numel() if rows is not None else x.shape[0])
         out = torch.empty((R, self.size), dtype=self.rt.dtype, device=x.device)
+        if hasattr(pending, "terms") and rows is None:      # sublayers' outputs, each with its scale
+            K.branch_norm(x, pending.terms, self.weight, self.eps, out)
+            return out
         K.rmsnorm(x, self.weight, self.eps, out, rows, R,
                   pending.partial if pending is not None else None)
         return out

@@ -4,7 +4,7 @@ large shapes.
 
 Matrices, tables and biases are N(0, std), norm weights 1 + N(0, norm_std), fractions (the
 weights of a blend of two rows) uniform in [0, 1), matrices near the identity I + N(0,
-norm_std); drawn in float32 from one
+norm_std), rows of choices int32 without repetition; drawn in float32 from one
 seeded generator in the order of the tensor names and then rounded to the stored type (the
 reference's fixture tool draws 0.08·randn and 1 + 0.25·randn and rounds to BF16:
 ``tools/infer-ref/make_reference_qwen3.py:837-844`` of the reference project).
@@ -31,6 +31,11 @@ def random_tensors(needs: Iterable[TensorNeed], seed: int, std: float = 0.02,
         if any(d < 0 for d in n.shape):
             raise ValueError(f"{n.name}: a size that only a stored tensor gives; the "
                              "configuration of a random model must name it")
+        if n.role == "choices":
+            # every row: the first of a random order of all numbers
+            rows = torch.rand((n.shape[0], n.choices), generator=gen, device=device)
+            out[n.name] = rows.argsort(dim=1)[:, :n.shape[1]].to(torch.int32).contiguous()
+            continue
         if device == "cpu":
             t = torch.randn(n.shape, generator=gen, dtype=torch.float32)
         else:

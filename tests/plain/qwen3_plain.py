@@ -25,7 +25,8 @@ f64 = np.float64
 # ----------------------------------------------------------------------------- files
 def read_safetensors(path: str) -> Dict[str, np.ndarray]:
     """Every tensor of a safetensors file as float32 (BF16 widened exactly: a BF16 value is the
-    upper half of a float32, src/infer/mormot.ai.infer.tensor.pas:483)."""
+    upper half of a float32, src/infer/mormot.ai.infer.tensor.pas:483); integer tables as
+    int32."""
     with open(path, "rb") as f:
         (n,) = struct.unpack("<Q", f.read(8))
         header = json.loads(f.read(n))
@@ -41,6 +42,8 @@ def read_safetensors(path: str) -> Dict[str, np.ndarray]:
             a = u.view(np.float32)
         elif e["dtype"] == "F32":
             a = np.frombuffer(raw, dtype=np.float32)
+        elif e["dtype"] == "I32":
+            a = np.frombuffer(raw, dtype=np.int32)
         else:
             raise ValueError(f"{name}: {e['dtype']}")
         out[name] = a.reshape(e["shape"]).copy()
