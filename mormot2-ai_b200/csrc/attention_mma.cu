@@ -21,8 +21,7 @@
 // template parameter of the kernels so that models without one run the code they ran before)
 // and a gate (`gate` not null: head h of token t at gate[t * gate_stride + h], a logit whose
 // sigmoid multiplies the head's output where it is written).
-#include "mma_common.cuh"
-#include "tc_common.cuh"
+#include "attention_mma.cuh"
 
 MB_DEFINE_LAST_ERROR
 
@@ -101,31 +100,7 @@ __device__ __forceinline__ void load_q(const bf16* q0, const bf16* q1, int c, ui
   }
 }
 
-// 16 bytes of a tile in shared memory
-__device__ __forceinline__ uint4 lds16(uint32_t addr) {
-  uint4 v;
-  asm volatile("ld.shared.v4.u32 {%0, %1, %2, %3}, [%4];"
-               : "=r"(v.x), "=r"(v.y), "=r"(v.z), "=r"(v.w)
-               : "r"(addr));
-  return v;
-}
-
-// `bytes` contiguous bytes from global to shared memory (both 16-byte aligned), completing `bar`
-__device__ __forceinline__ void bulk_copy(uint32_t dst, const void* src, uint32_t bytes,
-                                          uint32_t bar) {
-  asm volatile(
-      "cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];"
-      ::"r"(dst), "l"(src), "r"(bytes), "r"(bar)
-      : "memory");
-}
-
 #define DEC_STAGES 3
-
-__device__ __forceinline__ float ld_cluster_f32(uint32_t cluster_addr) {
-  float v;
-  asm volatile("ld.shared::cluster.f32 %0, [%1];" : "=f"(v) : "r"(cluster_addr) : "memory");
-  return v;
-}
 
 // One CTA per (token, KV head [x 16 query heads of its group], split). Warp 4 streams the
 // pages of this split (every `splits`-th page of the sequence) into shared memory, a whole K
@@ -570,60 +545,6 @@ MB_EXPORT int mb_attention_decode_clusters(const void* q, int q_stride, void* ou
 // query head; each of its four warps owns 16 of them as the rows of the MMA and walks the pages
 // from the first key its rows may see to the last, with an online softmax per row. The four
 // warps read the same pages, so all but the first read hit the L1 cache.
-// the same pieces as qk_page / pv_page with the page's tiles in shared memory
-template <int HD, int KP>
-__device__ __forceinline__ void qk_page_smem(const uint4* qa, const uint4* qb, uint32_t ks, int r,
-                                             int c, float sc[8][4]) {
-#pragma unroll
-  for (int u = 0; u < 8; ++u) {
-    sc[u][0] = sc[u][1] = sc[u][2] = sc[u][3] = 0.f;
-    const uint32_t krow = ks + (uint32_t)(u * 8 + r) * KP + c * 16;
-#pragma unroll
-    for (int ch = 0; ch < HD / 32; ++ch) {
-      const uint4 kb = lds16(krow + ch * 64);
-      mma_bf16(sc[u], qa[ch].x, qb[ch].x, qa[ch].y, qb[ch].y, kb.x, kb.y);
-      mma_bf16(sc[u], qa[ch].z, qb[ch].z, qa[ch].w, qb[ch].w, kb.z, kb.w);
-    }
-  }
-}
-
-template <int HD, int VP>
-__device__ __forceinline__ void pv_page_smem(const float sc[8][4], uint32_t vs, int r, int c,
-                                             float o[HD / 64][8][4]) {
-#pragma unroll
-  for (int kk = 0; kk < 4; ++kk) {
-    const uint32_t a0 = pack_bf16(sc[2 * kk][0], sc[2 * kk][1]);
-    const uint32_t a1 = pack_bf16(sc[2 * kk][2], sc[2 * kk][3]);
-    const uint32_t a2 = pack_bf16(sc[2 * kk + 1][0], sc[2 * kk + 1][1]);
-    const uint32_t a3 = pack_bf16(sc[2 * kk + 1][2], sc[2 * kk + 1][3]);
-    const uint32_t vrow = vs + (uint32_t)(kk * 16 + 2 * c) * VP + r * 16;
-#pragma unroll
-    for (int db = 0; db < HD / 64; ++db) {
-      const uint4 va = lds16(vrow + db * 128);
-      const uint4 vb = lds16(vrow + VP + db * 128);
-      const uint4 vc = lds16(vrow + 8 * VP + db * 128);
-      const uint4 vd = lds16(vrow + 9 * VP + db * 128);
-      const uint32_t wa[4] = {va.x, va.y, va.z, va.w}, wb[4] = {vb.x, vb.y, vb.z, vb.w};
-      const uint32_t wc[4] = {vc.x, vc.y, vc.z, vc.w}, wd[4] = {vd.x, vd.y, vd.z, vd.w};
-#pragma unroll
-      for (int j = 0; j < 8; ++j) {
-        const int w = j >> 1;
-        const uint32_t b0 = (j & 1) ? pack_hi(wa[w], wb[w]) : pack_lo(wa[w], wb[w]);
-        const uint32_t b1 = (j & 1) ? pack_hi(wc[w], wd[w]) : pack_lo(wc[w], wd[w]);
-        mma_bf16(o[db][j], a0, a1, a2, a3, b0, b1);
-      }
-    }
-  }
-}
-
-__device__ __forceinline__ void cp_async16(uint32_t dst, const void* src) {
-  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst), "l"(src) : "memory");
-}
-__device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
-template <int N> __device__ __forceinline__ void cp_async_wait() {
-  asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory");
-}
-
 #define PRE_STAGES 3
 
 // A CTA takes 64 consecutive new tokens of one sequence and one query head; each of its four

@@ -57,7 +57,8 @@ SOURCES = {
 }
 HEADERS = ["common.cuh"]
 EXTRA_HEADERS = {"gemm_tc": ["tc_common.cuh"],
-                 "attention_mma": ["mma_common.cuh", "tc_common.cuh", "no_alloc.h"],
+                 "attention_mma": ["attention_mma.cuh", "mma_common.cuh", "tc_common.cuh", "no_alloc.h"],
+                 "attention_diff": ["attention_mma.cuh", "mma_common.cuh", "tc_common.cuh"],
                  "attention_tc": ["tc_common.cuh"],
                  "latent": ["mma_common.cuh", "mma_tile.cuh"],
                  "moe": ["mma_common.cuh", "mma_tile.cuh"],

@@ -162,6 +162,11 @@ class Runtime:
                                factor, eps) -> None:
         """Differential attention: the tensor-core kernels for bfloat16 and the sizes they take,
         else the float32 kernel."""
+        if self.fast_kernels:
+            from ..parts import attention_fast
+            if attention_fast.run_differential(self, q, out, step, line, nh, nkv, dim, vd, window,
+                                               scale, lam, factor, eps):
+                return
         K.attention_diff(q, out, step, line, nh, nkv, dim, vd, window, scale, lam, factor, eps)
 
     def attention(self, q, q_stride, out, step, line, nh, nkv, hd, window, scale, vd=0,

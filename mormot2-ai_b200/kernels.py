@@ -1001,6 +1001,36 @@ def attention_diff(q: torch.Tensor, out: torch.Tensor, step, line, nh: int, nkv:
           float(factor), float(eps), _stream())
 
 
+def attention_diff_decode(q: torch.Tensor, out: torch.Tensor, step, line, nh: int, nkv: int,
+                          dim: int, vd: int, window: int, scale: float, lam: float,
+                          factor: float, eps: float, splits: int,
+                          error: torch.Tensor) -> None:
+    """``attention_diff`` of a decode step on the tensor cores (bfloat16; dim and vd multiples
+    of 8, at most 128 and 256); ``splits`` CTAs share a sequence's pages."""
+    T = _diff_args(q, out, step, line, nh, nkv, dim, vd)
+    _call("attention_diff", "mb_attention_diff_decode",
+          [_vp, _vp, _vp, _vp, _vp, _i, _i, _vp, _vp, _i, _i, _i, _i, _i, _i, _f, _f, _f, _f, _i,
+           _vp, _vp],
+          _ptr(q), _ptr(out), _ptr(line.k), _ptr(line.v), _ptr(line.page_table), line.max_pages,
+          line.ring_pages, _ptr(step.tok_slot), _ptr(step.tok_pos), T, nh, nkv, dim, vd, window,
+          float(scale), float(lam), float(factor), float(eps), splits, _ptr(error), _stream())
+
+
+def attention_diff_prefill(q: torch.Tensor, out: torch.Tensor, step, line, nh: int, nkv: int,
+                           dim: int, vd: int, window: int, scale: float, lam: float,
+                           factor: float, eps: float) -> None:
+    """``attention_diff`` of the new tokens of several sequences on the tensor cores (sizes as
+    for ``attention_diff_decode``)."""
+    _diff_args(q, out, step, line, nh, nkv, dim, vd)
+    _call("attention_diff", "mb_attention_diff_prefill",
+          [_vp, _vp, _vp, _vp, _vp, _i, _i, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _f, _f,
+           _f, _f, _vp],
+          _ptr(q), _ptr(out), _ptr(line.k), _ptr(line.v), _ptr(line.page_table), line.max_pages,
+          line.ring_pages, _ptr(step.seq_start), _ptr(step.seq_past), _ptr(step.seq_slot),
+          step.B, step.max_new, nh, nkv, dim, vd, window, float(scale), float(lam),
+          float(factor), float(eps), _stream())
+
+
 # ------------------------------------------------------------------------------ products
 def gemm_simt(a: torch.Tensor, w: torch.Tensor, c: torch.Tensor, epilogue: int = EPI_STORE) -> None:
     """c = a · wᵀ (store), c += a · wᵀ (add, float32 c), or SwiGLU over w = [gate; up]

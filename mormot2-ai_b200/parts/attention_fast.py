@@ -82,3 +82,28 @@ def run(rt, q, q_stride, out, step, line, nh, nkv, hd, window, scale, sink=None,
     K.attention_prefill(q, q_stride, out, step, line, nh, nkv, hd, window, scale,
                         rt.error_word, sink, *more)
     return True
+
+
+def diff_decode_splits(line, T: int, nh: int, nkv: int, sms: int, window: int) -> int:
+    """``decode_splits`` for differential attention, whose CTAs take 8 query heads of a KV head
+    (two maps each)."""
+    pages = line.max_pages
+    if window > 0:
+        pages = min(pages, pages_for(window) + 1)
+    groups = max(1, T * nkv * ((nh // nkv + 7) // 8))
+    return max(1, min((2 * sms) // groups, pages, MAX_DECODE_SPLITS))
+
+
+def run_differential(rt, q, out, step, line, nh, nkv, dim, vd, window, scale, lam, factor,
+                     eps) -> bool:
+    """Differential attention: True if a tensor-core kernel took the call."""
+    if (q.dtype != torch.bfloat16 or dim % 8 or vd % 8 or dim > 128 or vd > 256
+            or any(t.data_ptr() % 16 for t in (q, out, line.k, line.v))):
+        return False
+    if step.decode:
+        K.attention_diff_decode(q, out, step, line, nh, nkv, dim, vd, window, scale, lam, factor,
+                                eps, diff_decode_splits(line, step.T, nh, nkv, rt.sms, window),
+                                rt.error_word)
+        return True
+    K.attention_diff_prefill(q, out, step, line, nh, nkv, dim, vd, window, scale, lam, factor, eps)
+    return True
