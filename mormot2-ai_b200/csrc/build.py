@@ -54,12 +54,14 @@ SOURCES = {
     "recurrent": "recurrent.cu",
     "linear_state": "linear_state.cu",
     "attention_diff": "attention_diff.cu",
+    "attention_diff_tc": "attention_diff_tc.cu",
 }
 HEADERS = ["common.cuh"]
 EXTRA_HEADERS = {"gemm_tc": ["tc_common.cuh"],
                  "attention_mma": ["attention_mma.cuh", "mma_common.cuh", "tc_common.cuh", "no_alloc.h"],
                  "attention_diff": ["attention_mma.cuh", "mma_common.cuh", "tc_common.cuh"],
-                 "attention_tc": ["tc_common.cuh"],
+                 "attention_tc": ["attention_tc.cuh", "tc_common.cuh"],
+                 "attention_diff_tc": ["attention_tc.cuh", "tc_common.cuh"],
                  "latent": ["mma_common.cuh", "mma_tile.cuh"],
                  "moe": ["mma_common.cuh", "mma_tile.cuh"],
                  "latent_mma": ["mma_common.cuh"]}

@@ -1031,6 +1031,22 @@ def attention_diff_prefill(q: torch.Tensor, out: torch.Tensor, step, line, nh: i
           float(factor), float(eps), _stream())
 
 
+def attention_diff_prefill_tc(q: torch.Tensor, out: torch.Tensor, step, line, nh: int, nkv: int,
+                              dim: int, vd: int, window: int, scale: float, lam: float,
+                              factor: float, eps: float, error: torch.Tensor) -> None:
+    """``attention_diff_prefill`` on tcgen05 (dim 64; vd 64 or 128; a positive scale): both
+    maps' scores and outputs in tensor memory, tiles by TMA."""
+    T = _diff_args(q, out, step, line, nh, nkv, dim, vd)
+    pool_rows = line.k.shape[0] * line.k.shape[1] * line.k.shape[2]
+    _call("attention_diff_tc", "mb_attention_diff_prefill_tc",
+          [_vp, _vp, _vp, _vp, _ll, _vp, _i, _i, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _i,
+           _f, _f, _f, _f, _vp, _vp],
+          _ptr(q), _ptr(out), _ptr(line.k), _ptr(line.v), pool_rows, _ptr(line.page_table),
+          line.max_pages, line.ring_pages, _ptr(step.seq_start), _ptr(step.seq_past),
+          _ptr(step.seq_slot), step.B, T, step.max_new, nh, nkv, dim, vd, window, float(scale),
+          float(lam), float(factor), float(eps), _ptr(error), _stream())
+
+
 # ------------------------------------------------------------------------------ products
 def gemm_simt(a: torch.Tensor, w: torch.Tensor, c: torch.Tensor, epilogue: int = EPI_STORE) -> None:
     """c = a · wᵀ (store), c += a · wᵀ (add, float32 c), or SwiGLU over w = [gate; up]

@@ -105,5 +105,10 @@ def run_differential(rt, q, out, step, line, nh, nkv, dim, vd, window, scale, la
                                 eps, diff_decode_splits(line, step.T, nh, nkv, rt.sms, window),
                                 rt.error_word)
         return True
+    if dim == 64 and vd in (64, 128) and scale > 0:
+        # S and O of both maps in tensor memory, tiles by TMA (csrc/attention_diff_tc.cu)
+        K.attention_diff_prefill_tc(q, out, step, line, nh, nkv, dim, vd, window, scale, lam,
+                                    factor, eps, rt.error_word)
+        return True
     K.attention_diff_prefill(q, out, step, line, nh, nkv, dim, vd, window, scale, lam, factor, eps)
     return True

@@ -49,7 +49,7 @@ class DifferentialAttention(Part):
         self.ow = self.nh * self.vd
 
     def libraries(self, rt) -> List[str]:
-        return ["rope", "attention_diff"]
+        return ["rope", "attention_diff"] + (["attention_diff_tc"] if rt.fast_kernels else [])
 
     def tensors(self) -> List[TensorNeed]:
         n, d = self.names, self.dim
