@@ -1,7 +1,7 @@
 """Measures decoding and prefill of the Qwen3-8B shape with random weights on one B200.
 
     python bench.py [--gpus 1] [--steps K] [--warmup W] [--impl ours|reference]
-    python bench.py --design busavik|fimudra|sezopel|laralix [--sizes small,mid]   (another workload, see below)
+    python bench.py --design busavik|fimudra|sezopel|laralix|lotirax [--sizes small,mid]   (another workload, see below)
 
 A step is one decode step of a batch of 8 sequences whose context reaches 4,096 at the end of
 the timed steps. ``value`` is decoded tokens a second with the steps running back to back on
@@ -28,7 +28,8 @@ state, routed experts with identity experts), ``--design sezopel`` for the Sezop
 keys and values, retention, normed sublayer outputs, an input from the token after every layer),
 ``--design laralix`` for the Laralix design (windowed attention with a distance bias beside the
 gated delta rule, attention whose values are its keys beside gated linear attention, latent
-attention with neighbours turned).
+attention with neighbours turned), ``--design lotirax`` for the Lotirax design (windowed
+differential attention, sublayers side by side, experts that a table names, looped layers).
 """
 import argparse
 import json
@@ -488,6 +489,71 @@ def laralix_shapes(name):
     return LaralixConfig.from_dict(doc), twin
 
 
+def lotirax_shapes(name):
+    """A Lotirax configuration whose layers have the sizes of a real model's (a layer with a gated
+    feed-forward, one with experts that a table names and one gated again, the last two passed
+    twice; windows of 1,024 positions) and the Qwen3 configuration of equal width, head count,
+    KV heads, feed-forward size, layer runs and windows whose heads have as many values as a
+    head's two maps together: the closest model of this library."""
+    from mormot2_ai_b200 import LotiraxConfig, Qwen3Config
+    sizes = {
+        # width, heads, kv heads, dim, vdim, ff, experts, top, expert ff, shared ff
+        "small": (1024, 8, 2, 64, 128, 2816, 16, 2, 704, 1408),
+        "mid": (4096, 32, 8, 64, 128, 11008, 32, 4, 1376, 5504),
+    }[name]
+    w, h, kv, dim, vd, ff, ne, top, eff, sff = sizes
+    vocab, window = 32768, 1024
+    mixer = {"heads": h, "kv_heads": kv, "dim": dim, "vdim": vd, "scale": dim ** -0.5,
+             "diff": 0.5, "mask": {"size": window},
+             "rot": {"base": 1e6, "dims": dim,
+                     "scaling": {"factor": 4.0, "original": 4096, "fast": 32.0, "slow": 1.0}}}
+    dense = {"type": "attention", "mixer": mixer, "mlp": {"kind": "dense", "ff": ff}}
+    moe = {"type": "attention", "mixer": mixer,
+           "mlp": {"kind": "moe", "expert": {"ff": eff}, "router": {"experts": ne, "top": top},
+                   "shared": {"ff": sff}}}
+    doc = {"architecture": "Lotirax", "vocab": vocab, "width": w, "norm": {"eps": 1e-6},
+           "residual_mult": 0.5, "loop": {"start": 1, "stop": 3, "times": 2},
+           "layers": [dense, moe, dense]}
+    twin = Qwen3Config(vocab_size=vocab, hidden_size=w, num_hidden_layers=5,
+                       num_attention_heads=h, num_key_value_heads=kv, head_dim=2 * dim,
+                       intermediate_size=ff, max_position_embeddings=40960,
+                       rms_norm_eps=1e-6, rope_theta=1e6, tie_word_embeddings=True,
+                       layer_windows=(window,) * 5)
+    return LotiraxConfig.from_dict(doc), twin
+
+
+def lotirax_work(cfg, tokens, batch, held, experts_read=None):
+    """As ``busavik_work`` for the Lotirax family: attention counts both products of both maps
+    over the pairs that the windows leave (a decode step the keys and values inside them, once),
+    the products every matrix of every layer run and the projection that opens a pass."""
+    out = {"prefill_flops": {"attention": 0.0, "products": 0.0},
+           "decode_bytes": {"attention": 0.0, "products": 0.0}}
+    w = cfg.width
+    for l, opens in cfg.order():
+        m, mlp = cfg.layers[l]["mixer"], cfg.layers[l].get("mlp")
+        h, kv, dim, vd = m["heads"], m["kv_heads"], m["dim"], m["vdim"]
+        size = (m.get("mask") or {}).get("size") or 0
+        run = (2 * (h + kv) * dim + kv * vd + h * vd) * w + (2 * w * w if opens >= 0 else 0)
+        read = run
+        out["prefill_flops"]["attention"] += 4 * h * (dim + vd) * windowed_pairs(tokens, size)
+        seen = min(held / batch, size) if size else held / batch
+        out["decode_bytes"]["attention"] += 2 * batch * seen * kv * (2 * dim + vd)
+        if mlp and mlp["kind"] == "dense":
+            run += 3 * w * mlp["ff"]
+            read += 3 * w * mlp["ff"]
+        elif mlp:
+            one = 2 * w * mlp["expert"]["ff"]
+            shared = 2 * w * mlp["shared"]["ff"] if mlp.get("shared") else 0
+            top, e = mlp["router"]["top"], mlp["router"]["experts"]
+            run += top * one + shared
+            read += (min(e, batch * top) if experts_read is None else experts_read) * one + shared
+        out["prefill_flops"]["products"] += 2 * tokens * run
+        out["decode_bytes"]["products"] += 2 * read
+    out["prefill_flops"]["products"] += 2 * cfg.vocab * w
+    out["decode_bytes"]["products"] += 2 * cfg.vocab * w
+    return out
+
+
 def windowed_pairs(tokens, window, keep=0):
     """How many (query, key) pairs a prompt of ``tokens`` tokens has under a window that also
     keeps the first ``keep`` positions (0: all earlier positions are seen)."""
@@ -641,6 +707,8 @@ def busavik_work(cfg, tokens, batch, held, experts_read=None):
         return sezopel_work(cfg, tokens, batch, held)
     if getattr(cfg, "ARCHITECTURE", "") == "Laralix":
         return laralix_work(cfg, tokens, batch, held)
+    if getattr(cfg, "ARCHITECTURE", "") == "Lotirax":
+        return lotirax_work(cfg, tokens, batch, held, experts_read)
     pairs = tokens * (tokens + 1) / 2
     out = {"prefill_flops": {"attention": 0.0, "products": 0.0},
            "decode_bytes": {"attention": 0.0, "products": 0.0}}
@@ -696,7 +764,7 @@ def busavik_bench(a):
     points = {}
     for size in [v for v in a.sizes.split(",") if v]:
         shapes = {"fimudra": fimudra_shapes, "sezopel": sezopel_shapes,
-                  "laralix": laralix_shapes}.get(a.design, busavik_shapes)
+                  "laralix": laralix_shapes, "lotirax": lotirax_shapes}.get(a.design, busavik_shapes)
         for family, cfg in zip((a.design, "qwen3"), shapes(size)):
             eng = Engine.from_random(cfg, seed=5, std=0.02, max_tokens=batch * ctx + tokens,
                                      max_context=max(ctx, tokens), max_slots=batch,
@@ -726,7 +794,10 @@ def busavik_bench(a):
                         int(ids[ids < real].unique().numel()))
             dshares = {}
             for k in range(6):
-                _, sh, _ = eng.timed_step([Entry(s, [1 + k]) for s in slots])
+                # a table of experts is read by token ids: different ones in the batch
+                apart = 97 if a.design == "lotirax" else 0
+                _, sh, _ = eng.timed_step([Entry(s, [1 + k + apart * i])
+                                           for i, s in enumerate(slots)])
                 if k >= 2:
                     for name, ms in sh.items():
                         dshares[name] = dshares.get(name, 0.0) + ms / 4
@@ -775,8 +846,9 @@ def main():
                     help="token counts of the long prefill points (one sequence each)")
     ap.add_argument("--only-prefill", type=int, nargs="?", const=PREFILL_TOKENS, default=0,
                     help="only a prefill of this many tokens (for profiles; prints a short line)")
-    ap.add_argument("--design", default="", choices=["", "busavik", "fimudra", "sezopel", "laralix"],
-                    help="busavik, fimudra, sezopel, laralix: instead of the default workload, prefill and decode "
+    ap.add_argument("--design", default="", choices=["", "busavik", "fimudra", "sezopel", "laralix",
+                                                          "lotirax"],
+                    help="busavik, fimudra, sezopel, laralix, lotirax: instead of the default workload, prefill and decode "
                          "of that design at layer sizes of real models beside the Qwen3 model of "
                          "equal size (prints its own JSON line)")
     ap.add_argument("--sizes", default="small,mid", help="with --design: which layer sizes")

@@ -49,6 +49,7 @@ SOURCES = {
     "attention_tc": "attention_tc.cu",
     "latent": "latent.cu",
     "moe": "moe.cu",
+    "moe_tc": "moe_tc.cu",
     "latent_mma": "latent_mma.cu",
     "streams": "streams.cu",
     "recurrent": "recurrent.cu",
@@ -63,7 +64,8 @@ EXTRA_HEADERS = {"gemm_tc": ["tc_common.cuh"],
                  "attention_tc": ["attention_tc.cuh", "tc_common.cuh"],
                  "attention_diff_tc": ["attention_tc.cuh", "tc_common.cuh"],
                  "latent": ["mma_common.cuh", "mma_tile.cuh"],
-                 "moe": ["mma_common.cuh", "mma_tile.cuh"],
+                 "moe": ["mma_common.cuh", "mma_tile.cuh", "moe_act.cuh"],
+                 "moe_tc": ["tc_common.cuh", "moe_act.cuh"],
                  "latent_mma": ["mma_common.cuh"]}
 
 _lock = threading.Lock()

@@ -465,9 +465,11 @@ MB_EXPORT int mb_pass_input(float* x, const float* x0, const void* b, int b_dtyp
 // token's experts, a stored output), each with a factor and a vector over the columns:
 //   v[t, c] = x[t, c] + sum over the terms of scale[c] * factor * (p0 + p1 + ...)[t, c]
 // in the order of the terms and of their parts. CONCAT false: x = v and, with y, the RMS norm
-// y[t] = w * v / sqrt(mean(v^2) + eps). CONCAT true: y[t] = [v ; x0[t]] (2 H values) and
-// x[t] = w (float32), what the product of y is then added onto.
-// A thread holds 4 * VEC columns (V4; 16-byte accesses) or walks them one by one.
+// y[t] = w * v / sqrt(mean(v^2) + eps). CONCAT true: y[t] = [v ; x0[t]] (2 H values), x0[t] the
+// token's embedding (a row of `table` times `emb_scale`), and x[t] = w (float32), what the
+// product of y is then added onto.
+// A thread holds 4 * VEC columns (16-byte accesses) or walks them one by one. Up to BRANCH_FLAT
+// parts of all the terms together are one list whose loads are all asked for at once.
 struct BranchTerm {
   const float* p;
   const float* scale;      // [H] or null
@@ -480,13 +482,39 @@ struct BranchTerm {
 struct BranchTerms {
   BranchTerm t[BRANCH_TERMS];
   int n;
+  int parts;               // of all terms together
 };
+#define BRANCH_FLAT 8
+struct Embedding {         // what a pass concatenates: rows of a table by token id
+  const void* table;
+  const int* ids;
+  int bf16, rows;
+  float scale;
+};
+__device__ __forceinline__ size_t embedding_row(const Embedding& e, int t, int H) {
+  const int id = e.ids[t];
+  return (size_t)(id < 0 || id >= e.rows ? 0 : id) * H;
+}
+__device__ __forceinline__ float4 embedding4(const Embedding& e, size_t at) {
+  float4 v = e.bf16 ? load4<__nv_bfloat16>((const __nv_bfloat16*)e.table + at)
+                    : *(const float4*)((const float*)e.table + at);
+  v.x *= e.scale; v.y *= e.scale; v.z *= e.scale; v.w *= e.scale;
+  return v;
+}
 
-template <typename TO, int VEC, int THREADS, bool CONCAT>
+__device__ __forceinline__ void branch_add(float4& v, const float4& s, float factor,
+                                           const float4& u) {
+  v.x = fmaf(s.x * factor, u.x, v.x);
+  v.y = fmaf(s.y * factor, u.y, v.y);
+  v.z = fmaf(s.z * factor, u.z, v.z);
+  v.w = fmaf(s.w * factor, u.w, v.w);
+}
+
+template <typename TO, int VEC, int THREADS, int FLAT, bool CONCAT>
 __global__ void __launch_bounds__(THREADS)
 branch_vec_kernel(float* __restrict__ x, const __grid_constant__ BranchTerms terms,
                   const void* __restrict__ w, int w_bf16, float eps, TO* __restrict__ y,
-                  const float* __restrict__ x0, int H) {
+                  const __grid_constant__ Embedding emb, int H) {
   __shared__ float red[33];
   const int r = blockIdx.x;
   float* xr = x + (size_t)r * H;
@@ -508,6 +536,7 @@ branch_vec_kernel(float* __restrict__ x, const __grid_constant__ BranchTerms ter
       wv[i][0] = raw.x; wv[i][1] = raw.y; wv[i][2] = raw.z; wv[i][3] = raw.w;
     }
   }
+  const size_t row0 = CONCAT ? embedding_row(emb, r, H) : 0;
   mb_grid_wait();
   mb_grid_launch_next();
   float sum = 0.f;
@@ -516,29 +545,54 @@ branch_vec_kernel(float* __restrict__ x, const __grid_constant__ BranchTerms ter
     const int c = (i * THREADS + threadIdx.x) * 4;
     if (c >= H) continue;
     if (terms.n == 0) v[i] = *(const float4*)(xr + c);
-    for (int k = 0; k < terms.n; ++k) {
-      const BranchTerm& t = terms.t[k];
-      const float* pp = t.p + (size_t)r * t.row_stride + c;
-      float4 s = make_float4(1.f, 1.f, 1.f, 1.f), u = make_float4(0.f, 0.f, 0.f, 0.f);
-      if (t.scale) s = __ldg((const float4*)(t.scale + c));
-      for (int p0 = 0; p0 < t.parts; p0 += 8) {       // up to eight loads in flight
-        float4 a[8];
+    if (FLAT > 0) {
+      float4 a[FLAT > 0 ? FLAT : 1];
+      int j = 0;
 #pragma unroll
-        for (int j = 0; j < 8; ++j)
-          if (p0 + j < t.parts) a[j] = __ldg((const float4*)(pp + (size_t)(p0 + j) * t.part_stride));
+      for (int k = 0; k < BRANCH_TERMS; ++k) {
+        if (k >= terms.n) break;
+        const BranchTerm& t = terms.t[k];
+        const float* pp = t.p + (size_t)r * t.row_stride + c;
 #pragma unroll
-        for (int j = 0; j < 8; ++j)
-          if (p0 + j < t.parts) { u.x += a[j].x; u.y += a[j].y; u.z += a[j].z; u.w += a[j].w; }
+        for (int q = 0; q < FLAT; ++q)
+          if (q >= j && q < j + t.parts) a[q] = __ldg((const float4*)(pp + (size_t)(q - j) * t.part_stride));
+        j += t.parts;
       }
-      v[i].x = fmaf(s.x * t.factor, u.x, v[i].x);
-      v[i].y = fmaf(s.y * t.factor, u.y, v[i].y);
-      v[i].z = fmaf(s.z * t.factor, u.z, v[i].z);
-      v[i].w = fmaf(s.w * t.factor, u.w, v[i].w);
+      j = 0;
+#pragma unroll
+      for (int k = 0; k < BRANCH_TERMS; ++k) {
+        if (k >= terms.n) break;
+        const BranchTerm& t = terms.t[k];
+        float4 s = make_float4(1.f, 1.f, 1.f, 1.f), u = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (t.scale) s = __ldg((const float4*)(t.scale + c));
+#pragma unroll
+        for (int q = 0; q < FLAT; ++q)
+          if (q >= j && q < j + t.parts) { u.x += a[q].x; u.y += a[q].y; u.z += a[q].z; u.w += a[q].w; }
+        j += t.parts;
+        branch_add(v[i], s, t.factor, u);
+      }
+    } else {
+      for (int k = 0; k < terms.n; ++k) {
+        const BranchTerm& t = terms.t[k];
+        const float* pp = t.p + (size_t)r * t.row_stride + c;
+        float4 s = make_float4(1.f, 1.f, 1.f, 1.f), u = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (t.scale) s = __ldg((const float4*)(t.scale + c));
+        for (int p0 = 0; p0 < t.parts; p0 += 8) {       // up to eight loads in flight
+          float4 a[8];
+#pragma unroll
+          for (int j = 0; j < 8; ++j)
+            if (p0 + j < t.parts) a[j] = __ldg((const float4*)(pp + (size_t)(p0 + j) * t.part_stride));
+#pragma unroll
+          for (int j = 0; j < 8; ++j)
+            if (p0 + j < t.parts) { u.x += a[j].x; u.y += a[j].y; u.z += a[j].z; u.w += a[j].w; }
+        }
+        branch_add(v[i], s, t.factor, u);
+      }
     }
     if (CONCAT) {
       TO* yr = y + (size_t)r * 2 * H + c;
       store4<TO>(yr, v[i]);
-      store4<TO>(yr + H, *(const float4*)(x0 + (size_t)r * H + c));
+      store4<TO>(yr + H, embedding4(emb, row0 + c));
       *(float4*)(xr + c) = make_float4(wv[i][0], wv[i][1], wv[i][2], wv[i][3]);
     } else {
       if (terms.n > 0) *(float4*)(xr + c) = v[i];
@@ -562,10 +616,11 @@ template <typename TO, bool CONCAT>
 __global__ void __launch_bounds__(256)
 branch_kernel(float* __restrict__ x, const __grid_constant__ BranchTerms terms,
               const void* __restrict__ w, int w_bf16, float eps, TO* __restrict__ y,
-              const float* __restrict__ x0, int H) {
+              const __grid_constant__ Embedding emb, int H) {
   mb_grid_wait();
   mb_grid_launch_next();
   __shared__ float red[33];
+  const size_t row0 = CONCAT ? embedding_row(emb, blockIdx.x, H) : 0;
   const int r = blockIdx.x;
   float* xr = x + (size_t)r * H;
   float sum = 0.f;
@@ -578,7 +633,9 @@ branch_kernel(float* __restrict__ x, const __grid_constant__ BranchTerms terms,
     }
     if (CONCAT) {
       y[(size_t)r * 2 * H + c] = from_f32<TO>(v);
-      y[(size_t)r * 2 * H + H + c] = from_f32<TO>(x0[(size_t)r * H + c]);
+      const float e = emb.bf16 ? __bfloat162float(((const __nv_bfloat16*)emb.table)[row0 + c])
+                               : ((const float*)emb.table)[row0 + c];
+      y[(size_t)r * 2 * H + H + c] = from_f32<TO>(e * emb.scale);
       xr[c] = ((const float*)w)[c];
     } else {
       if (terms.n > 0) xr[c] = v;
@@ -596,17 +653,21 @@ branch_kernel(float* __restrict__ x, const __grid_constant__ BranchTerms terms,
 
 template <typename TO, bool CONCAT>
 static int branch_launch(float* x, const BranchTerms& terms, const void* w, int w_bf16, float eps,
-                         void* y, const float* x0, int R, int H, cudaStream_t s) {
-  uintptr_t bits = (uintptr_t)x | (uintptr_t)w | (uintptr_t)y | (uintptr_t)x0;
+                         void* y, const Embedding& emb, int R, int H, cudaStream_t s) {
+  uintptr_t bits = (uintptr_t)x | (uintptr_t)w | (uintptr_t)y | (uintptr_t)emb.table;
   long long strides = 0;
   for (int k = 0; k < terms.n; ++k) {
     bits |= (uintptr_t)terms.t[k].p | (uintptr_t)terms.t[k].scale;
     strides |= terms.t[k].part_stride | terms.t[k].row_stride;
   }
   if (H % 4 == 0 && H <= 4 * 1024 * 4 && (bits & 15) == 0 && (strides & 3) == 0) {
+#define BR_GO_F(V_, T_, F_)                                                                  \
+  mb_launch(branch_vec_kernel<TO, V_, T_, F_, CONCAT>, dim3(R), dim3(T_), 0, s, x, terms, w, \
+            w_bf16, eps, (TO*)y, emb, H)
 #define BR_GO(V_, T_)                                                                        \
-  mb_launch(branch_vec_kernel<TO, V_, T_, CONCAT>, dim3(R), dim3(T_), 0, s, x, terms, w,     \
-            w_bf16, eps, (TO*)y, x0, H)
+  if (terms.parts <= 2) BR_GO_F(V_, T_, 2);                                                  \
+  else if (terms.parts <= BRANCH_FLAT) BR_GO_F(V_, T_, BRANCH_FLAT);                         \
+  else BR_GO_F(V_, T_, 0)
     if ((R <= 256 && H > 1024) || H > 4 * 256 * 4) {
       const int vec = (H + 4 * 1024 - 1) / (4 * 1024);
       if (vec <= 1) { BR_GO(1, 1024); }
@@ -619,10 +680,11 @@ static int branch_launch(float* x, const BranchTerms& terms, const void* w, int 
       else { BR_GO(4, 256); }
     }
 #undef BR_GO
+#undef BR_GO_F
     return 0;
   }
   mb_launch(branch_kernel<TO, CONCAT>, dim3(R), dim3(256), 0, s, x, terms, w, w_bf16, eps, (TO*)y,
-            x0, H);
+            emb, H);
   return 0;
 }
 
@@ -632,6 +694,7 @@ static bool branch_terms(const BranchTerm* list, int n, BranchTerms* out) {
   for (int k = 0; k < n; ++k) {
     if (list[k].p == nullptr || list[k].parts < 1) return false;
     out->t[k] = list[k];
+    out->parts += list[k].parts;
   }
   out->n = n;
   return true;
@@ -645,21 +708,23 @@ MB_EXPORT int mb_branch_norm(float* x, const BranchTerm* list, int n, const void
   if (y != nullptr && w == nullptr) MB_FAIL("mb_branch_norm: a norm without weights");
   cudaStream_t s = (cudaStream_t)stream;
   if (y_dtype == MB_F32)
-    branch_launch<float, false>(x, terms, w, w_dtype == MB_BF16, eps, y, nullptr, R, H, s);
+    branch_launch<float, false>(x, terms, w, w_dtype == MB_BF16, eps, y, Embedding{}, R, H, s);
   else
-    branch_launch<__nv_bfloat16, false>(x, terms, w, w_dtype == MB_BF16, eps, y, nullptr, R, H, s);
+    branch_launch<__nv_bfloat16, false>(x, terms, w, w_dtype == MB_BF16, eps, y, Embedding{}, R, H, s);
   MB_CHECK_LAUNCH("mb_branch_norm");
 }
 
-MB_EXPORT int mb_pass_concat(float* x, const BranchTerm* list, int n, const float* x0,
+MB_EXPORT int mb_pass_concat(float* x, const BranchTerm* list, int n, const void* table,
+                             int t_dtype, int rows, const int* ids, float emb_scale,
                              const float* vector, void* y, int y_dtype, int R, int H,
                              void* stream) {
   if (R <= 0) return 0;
   BranchTerms terms;
   if (!branch_terms(list, n, &terms)) MB_FAIL("mb_pass_concat: %d terms", n);
   cudaStream_t s = (cudaStream_t)stream;
-  if (y_dtype == MB_F32) branch_launch<float, true>(x, terms, vector, 0, 0.f, y, x0, R, H, s);
-  else branch_launch<__nv_bfloat16, true>(x, terms, vector, 0, 0.f, y, x0, R, H, s);
+  const Embedding emb = {table, ids, t_dtype == MB_BF16, rows, emb_scale};
+  if (y_dtype == MB_F32) branch_launch<float, true>(x, terms, vector, 0, 0.f, y, emb, R, H, s);
+  else branch_launch<__nv_bfloat16, true>(x, terms, vector, 0, 0.f, y, emb, R, H, s);
   MB_CHECK_LAUNCH("mb_pass_concat");
 }
 

@@ -17,6 +17,7 @@
 // to run; no result depends on it (a row's sums are formed alone, in a fixed order).
 #include "common.cuh"
 #include "mma_tile.cuh"
+#include "moe_act.cuh"
 
 MB_DEFINE_LAST_ERROR
 
@@ -315,40 +316,6 @@ MB_EXPORT int mb_moe_route_plan(const float* z, int ldz, int parts, long long pa
 }
 
 // ------------------------------------------------------------------ the experts' products
-// act(gate) * up. 0: SiLU; 1: the tanh form of GELU; 2: the clamped form
-// g' = min(g, limit), u' = clamp(u, -limit, limit), g' sigmoid(1.702 g') (u' + 1).
-__device__ __forceinline__ float moe_gated(float z, float u, int act, float limit) {
-  if (act == 2) {
-    z = fminf(z, limit);
-    u = fminf(fmaxf(u, -limit), limit);
-    return z / (1.0f + expf(-1.702f * z)) * (u + 1.0f);
-  }
-  if (act == 1)
-    return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z))) * u;
-  return z / (1.0f + expf(-z)) * u;
-}
-
-// An activation of one input, for experts without a gate (the codes of the elementwise kernels).
-// 0: SiLU; 1: the tanh form of GELU; 3: the square of relu.
-__device__ __forceinline__ float moe_plain(float z, int act) {
-  if (act == 3) {
-    z = fmaxf(z, 0.f);
-    return z * z;
-  }
-  if (act == 1)
-    return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
-  return z / (1.0f + expf(-z));
-}
-
-// What a product of the experts is: the second one, the first with gate and up rows, or the first
-// of experts without a gate (W [E][N][K]).
-enum { MOE_DOWN = 0, MOE_GATED_UP = 1, MOE_PLAIN_UP = 2 };
-
-template <int MODE>
-__device__ __forceinline__ float moe_act(float z, float u, int act, float limit) {
-  return MODE == MOE_GATED_UP ? moe_gated(z, u, act, limit) : moe_plain(z, act);
-}
-
 #define MG_BN 64
 #define MG_BK 16
 // UP:   in = h [T, K] (row of list row r: perm[r] / top), W [E][2N][K] (gate rows, then up

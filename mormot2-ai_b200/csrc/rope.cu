@@ -601,6 +601,105 @@ maps_norm_rope_store_kernel(const TI* __restrict__ rows, int parts, size_t part_
   }
 }
 
+// The same for steps of many tokens, with 16-byte accesses: bfloat16 rows, maps of 64 or 128 values
+// that rotate as a whole, value rows that are whole multiples of a map's size (taken as that
+// many vectors). HD / 16 neighbouring lanes share a vector, each holds eight neighbouring values
+// of the first half and their rotation partners of the second half; a warp works on 512 / HD
+// vectors at once, takes up to QK_PASSES such groups of its token and forms the angles once.
+template <int HD>
+__global__ void __launch_bounds__(QK_WARPS * 32)
+maps_wide_kernel(const __nv_bfloat16* __restrict__ rows, int ld, const float* __restrict__ bias,
+                 const float* __restrict__ q_norm, const float* __restrict__ k_norm, float eps,
+                 const float* __restrict__ inv_freq, float amp, const int* __restrict__ tok_slot,
+                 const int* __restrict__ tok_pos, const int* __restrict__ page_table,
+                 int max_pages, int ring_pages, __nv_bfloat16* __restrict__ kpool,
+                 __nv_bfloat16* __restrict__ vpool, __nv_bfloat16* __restrict__ q_out, int nh,
+                 int nkv, int maps, int vd) {
+  constexpr int HALF = HD / 2, L = HALF / 8, HPP = 32 / L;  // lanes a vector, vectors a group
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int sl = lane % L, hl = lane / L;
+  const int t = blockIdx.x;
+  const int nq = nh * maps, nk = nkv * maps, per_v = vd / HD, total = nq + nk + nkv * per_v;
+  const int pos = tok_pos[t], slot = tok_slot[t];
+  const int group0 = (blockIdx.y * QK_WARPS + warp) * QK_PASSES;
+  // ahead of the wait: the angles (each lane that holds the same columns of another vector forms
+  // 8 / HPP of the eight sines and cosines and hands them round)
+  float cs[8], sn[8];
+  {
+    constexpr int PER = 8 / HPP > 0 ? 8 / HPP : 1;
+    float my_sn[PER], my_cs[PER];
+#pragma unroll
+    for (int r = 0; r < PER; ++r) {
+      const int f = 8 * sl + (hl * PER + r) % 8;
+      sincosf(inv_freq[f] * (float)pos, &my_sn[r], &my_cs[r]);
+    }
+#pragma unroll
+    for (int j = 0; j < 8; ++j) {
+      sn[j] = amp * __shfl_sync(0xffffffffu, my_sn[j % PER], (j / PER) * L + sl);
+      cs[j] = amp * __shfl_sync(0xffffffffu, my_cs[j % PER], (j / PER) * L + sl);
+    }
+  }
+  mb_grid_wait();
+  mb_grid_launch_next();
+  uint4 raw[QK_PASSES][2];       // every group's values are asked for before the first is worked on
+#pragma unroll
+  for (int i = 0; i < QK_PASSES; ++i) {
+    const int n = (group0 + i) * HPP + hl;
+    raw[i][0] = raw[i][1] = make_uint4(0u, 0u, 0u, 0u);
+    if (n < total) {
+      const __nv_bfloat16* src = rows + (size_t)t * ld + (size_t)n * HD + 8 * sl;
+      raw[i][0] = *reinterpret_cast<const uint4*>(src);
+      raw[i][1] = *reinterpret_cast<const uint4*>(src + HALF);
+    }
+  }
+#pragma unroll
+  for (int i = 0; i < QK_PASSES; ++i) {
+    const int n0 = (group0 + i) * HPP, n = n0 + hl;
+    if (n0 >= total) break;  // the whole warp
+    const bool live = n < total, is_q = n < nq, is_k = !is_q && n < nq + nk;
+    float a[8], b[8];
+    unpack8(raw[i][0], a);
+    unpack8(raw[i][1], b);
+    if (bias && live) {
+      const float* bp = bias + (size_t)n * HD + 8 * sl;
+#pragma unroll
+      for (int j = 0; j < 8; j += 4) {
+        const float4 x = __ldg((const float4*)(bp + j)), y = __ldg((const float4*)(bp + HALF + j));
+        a[j] += x.x; a[j + 1] += x.y; a[j + 2] += x.z; a[j + 3] += x.w;
+        b[j] += y.x; b[j + 1] += y.y; b[j + 2] += y.z; b[j + 3] += y.w;
+      }
+    }
+    if (n0 < nq + nk) {  // some vector of this group is a query or key (uniform over the warp)
+      float sum = 0.f;
+#pragma unroll
+      for (int j = 0; j < 8; ++j) sum = fmaf(a[j], a[j], fmaf(b[j], b[j], sum));
+#pragma unroll
+      for (int o = L / 2; o > 0; o >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
+      if (is_q || is_k) {
+        const float* w = (is_q ? q_norm : k_norm) + 8 * sl;
+        const float inv = 1.0f / sqrtf(sum / (float)HD + eps);
+#pragma unroll
+        for (int j = 0; j < 8; ++j) {
+          const float x = __ldg(w + j) * (a[j] * inv), y = __ldg(w + HALF + j) * (b[j] * inv);
+          a[j] = x * cs[j] - y * sn[j];
+          b[j] = y * cs[j] + x * sn[j];
+        }
+      }
+    }
+    if (!live) continue;
+    __nv_bfloat16* dst;
+    if (is_q) {
+      dst = q_out + ((size_t)t * nq + n) * HD;
+    } else {
+      const int m = is_k ? n - nq : n - nq - nk, per = is_k ? maps : per_v, g = m / per;
+      const size_t row = kv_row(page_table, max_pages, ring_pages, slot, pos, nkv, g);
+      dst = (is_k ? kpool : vpool) + (row * per + (m - g * per)) * HD;
+    }
+    *reinterpret_cast<uint4*>(dst + 8 * sl) = pack8(a);
+    *reinterpret_cast<uint4*>(dst + 8 * sl + HALF) = pack8(b);
+  }
+}
+
 MB_EXPORT int mb_maps_norm_rope_store(const void* rows, int in_dtype, int parts,
                                       long long part_stride, int ld, const float* bias,
                                       const float* q_norm, const float* k_norm, float eps,
@@ -625,6 +724,22 @@ MB_EXPORT int mb_maps_norm_rope_store(const void* rows, int in_dtype, int parts,
   const int most = (pairs ? 64 : 32) * MP_MAX;
   if (dim <= 0 || vd <= 0 || dim > most || vd > most)
     MB_FAIL("mb_maps_norm_rope_store: vectors of %d and %d values (at most %d)", dim, vd, most);
+  if (T >= 128 && in_dtype == MB_BF16 && dtype == MB_BF16 && parts == 1 &&
+      (dim == 64 || dim == 128) && rot_dim == dim && vd % dim == 0 && ld % 8 == 0 &&
+      (((uintptr_t)rows | (uintptr_t)kpool | (uintptr_t)vpool | (uintptr_t)q_out |
+        (uintptr_t)bias) & 15) == 0) {
+    typedef __nv_bfloat16 bf;
+    const int vectors = (nh + nkv) * maps + nkv * (vd / dim), each = QK_WARPS * QK_PASSES * (512 / dim);
+    dim3 wide(T, (vectors + each - 1) / each);
+#define GOW(HD_)                                                                               \
+  mb_launch(maps_wide_kernel<HD_>, wide, dim3(QK_WARPS * 32), 0, (cudaStream_t)stream,         \
+            (const bf*)rows, ld, bias, q_norm, k_norm, eps, inv_freq, amp, tok_slot, tok_pos,  \
+            page_table, max_pages, ring_pages, (bf*)kpool, (bf*)vpool, (bf*)q_out, nh, nkv,    \
+            maps, vd)
+    if (dim == 64) GOW(64); else GOW(128);
+#undef GOW
+    MB_CHECK_LAUNCH("mb_maps_norm_rope_store");
+  }
   const size_t smem = (size_t)(rot_dim + MP_WARPS * dim) * sizeof(float);
   const int total = (nh + nkv) * maps + nkv;
   // few tokens: a vector a warp; many: four a warp, so that a block's angles serve sixteen

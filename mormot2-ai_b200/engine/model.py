@@ -142,7 +142,7 @@ class DecoderModel:
             if i in self.entries:
                 entry = self.entries[i]
                 if getattr(entry, "accepts_pending", False):
-                    pending = entry.forward(x, x0, pending=pending)
+                    pending = entry.forward(x, step, self.embedding, pending=pending)
                 else:
                     if pending is not None:
                         settle(x, pending)

@@ -74,6 +74,7 @@ CLASS_OF = {"mb_gemm_tc": "products", "mb_gemm_simt": "products",
             "mb_latent_attention_mma": "attention",
             "mb_moe_route": "routing", "mb_moe_plan": "routing", "mb_moe_route_plan": "routing", "mb_moe_gemm": "products",
             "mb_moe_combine": "routing", "mb_moe_table_plan": "routing",
+            "mb_moe_gather": "routing", "mb_moe_gemm_tc": "products",
             "mb_branch_norm": "norms", "mb_pass_concat": "norms",
             "mb_maps_norm_rope_store": "rotary", "mb_attention_diff": "attention",
             "mb_attention_diff_decode": "attention", "mb_attention_diff_prefill": "attention",
@@ -440,19 +441,22 @@ def branch_norm(x: torch.Tensor, terms, w: Optional[torch.Tensor] = None, eps: f
           float(eps), _ptr(out), code_of(out.dtype) if out is not None else F32, T, H, _stream())
 
 
-def pass_concat(x: torch.Tensor, terms, x0: torch.Tensor, vector: torch.Tensor,
-                both: torch.Tensor) -> None:
-    """both[t] = [x[t] + the terms (as in ``branch_norm``) ; x0[t]] in both's type, and then
-    x[t] = vector."""
+def pass_concat(x: torch.Tensor, terms, table: torch.Tensor, ids: torch.Tensor, scale: float,
+                vector: torch.Tensor, both: torch.Tensor) -> None:
+    """both[t] = [x[t] + the terms (as in ``branch_norm``) ; table[ids[t]] * scale] in both's
+    type, and then x[t] = vector."""
     T, H = x.shape
-    assert x.dtype == x0.dtype == vector.dtype == torch.float32 and x0.shape == x.shape
-    assert both.shape == (T, 2 * H) and vector.numel() == H
-    for t, what in ((x, "x"), (x0, "x0"), (vector, "the pass's vector"), (both, "the rows")):
+    assert x.dtype == vector.dtype == torch.float32 and ids.dtype == torch.int32
+    assert both.shape == (T, 2 * H) and vector.numel() == H and ids.numel() == T
+    assert table.shape[1] == H
+    for t, what in ((x, "x"), (table, "the embedding"), (vector, "the pass's vector"),
+                    (both, "the rows")):
         _contig(t, what)
     arr, n = _branch_terms(terms, T, H)
-    _call("elementwise", "mb_pass_concat", [_vp, _vp, _i, _vp, _vp, _vp, _i, _i, _i, _vp],
-          _ptr(x), _c.cast(arr, _vp), n, _ptr(x0), _ptr(vector), _ptr(both),
-          code_of(both.dtype), T, H, _stream())
+    _call("elementwise", "mb_pass_concat",
+          [_vp, _vp, _i, _vp, _i, _i, _vp, _f, _vp, _vp, _i, _i, _i, _vp],
+          _ptr(x), _c.cast(arr, _vp), n, _ptr(table), code_of(table.dtype), table.shape[0],
+          _ptr(ids), float(scale), _ptr(vector), _ptr(both), code_of(both.dtype), T, H, _stream())
 
 
 def wide_qk_norm(qkv: torch.Tensor, qw: int, kw: int, wq: torch.Tensor, wk: torch.Tensor,
@@ -910,6 +914,36 @@ def moe_gemm(src: torch.Tensor, w: torch.Tensor, out: torch.Tensor, plan: torch.
           assignments, E, max_tiles, bm, top, N, Kd, (1 if gated else 2) if up else 0, act,
           _ptr(weight),
           float(limit), _stream())
+
+
+def moe_gather(src: torch.Tensor, plan: torch.Tensor, assignments: int, experts: int, top: int,
+               out: torch.Tensor) -> None:
+    """out[r] = src[perm[r] / top]: the rows of ``src`` [T, K] in the order of the plan's lists."""
+    _contig(src, "src"), _contig(out, "out")
+    assert src.dtype == out.dtype == torch.bfloat16 and out.shape == (assignments, src.shape[1])
+    _call("moe_tc", "mb_moe_gather", [_vp, _vp, _i, _i, _i, _i, _vp, _vp],
+          _ptr(src), _ptr(plan), assignments, experts, top, src.shape[1], _ptr(out), _stream())
+
+
+def moe_gemm_tc(rows: torch.Tensor, w: torch.Tensor, out: torch.Tensor, plan: torch.Tensor,
+                max_tiles: int, up: bool, sms: int, error: torch.Tensor, act: int = ACT_SILU,
+                weight: Optional[torch.Tensor] = None, limit: float = 0.0,
+                gated: bool = True) -> None:
+    """``moe_gemm`` on tcgen05 (bfloat16, a plan in tiles of 128 rows, N and K multiples of 8);
+    ``rows`` [A, K] are in list order for the first product too (``moe_gather``)."""
+    E = w.shape[0]
+    N, Kd = w.shape[1] // (2 if up and gated else 1), w.shape[2]
+    A = rows.shape[0]
+    _contig(rows, "rows"), _contig(out, "out"), _contig(w, "the experts' weight")
+    assert rows.shape[1] == Kd and out.shape == (A, N)
+    assert rows.dtype == w.dtype == torch.bfloat16
+    assert out.dtype == (torch.bfloat16 if up else torch.float32)
+    assert weight is None or weight.dtype == torch.float32
+    _call("moe_tc", "mb_moe_gemm_tc",
+          [_vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _vp, _f, _i, _vp, _vp],
+          _ptr(rows), _ptr(w), _ptr(out), _ptr(plan), A, E, max_tiles, N, Kd,
+          (1 if gated else 2) if up else 0, act, _ptr(weight), float(limit), sms, _ptr(error),
+          _stream())
 
 
 def moe_combine(x: torch.Tensor, y: torch.Tensor, top: int, shared: Optional[torch.Tensor],

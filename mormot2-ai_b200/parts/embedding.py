@@ -93,9 +93,9 @@ class PassProjection(Part):
     """What a pass through looped layers starts from: x = W_in [x ; x0] + step[row], x0 the
     embedding's output (``names``: ``in`` [size, 2 size], x's columns first, and ``step`` [rows,
     size]). One kernel adds what is still pending into x, writes [x ; x0] in the activation type
-    and puts step[row] in x's place; the product is added onto that."""
+    (x0 from the embedding's table) and puts step[row] in x's place; the product is added onto
+    that."""
     capturable = True
-    add_embedding = True        # the model keeps a copy of the embedding's output
     accepts_pending = True      # forward(..., pending=) -> what is pending afterwards
 
     def __init__(self, spec, prefix: str = ""):
@@ -113,13 +113,14 @@ class PassProjection(Part):
         self.linear = Linear(weights[self.names["in"]], rt)
         self.vector = weights[self.names["step"]][self.row].to(torch.float32).contiguous()
 
-    def forward(self, x: torch.Tensor, x0, pending=None):
+    def forward(self, x: torch.Tensor, step, embedding, pending=None):
         from .block import BranchSums, settle
         if pending is not None and not isinstance(pending, BranchSums):
             settle(x, pending)
             pending = None
         both = torch.empty((x.shape[0], 2 * self.size), dtype=self.rt.dtype, device=x.device)
-        K.pass_concat(x, pending.terms if pending is not None else [], x0, self.vector, both)
+        K.pass_concat(x, pending.terms if pending is not None else [], embedding.table,
+                      step.tok_ids, embedding.scale, self.vector, both)
         y = self.linear(both, out_dtype=torch.float32, defer="any")
         return BranchSums([(y.partial if isinstance(y, Pending) else y, 1.0, None)])
 

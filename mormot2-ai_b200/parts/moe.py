@@ -52,6 +52,27 @@ def tile_rows(rt, w_up, T: int, A: int, E: int, hidden: int, inter: int) -> int:
     return 128 if fast else (64 if A > 16 * E else 16)
 
 
+def expert_products(rt, h, w_up, w_down, plan, bm: int, max_tiles: int, top: int, act: int,
+                    gated: bool = True, limit: float = 0.0, weight=None):
+    """Both products of the chosen experts over a step's lists: y [T * top, hidden] float32, the
+    row of assignment t * top + k times ``weight`` (None: one)."""
+    A, dev = h.shape[0] * top, h.device
+    inter = w_down.shape[2]
+    mid = torch.empty((A, inter), dtype=rt.dtype, device=dev)
+    y = torch.empty((A, w_down.shape[1]), dtype=torch.float32, device=dev)
+    if bm == 128:       # the tcgen05 kernel, whose tiles are rows that lie one after the other
+        rows = torch.empty((A, h.shape[1]), dtype=h.dtype, device=dev)
+        K.moe_gather(h, plan, A, w_up.shape[0], top, rows)
+        K.moe_gemm_tc(rows, w_up, mid, plan, max_tiles, True, rt.sms, rt.error_word, act,
+                      gated=gated, limit=limit)
+        K.moe_gemm_tc(mid, w_down, y, plan, max_tiles, False, rt.sms, rt.error_word,
+                      weight=weight)
+    else:
+        K.moe_gemm(h, w_up, mid, plan, A, max_tiles, bm, top, True, act, limit=limit, gated=gated)
+        K.moe_gemm(mid, w_down, y, plan, A, max_tiles, bm, top, False, act, weight)
+    return y
+
+
 class RoutedExperts(Part):
     capturable = True
 
@@ -99,7 +120,7 @@ class RoutedExperts(Part):
         self.probe = None
 
     def libraries(self, rt) -> List[str]:
-        return ["moe"]
+        return ["moe"] + (["moe_tc"] if rt.fast_kernels else [])
 
     can_store = True      # forward(..., store=True) writes its output into x instead of adding
 
@@ -184,11 +205,8 @@ class RoutedExperts(Part):
             K.moe_plan(ids, E, bm, max_tiles, plan)
         if self.probe is not None:
             self.probe(self, step, ids)
-        act = torch.empty((A, self.inter), dtype=self.rt.dtype, device=dev)
-        K.moe_gemm(h, self.w_up, act, plan, A, max_tiles, bm, top, True, self.act,
-                   limit=self.limit)
-        y = torch.empty((A, self.hidden), dtype=torch.float32, device=dev)
-        K.moe_gemm(act, self.w_down, y, plan, A, max_tiles, bm, top, False, self.act, w)
+        y = expert_products(self.rt, h, self.w_up, self.w_down, plan, bm, max_tiles, top, self.act,
+                            limit=self.limit, weight=w)
         shared = None
         if self.shared_size:
             if self.shared_fused:
@@ -225,9 +243,11 @@ class TableExperts(Part):
         self.n_expert = [prefix + names["expert"].format(e) for e in range(self.experts)]
         self.n_shared = prefix + names["shared"]
         self.up, self.down = names["up"], names["down"]
+        # for measurements: as ``RoutedExperts.probe``, once for all runs of the layer in a pass
+        self.probe = None
 
     def libraries(self, rt) -> List[str]:
-        return ["moe"]
+        return ["moe"] + (["moe_tc"] if rt.fast_kernels else [])
 
     def tensors(self) -> List[TensorNeed]:
         out = [TensorNeed(self.n_table, (self.vocab, self.top), "choices", choices=self.experts)]
@@ -275,6 +295,8 @@ class TableExperts(Part):
             max_tiles = (A + bm - 1) // bm + self.experts
             plan = torch.empty((2 + self.experts + A + 2 * max_tiles,), dtype=torch.int32,
                                device=self.table.device)
+            if self.probe is not None:
+                self.probe(self, step, self.table[step.tok_ids.long()])
             K.moe_table_plan(self.table, step.tok_ids, self.experts, bm, max_tiles, plan)
             have = step.memo[id(self)] = (bm, max_tiles, plan)
         return have
@@ -282,14 +304,10 @@ class TableExperts(Part):
     def forward_terms(self, h, step):
         """The output as terms [(y, factor)]: the experts' rows as one part per choice, and the
         shared expert's product."""
-        T, dev = h.shape[0], h.device
-        A = T * self.top
+        T = h.shape[0]
         bm, max_tiles, plan = self.plan(step, T)
-        act = torch.empty((A, self.inter), dtype=self.rt.dtype, device=dev)
-        K.moe_gemm(h, self.w_up, act, plan, A, max_tiles, bm, self.top, True, self.act,
-                   gated=False)
-        y = torch.empty((A, self.hidden), dtype=torch.float32, device=dev)
-        K.moe_gemm(act, self.w_down, y, plan, A, max_tiles, bm, self.top, False, self.act)
+        y = expert_products(self.rt, h, self.w_up, self.w_down, plan, bm, max_tiles, self.top,
+                            self.act, gated=False)
         # row t * top + k is token t's k-th choice
         terms = [(y.view(T, self.top, self.hidden).transpose(0, 1), 1.0 / self.top)]
         if self.shared_size:
