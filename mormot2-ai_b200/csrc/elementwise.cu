@@ -668,7 +668,8 @@ static int branch_launch(float* x, const BranchTerms& terms, const void* w, int 
   if (terms.parts <= 2) BR_GO_F(V_, T_, 2);                                                  \
   else if (terms.parts <= BRANCH_FLAT) BR_GO_F(V_, T_, BRANCH_FLAT);                         \
   else BR_GO_F(V_, T_, 0)
-    if ((R <= 256 && H > 1024) || H > 4 * 256 * 4) {
+    // (a row's terms also take wide blocks: fewer registers a thread, more loads in flight)
+    if (((R <= 256 || terms.parts > 0) && H > 1024) || H > 4 * 256 * 4) {
       const int vec = (H + 4 * 1024 - 1) / (4 * 1024);
       if (vec <= 1) { BR_GO(1, 1024); }
       else if (vec <= 2) { BR_GO(2, 1024); }
