@@ -64,7 +64,7 @@ EXTRA_HEADERS = {"gemm_tc": ["tc_common.cuh"],
                  "attention_tc": ["attention_tc.cuh", "tc_common.cuh"],
                  "attention_diff_tc": ["attention_tc.cuh", "tc_common.cuh"],
                  "latent": ["mma_common.cuh", "mma_tile.cuh"],
-                 "moe": ["mma_common.cuh", "mma_tile.cuh", "moe_act.cuh"],
+                 "moe": ["mma_common.cuh", "moe_act.cuh"],
                  "moe_tc": ["tc_common.cuh", "moe_act.cuh"],
                  "latent_mma": ["mma_common.cuh"]}
 

@@ -6,17 +6,21 @@
 //   moe_route    per token: the `top` largest router logits (the lower index on a tie), their
 //                weights = softmax over the chosen logits only, and the shared expert's gate
 //                sigmoid(logit) when the router's product carries that column
-//   moe_plan     assignments (token, k) listed expert by expert, cut into tiles of rows
+//   moe_plan     assignments (token, k) listed expert by expert, cut into tiles of rows (the
+//                choices come from the router, or from a table by token id)
 //   moe_gemm     for every tile the product with its expert's weight:
 //                up:   act[r, :] = f(h[token(r)] · Wgᵀ) * (h[token(r)] · Wuᵀ)   (rows gathered)
 //                down: y[a(r), :] = weight[a(r)] * (act[r] · Wdᵀ)              (float32, scattered
 //                      to the assignment's own row, so the sum below has a fixed order)
 //   moe_combine  x[t] += sum_k y[t·top + k] + gate[t] · shared[t]
 //
+// Experts may have no gate: act[r, :] = f(h[token(r)] · Wuᵀ). In bfloat16 the products of a step
+// of more than 8 tokens are moe_tc.cu's.
+//
 // The order of an expert's rows in its list comes from atomic counters and may differ from run
 // to run; no result depends on it (a row's sums are formed alone, in a fixed order).
 #include "common.cuh"
-#include "mma_tile.cuh"
+#include "mma_common.cuh"
 #include "moe_act.cuh"
 
 MB_DEFINE_LAST_ERROR
@@ -411,56 +415,6 @@ moe_gemm_kernel(const T* __restrict__ in, const TW* __restrict__ W, void* __rest
   }
 }
 
-// The same two products on the tensor cores for bfloat16 operands (mma_tile.cuh); the plan's
-// tiles have 128 rows. The first product multiplies the gathered rows with the gate and the up
-// rows of the expert at once.
-template <int MODE>
-__global__ void __launch_bounds__(MT_THREADS)
-moe_gemm_mma_kernel(const __nv_bfloat16* __restrict__ in, const __nv_bfloat16* __restrict__ W,
-                    void* __restrict__ out, const int* __restrict__ plan, int A, int E,
-                    int max_tiles, int top, int N, int K, int act,
-                    const float* __restrict__ weight, float limit) {
-  mb_grid_wait();
-  mb_grid_launch_next();
-  constexpr bool UP = MODE != MOE_DOWN;
-  constexpr int NB = MODE == MOE_GATED_UP ? 2 : 1;
-  constexpr int MT_BN = 128 / NB;
-  const int tile = blockIdx.y;
-  if (tile >= plan[0]) return;
-  const int* offsets = plan + 1;
-  const int* perm = offsets + E + 1;
-  const int e = perm[A + tile];
-  const int r0 = perm[A + max_tiles + tile];
-  const int rows = min(MT_BM, offsets[e + 1] - r0);
-  __shared__ __align__(16) MtShared<NB> sh;
-  __shared__ int src[MT_BM];
-  if (threadIdx.x < MT_BM) {
-    const int r = threadIdx.x;
-    const int a = r < rows ? perm[r0 + r] : -1;
-    src[r] = a;
-    sh.a_rows[r] = a < 0 ? nullptr : in + (UP ? (size_t)(a / top) : (size_t)(r0 + r)) * K;
-  }
-  __syncthreads();
-  const int n0 = blockIdx.x * MT_BN;
-  const __nv_bfloat16* We = W + (size_t)e * NB * N * K;
-  const __nv_bfloat16* b[NB];
-#pragma unroll
-  for (int nb = 0; nb < NB; ++nb) b[nb] = We + ((size_t)nb * N + n0) * K;
-  float acc[NB][2][8 / NB][4];
-  mt_mainloop<NB>(sh, b, min(MT_BN, N - n0), K, acc);
-  mt_for_each<NB>([&](int r, int c, int mi, int ni, int el) {
-    const int gn = n0 + c;
-    if (r >= rows || gn >= N) return;
-    if (UP) {
-      ((__nv_bfloat16*)out)[(size_t)(r0 + r) * N + gn] =
-          __float2bfloat16_rn(moe_act<MODE>(acc[0][mi][ni][el], acc[NB - 1][mi][ni][el], act, limit));
-    } else {
-      const int a = src[r];
-      ((float*)out)[(size_t)a * N + gn] = (weight ? weight[a] : 1.0f) * acc[0][mi][ni][el];
-    }
-  });
-}
-
 // The two products for a decode step of at most eight tokens (tiles of at most 8 rows, so an
 // expert's weights are streamed exactly once): the WEIGHT rows are the 16 rows of the m16n8k16
 // product and the tile's tokens its 8 columns. A warp owns 16 output features (for the first
@@ -562,7 +516,7 @@ MB_EXPORT int mb_moe_gemm(const void* in, int dtype, const void* W, int w_dtype,
                           const int* plan, int A, int E, int max_tiles, int bm, int top, int N,
                           int K, int up, int act, const float* weight, float limit, void* stream) {
   if (A <= 0) return 0;
-  if (bm != 8 && bm != 16 && bm != 64 && bm != 128) MB_FAIL("mb_moe_gemm: tiles of %d rows", bm);
+  if (bm != 8 && bm != 16 && bm != 64) MB_FAIL("mb_moe_gemm: tiles of %d rows", bm);
   if (up < 0 || up > 2) MB_FAIL("mb_moe_gemm: product %d", up);
   if (up == MOE_PLAIN_UP && act != 0 && act != 1 && act != 3)
     MB_FAIL("mb_moe_gemm: activation %d of one input", act);
@@ -591,24 +545,6 @@ MB_EXPORT int mb_moe_gemm(const void* in, int dtype, const void* W, int w_dtype,
     else if (up == MOE_PLAIN_UP) GO8(MOE_PLAIN_UP)
     else GO8(MOE_DOWN)
 #undef GO8
-    MB_CHECK_LAUNCH("mb_moe_gemm");
-  }
-  if (bm == 128) {
-    if (!(dtype == MB_BF16 && w_dtype == MB_BF16 && K % 8 == 0 &&
-          (((uintptr_t)in | (uintptr_t)W) & 15) == 0))
-      MB_FAIL("mb_moe_gemm: tiles of 128 rows are the tensor-core kernel's (bfloat16, K %% 8 == 0)");
-    if (up == MOE_GATED_UP)
-      mb_launch(moe_gemm_mma_kernel<MOE_GATED_UP>, dim3((N + 63) / 64, max_tiles),
-                dim3(MT_THREADS), 0, s, (const __nv_bfloat16*)in, (const __nv_bfloat16*)W, out,
-                plan, A, E, max_tiles, top, N, K, act, weight, limit);
-    else if (up == MOE_PLAIN_UP)
-      mb_launch(moe_gemm_mma_kernel<MOE_PLAIN_UP>, dim3((N + 127) / 128, max_tiles),
-                dim3(MT_THREADS), 0, s, (const __nv_bfloat16*)in, (const __nv_bfloat16*)W, out,
-                plan, A, E, max_tiles, top, N, K, act, weight, limit);
-    else
-      mb_launch(moe_gemm_mma_kernel<MOE_DOWN>, dim3((N + 127) / 128, max_tiles), dim3(MT_THREADS), 0,
-                s, (const __nv_bfloat16*)in, (const __nv_bfloat16*)W, out, plan, A, E, max_tiles,
-                top, N, K, act, weight, limit);
     MB_CHECK_LAUNCH("mb_moe_gemm");
   }
 #define GO(T_, TW_, BM_, M_)                                                                 \

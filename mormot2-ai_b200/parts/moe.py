@@ -43,9 +43,9 @@ def _sums(result):
 
 
 def tile_rows(rt, w_up, T: int, A: int, E: int, hidden: int, inter: int) -> int:
-    """Rows per tile of an expert's list: 128 where the tensor-core kernel runs (bfloat16; 8
-    for a decode step of at most 8 tokens, the form that reads weights into registers), else
-    64, or 16 while an expert has few rows, so that few multiply-adds are wasted."""
+    """Rows per tile of an expert's list: 128 where the tcgen05 kernel runs (bfloat16; 8 for a
+    decode step of at most 8 tokens, the form that reads weights into registers), else 64, or
+    16 while an expert has few rows, so that few multiply-adds are wasted."""
     fast = rt.fast_kernels and w_up.dtype == torch.bfloat16 and hidden % 8 == 0 and inter % 8 == 0
     if fast and T <= 8 and hidden % 32 == 0 and inter % 32 == 0:
         return 8        # a decode step: no expert has more rows, its weights stream once
