@@ -5,7 +5,7 @@ Qwen3 dense decoder: everything between a request's token ids and its next token
 """
 from . import parts  # registers the built-in parts
 from .config import (ModelSpec, PartSpec, Qwen3Config, BusavikConfig, FimudraConfig, SezopelConfig, LaralixConfig,
-                     LotiraxConfig, Run, LayerSpec, architectures,
+                     LotiraxConfig, TenusunConfig, Run, LayerSpec, architectures,
                      config_of_folder, register_architecture)
 from .errors import CacheError, ConfigError, InferError, KernelError, WeightsError
 from .weights import SafeTensorsFolder, write_random_model, write_safetensors
@@ -14,7 +14,7 @@ from .sampling import Sampling, sampling_from_config
 from .client import LlmClient
 
 __all__ = ["ModelSpec", "PartSpec", "Qwen3Config", "BusavikConfig", "FimudraConfig", "SezopelConfig", "LaralixConfig",
-           "LotiraxConfig", "Run", "LayerSpec", "architectures",
+           "LotiraxConfig", "TenusunConfig", "Run", "LayerSpec", "architectures",
            "config_of_folder", "register_architecture", "CacheError", "ConfigError",
            "InferError", "KernelError", "WeightsError", "SafeTensorsFolder",
            "write_random_model", "write_safetensors", "DecoderModel", "Engine", "Entry",

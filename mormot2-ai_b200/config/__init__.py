@@ -6,6 +6,7 @@ from .fimudra import FimudraConfig
 from .sezopel import SezopelConfig
 from .laralix import LaralixConfig
 from .lotirax import LotiraxConfig
+from .tenusun import TenusunConfig
 from .registry import (architectures, config_of_folder, family_of, read_config_json,
                        register_architecture)
 
@@ -15,8 +16,9 @@ register_architecture(FimudraConfig, FimudraConfig.ARCHITECTURE, FimudraConfig.M
 register_architecture(SezopelConfig, SezopelConfig.ARCHITECTURE, SezopelConfig.MODEL_TYPE)
 register_architecture(LaralixConfig, LaralixConfig.ARCHITECTURE, LaralixConfig.MODEL_TYPE)
 register_architecture(LotiraxConfig, LotiraxConfig.ARCHITECTURE, LotiraxConfig.MODEL_TYPE)
+register_architecture(TenusunConfig, TenusunConfig.ARCHITECTURE, TenusunConfig.MODEL_TYPE)
 
 __all__ = ["LayerSpec", "ModelSpec", "PartSpec", "Run", "Qwen3Config", "BusavikConfig", "FimudraConfig", "SezopelConfig", "LaralixConfig",
-           "LotiraxConfig",
+           "LotiraxConfig", "TenusunConfig",
            "architectures",
            "config_of_folder", "family_of", "read_config_json", "register_architecture"]

@@ -1,5 +1,8 @@
 // Attention over the paged cache on the tensor cores (bfloat16 storage, float32 softmax and
-// accumulation), for head sizes 64 and 128.
+// accumulation), for query/key sizes and value sizes that are multiples of 8 up to 128. Sizes of
+// 64 and 128 are compile-time constants (EXACT); others are rounded up to DB and VB inside the
+// kernels: the queries' missing values are zeros, and output columns beyond a value row are not
+// stored.
 //
 // Decode (`mb_attention_decode`, `mb_attention_decode_clusters`): one new token per sequence.
 // The query heads that share a KV head are the 16 rows of the m16n8k16 MMA, so the keys and
@@ -19,8 +22,9 @@
 //
 // Every kernel takes a cap on the scores (`softcap` > 0: s <- c tanh(s / c) after the scale, a
 // template parameter of the kernels so that models without one run the code they ran before)
-// and a gate (`gate` not null: head h of token t at gate[t * gate_stride + h], a logit whose
-// sigmoid multiplies the head's output where it is written).
+// and a gate (`gate` not null): logits whose sigmoid multiplies the output where it is written,
+// one for a head (head h of token t at gate[t * gate_stride + h]) or, with `gate_dim` > 0, one
+// for every value (value d of the head at gate[t * gate_stride + h * gate_dim + d]).
 #include "attention_mma.cuh"
 
 MB_DEFINE_LAST_ERROR
@@ -35,9 +39,22 @@ template <bool CAP>
 __device__ __forceinline__ float score_log2(float s, float pre, float cap_log2) {
   return CAP ? cap_log2 * tanh_of_2xlog2e(s * pre) : s * pre;
 }
-__device__ __forceinline__ float gate_of(const bf16* gate, int gate_stride, int t, int h) {
-  return gate == nullptr ? 1.0f
-                         : sigmoid_f32(__bfloat162float(gate[(size_t)t * gate_stride + h]));
+__device__ __forceinline__ float gate_of(const bf16* gate, int gate_stride, int gate_dim, int t,
+                                         int h, int d) {
+  if (gate == nullptr) return 1.0f;
+  const size_t at = (size_t)t * gate_stride + (gate_dim > 0 ? h * gate_dim + d : h);
+  return sigmoid_f32(__bfloat162float(gate[at]));
+}
+// eight neighbouring outputs times the sigmoid of their logits
+__device__ __forceinline__ void gate8(const bf16* g, float* v) {
+  const uint4 raw = ldg16(g);
+  const uint32_t w[4] = {raw.x, raw.y, raw.z, raw.w};
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    const float2 f = __bfloat1622float2(*(const __nv_bfloat162*)&w[i]);
+    v[2 * i] *= sigmoid_f32(f.x);
+    v[2 * i + 1] *= sigmoid_f32(f.y);
+  }
 }
 
 // scores of one page: sc[u][e] = q(row) · k(key) for the keys u*8 + 2c + (e & 1) of the page and
@@ -90,23 +107,34 @@ __device__ __forceinline__ void pv_page(const float sc[8][4], const bf16* vbase,
 }
 
 // q fragments of the rows r and r + 8 (null: a row that is not there): 8 consecutive dims per
-// 32-dim chunk and thread
+// 32-dim chunk and thread; dims from `dim` on are zeros
 template <int HD>
-__device__ __forceinline__ void load_q(const bf16* q0, const bf16* q1, int c, uint4* qa, uint4* qb) {
+__device__ __forceinline__ void load_q(const bf16* q0, const bf16* q1, int c, uint4* qa, uint4* qb,
+                                       int dim) {
 #pragma unroll
   for (int ch = 0; ch < HD / 32; ++ch) {
-    qa[ch] = q0 ? ldg16(q0 + ch * 32 + c * 8) : make_uint4(0, 0, 0, 0);
-    qb[ch] = q1 ? ldg16(q1 + ch * 32 + c * 8) : make_uint4(0, 0, 0, 0);
+    const bool in = ch * 32 + c * 8 < dim;
+    qa[ch] = q0 && in ? ldg16(q0 + ch * 32 + c * 8) : make_uint4(0, 0, 0, 0);
+    qb[ch] = q1 && in ? ldg16(q1 + ch * 32 + c * 8) : make_uint4(0, 0, 0, 0);
   }
 }
 
 #define DEC_STAGES 3
+#define DEC_SLACK 128    // behind the last tile: what a rounded-up value row reads beyond its end
+
+// Shared memory of the decode kernel ahead of its barriers: the stages' tiles, over which the
+// warps' results and the CTA's own are laid afterwards.
+__host__ __device__ constexpr size_t decode_room(int dim, int vd, int VB) {
+  const size_t tiles = (size_t)DEC_STAGES * MB_PAGE * (dim + vd) * 2 + (vd < VB ? DEC_SLACK : 0);
+  const size_t merge = (size_t)(DEC_WARPS + 1) * 16 * VB * 4 + (DEC_WARPS + 1) * 32 * 4;
+  return tiles > merge ? tiles : merge;
+}
 
 // One CTA per (token, KV head [x 16 query heads of its group], split). Warp 4 streams the
 // pages of this split (every `splits`-th page of the sequence) into shared memory, a whole K
 // tile and a whole V tile per page (16 KB each for heads of 128) by bulk asynchronous copies,
 // three pages ahead. Warps 0-3 take 16 keys of every page each.
-template <int HD, bool CAP>
+template <int DB, int VB, bool EXACT, bool CAP>
 __global__ void __launch_bounds__((DEC_WARPS + 1) * 32, 2)
 attn_decode_kernel(const bf16* __restrict__ q, int q_stride, const bf16* __restrict__ kpool,
                    const bf16* __restrict__ vpool, const int* __restrict__ page_table,
@@ -115,17 +143,19 @@ attn_decode_kernel(const bf16* __restrict__ q, int q_stride, const bf16* __restr
                    int nkv, int window, float scale_log2, float* __restrict__ part_o,
                    float* __restrict__ part_ml, bf16* __restrict__ out, int out_stride,
                    int in_clusters, int* __restrict__ error, const float* __restrict__ sink,
-                   float cap_log2, const bf16* __restrict__ gate, int gate_stride,
-                   const float* __restrict__ slopes, int keep_first) {
-  constexpr int CH = HD / 32;  // 32-dim chunks of q·k
-  constexpr int DB = HD / 64;  // 64-dim blocks of p·v
-  constexpr uint32_t TILE = MB_PAGE * HD * 2;  // bytes of a page's keys (or values)
+                   float cap_log2, const bf16* __restrict__ gate, int gate_stride, int gate_dim,
+                   const float* __restrict__ slopes, int keep_first, int dim_rt, int vd_rt) {
+  constexpr int CH = DB / 32;  // 32-dim chunks of q·k
+  constexpr int OB = VB / 64;  // 64-dim blocks of p·v
+  const int dim = EXACT ? DB : dim_rt, vd = EXACT ? VB : vd_rt;
+  // bytes of a page's keys and of its values
+  const uint32_t KTILE = MB_PAGE * dim * 2, VTILE = MB_PAGE * vd * 2, STAGE = KTILE + VTILE;
   MB_TRACE_BEGIN();
   extern __shared__ __align__(128) uint8_t dec_smem[];
   // [stages][K tile | V tile], then the barriers; after the loop the tiles' memory holds the
   // warps' partial results for the merge
   const uint32_t tiles = smem_u32(dec_smem);
-  const uint32_t bars = tiles + DEC_STAGES * 2 * TILE;
+  const uint32_t bars = tiles + (uint32_t)decode_room(dim, vd, VB);
   const uint32_t full0 = bars, empty0 = bars + 8 * DEC_STAGES;
 
   const int s = blockIdx.x, S = gridDim.x, t = blockIdx.z;
@@ -158,9 +188,9 @@ attn_decode_kernel(const bf16* __restrict__ q, int q_stride, const bf16* __restr
   __syncthreads();
 
   float m0 = -INFINITY, m1 = -INFINITY, l0 = 0.f, l1 = 0.f;
-  float o[DB][8][4];
+  float o[OB][8][4];
 #pragma unroll
-  for (int db = 0; db < DB; ++db)
+  for (int db = 0; db < OB; ++db)
 #pragma unroll
     for (int j = 0; j < 8; ++j)
 #pragma unroll
@@ -193,10 +223,10 @@ attn_decode_kernel(const bf16* __restrict__ q, int q_stride, const bf16* __restr
         }
         if (lane == 0) {
           mbar_wait(empty0 + 8 * st, ph ^ 1, error, 4);
-          mbar_expect_tx(full0 + 8 * st, 2 * TILE);
-          const size_t at = ((size_t)page * nkv + g) * MB_PAGE * HD;
-          bulk_copy(tiles + st * 2 * TILE, kpool + at, TILE, full0 + 8 * st);
-          bulk_copy(tiles + st * 2 * TILE + TILE, vpool + at, TILE, full0 + 8 * st);
+          mbar_expect_tx(full0 + 8 * st, STAGE);
+          const size_t at = ((size_t)page * nkv + g) * MB_PAGE;
+          bulk_copy(tiles + st * STAGE, kpool + at * dim, KTILE, full0 + 8 * st);
+          bulk_copy(tiles + st * STAGE + KTILE, vpool + at * vd, VTILE, full0 + 8 * st);
         }
         if (++st == DEC_STAGES) { st = 0; ph ^= 1; }
       }
@@ -207,9 +237,9 @@ attn_decode_kernel(const bf16* __restrict__ q, int q_stride, const bf16* __restr
     mb_grid_wait();  // q comes from the kernel before
     uint4 qa[CH], qb[CH];
     {
-      const bf16* qrow = q + (size_t)t * q_stride + (size_t)(h0 + r) * HD;
-      load_q<HD>(r < rows_valid ? qrow : nullptr, r + 8 < rows_valid ? qrow + 8 * HD : nullptr, c,
-                 qa, qb);
+      const bf16* qrow = q + (size_t)t * q_stride + (size_t)(h0 + r) * dim;
+      load_q<DB>(r < rows_valid ? qrow : nullptr, r + 8 < rows_valid ? qrow + 8 * dim : nullptr, c,
+                 qa, qb, dim);
     }
     // a bias that grows with the distance (in units of log2 e, as the scores are)
     const float sl0 = slopes && r < rows_valid ? slopes[h0 + r] * 1.4426950408889634f : 0.f;
@@ -219,13 +249,14 @@ attn_decode_kernel(const bf16* __restrict__ q, int q_stride, const bf16* __restr
     for (int i = 0; i < n_pages; ++i) {
       const int key0 = page_at(i) * MB_PAGE + 16 * warp;  // this warp's 16 keys
       mbar_wait(full0 + 8 * st, ph, error, 5);
-      const uint32_t ks = tiles + st * 2 * TILE + (uint32_t)(16 * warp) * HD * 2;
-      const uint32_t vs = ks + TILE;
+      // (a rounded-up row reads on into what follows it, whose values meet zeros of q)
+      const uint32_t ks = tiles + st * STAGE + (uint32_t)(16 * warp) * dim * 2;
+      const uint32_t vs = tiles + st * STAGE + KTILE + (uint32_t)(16 * warp) * vd * 2;
       float sc[2][4];
 #pragma unroll
       for (int u = 0; u < 2; ++u) {
         sc[u][0] = sc[u][1] = sc[u][2] = sc[u][3] = 0.f;
-        const uint32_t krow = ks + (uint32_t)(u * 8 + r) * HD * 2 + c * 16;
+        const uint32_t krow = ks + (uint32_t)(u * 8 + r) * dim * 2 + c * 16;
 #pragma unroll
         for (int ch = 0; ch < CH; ++ch) {
           const uint4 kb = lds16(krow + ch * 64);
@@ -271,15 +302,15 @@ attn_decode_kernel(const bf16* __restrict__ q, int q_stride, const bf16* __restr
       l1 = l1 * c1 + s1;
       const uint32_t a0 = pack_bf16(sc[0][0], sc[0][1]), a1 = pack_bf16(sc[0][2], sc[0][3]);
       const uint32_t a2 = pack_bf16(sc[1][0], sc[1][1]), a3 = pack_bf16(sc[1][2], sc[1][3]);
-      const uint32_t vrow = vs + (uint32_t)(2 * c) * HD * 2 + r * 16;
+      const uint32_t vrow = vs + (uint32_t)(2 * c) * vd * 2 + r * 16;
 #pragma unroll
-      for (int db = 0; db < DB; ++db) {
+      for (int db = 0; db < OB; ++db) {
         const uint4 va = lds16(vrow + db * 128);
-        const uint4 vb = lds16(vrow + HD * 2 + db * 128);
-        const uint4 vc = lds16(vrow + 8 * HD * 2 + db * 128);
-        const uint4 vd = lds16(vrow + 9 * HD * 2 + db * 128);
+        const uint4 vb = lds16(vrow + vd * 2 + db * 128);
+        const uint4 vc = lds16(vrow + 8 * vd * 2 + db * 128);
+        const uint4 ve = lds16(vrow + 9 * vd * 2 + db * 128);
         const uint32_t wa[4] = {va.x, va.y, va.z, va.w}, wb[4] = {vb.x, vb.y, vb.z, vb.w};
-        const uint32_t wc[4] = {vc.x, vc.y, vc.z, vc.w}, wd[4] = {vd.x, vd.y, vd.z, vd.w};
+        const uint32_t wc[4] = {vc.x, vc.y, vc.z, vc.w}, wd[4] = {ve.x, ve.y, ve.z, ve.w};
 #pragma unroll
         for (int j = 0; j < 8; ++j) {
           o[db][j][0] *= c0;
@@ -303,11 +334,11 @@ attn_decode_kernel(const bf16* __restrict__ q, int q_stride, const bf16* __restr
   }
   // every copy has landed and been read: the tiles' memory now holds the warps' results
   __syncthreads();
-  float* sm_o = (float*)dec_smem;                       // [DEC_WARPS][16][HD]
-  float* sm_m = sm_o + DEC_WARPS * 16 * HD;             // [DEC_WARPS][16]
+  float* sm_o = (float*)dec_smem;                       // [DEC_WARPS][16][VB]
+  float* sm_m = sm_o + DEC_WARPS * 16 * VB;             // [DEC_WARPS][16]
   float* sm_l = sm_m + DEC_WARPS * 16;                  // [DEC_WARPS][16]
-  float* sm_c = sm_l + DEC_WARPS * 16;                  // [16][HD] the CTA's own result
-  float* sm_cml = sm_c + 16 * HD;                       // [16] its maxima, [16] its sums
+  float* sm_c = sm_l + DEC_WARPS * 16;                  // [16][VB] the CTA's own result
+  float* sm_cml = sm_c + 16 * VB;                       // [16] its maxima, [16] its sums
   if (warp < DEC_WARPS) {
     if (c == 0) {
       sm_m[warp * 16 + r] = m0;
@@ -316,19 +347,19 @@ attn_decode_kernel(const bf16* __restrict__ q, int q_stride, const bf16* __restr
       sm_l[warp * 16 + r + 8] = l1;
     }
 #pragma unroll
-    for (int db = 0; db < DB; ++db)
+    for (int db = 0; db < OB; ++db)
 #pragma unroll
       for (int j = 0; j < 8; ++j) {
         const int d0 = db * 64 + (2 * c) * 8 + j, d1 = d0 + 8;
-        sm_o[(warp * 16 + r) * HD + d0] = o[db][j][0];
-        sm_o[(warp * 16 + r) * HD + d1] = o[db][j][1];
-        sm_o[(warp * 16 + r + 8) * HD + d0] = o[db][j][2];
-        sm_o[(warp * 16 + r + 8) * HD + d1] = o[db][j][3];
+        sm_o[(warp * 16 + r) * VB + d0] = o[db][j][0];
+        sm_o[(warp * 16 + r) * VB + d1] = o[db][j][1];
+        sm_o[(warp * 16 + r + 8) * VB + d0] = o[db][j][2];
+        sm_o[(warp * 16 + r + 8) * VB + d1] = o[db][j][3];
       }
   }
   __syncthreads();
-  for (int idx = threadIdx.x; idx < rows_valid * HD; idx += blockDim.x) {
-    const int row = idx / HD, d = idx - row * HD;
+  for (int idx = threadIdx.x; idx < rows_valid * vd; idx += blockDim.x) {
+    const int row = idx / vd, d = idx - row * vd;
     // a sink: one more term exp(sink[h]) in the denominator, counted once, by the first split
     const float sk = (sink != nullptr && s == 0) ? sink[h0 + row] * 1.4426950408889634f : -INFINITY;
     float M = sk;
@@ -341,21 +372,21 @@ attn_decode_kernel(const bf16* __restrict__ q, int q_stride, const bf16* __restr
       for (int w = 0; w < DEC_WARPS; ++w) {
         const float f = exp2f(sm_m[w * 16 + row] - M);  // 0 for a warp without keys
         L += sm_l[w * 16 + row] * f;
-        acc += sm_o[(w * 16 + row) * HD + d] * f;
+        acc += sm_o[(w * 16 + row) * VB + d] * f;
       }
     }
     if (!in_clusters) {  // through the caller's scratch: the merge kernel adds the splits up
       const size_t at = ((size_t)t * nh + h0 + row) * S + s;
-      part_o[at * HD + d] = acc;
+      part_o[at * vd + d] = acc;
       if (d == 0) {
         part_ml[at * 2] = M;
         part_ml[at * 2 + 1] = L;
       }
     } else if (S == 1) {
-      out[(size_t)t * out_stride + (size_t)(h0 + row) * HD + d] =
-          __float2bfloat16_rn(acc / L * gate_of(gate, gate_stride, t, h0 + row));
+      out[(size_t)t * out_stride + (size_t)(h0 + row) * vd + d] =
+          __float2bfloat16_rn(acc / L * gate_of(gate, gate_stride, gate_dim, t, h0 + row, d));
     } else {
-      sm_c[row * HD + d] = acc;
+      sm_c[row * VB + d] = acc;
       if (d == 0) {
         sm_cml[row] = M;
         sm_cml[16 + row] = L;
@@ -366,11 +397,11 @@ attn_decode_kernel(const bf16* __restrict__ q, int q_stride, const bf16* __restr
     // The splits of a (token, group) are the CTAs of one cluster: each adds up a share of the
     // outputs from all the CTAs' shared memory, in split order.
     cluster_sync_all();
-    const int total = rows_valid * HD, share = (total + S - 1) / S;
+    const int total = rows_valid * vd, share = (total + S - 1) / S;
     const int hi = min(total, (s + 1) * share);
     const uint32_t c_addr = smem_u32(sm_c), ml_addr = smem_u32(sm_cml);
     for (int idx = s * share + threadIdx.x; idx < hi; idx += blockDim.x) {
-      const int row = idx / HD, d = idx - row * HD;
+      const int row = idx / vd, d = idx - row * vd;
       float M = -INFINITY;
       for (int k = 0; k < S; ++k)
         M = fmaxf(M, ld_cluster_f32(cluster_addr_of(ml_addr + 4 * row, k)));
@@ -378,13 +409,13 @@ attn_decode_kernel(const bf16* __restrict__ q, int q_stride, const bf16* __restr
       for (int k = 0; k < S; ++k) {
         const float m = ld_cluster_f32(cluster_addr_of(ml_addr + 4 * row, k));
         const float l = ld_cluster_f32(cluster_addr_of(ml_addr + 4 * (16 + row), k));
-        const float v = ld_cluster_f32(cluster_addr_of(c_addr + 4 * (row * HD + d), k));
+        const float v = ld_cluster_f32(cluster_addr_of(c_addr + 4 * (row * VB + d), k));
         const float f = m == -INFINITY ? 0.f : exp2f(m - M);
         L += l * f;
         acc += v * f;
       }
-      out[(size_t)t * out_stride + (size_t)(h0 + row) * HD + d] =
-          __float2bfloat16_rn(acc / L * gate_of(gate, gate_stride, t, h0 + row));
+      out[(size_t)t * out_stride + (size_t)(h0 + row) * vd + d] =
+          __float2bfloat16_rn(acc / L * gate_of(gate, gate_stride, gate_dim, t, h0 + row, d));
     }
     cluster_sync_all();  // no CTA leaves while another may still read its shared memory
   }
@@ -392,11 +423,10 @@ attn_decode_kernel(const bf16* __restrict__ q, int q_stride, const bf16* __restr
 }
 
 // out[t, h, :] = sum_s o_s 2^(m_s - M) / sum_s l_s 2^(m_s - M), the splits in order
-template <int HD>
 __global__ void attn_merge_kernel(const float* __restrict__ part_o,
                                   const float* __restrict__ part_ml, int S, bf16* __restrict__ out,
                                   int out_stride, int nh, const bf16* __restrict__ gate,
-                                  int gate_stride) {
+                                  int gate_stride, int gate_dim, int vd) {
   mb_grid_wait();
   mb_grid_launch_next();
   const int t = blockIdx.x, h = blockIdx.y, d = threadIdx.x;
@@ -409,21 +439,26 @@ __global__ void attn_merge_kernel(const float* __restrict__ part_o,
     if (m == -INFINITY) continue;
     const float f = exp2f(m - M);
     L += part_ml[(at + s) * 2 + 1] * f;
-    acc += part_o[(at + s) * HD + d] * f;
+    acc += part_o[(at + s) * vd + d] * f;
   }
-  out[(size_t)t * out_stride + (size_t)h * HD + d] =
-      __float2bfloat16_rn(acc / L * gate_of(gate, gate_stride, t, h));
+  out[(size_t)t * out_stride + (size_t)h * vd + d] =
+      __float2bfloat16_rn(acc / L * gate_of(gate, gate_stride, gate_dim, t, h, d));
 }
 
-// floats of scratch that mb_attention_decode needs for T tokens
-MB_EXPORT long long mb_attention_decode_scratch(int T, int nh, int hd, int splits) {
-  return (long long)T * nh * splits * (hd + 2);
+// floats of scratch that mb_attention_decode needs for T tokens with value rows of `vd`
+MB_EXPORT long long mb_attention_decode_scratch(int T, int nh, int vd, int splits) {
+  return (long long)T * nh * splits * (vd + 2);
+}
+
+static bool head_sizes_ok(int hd, int vd) {
+  return hd > 0 && hd <= 128 && hd % 8 == 0 && vd > 0 && vd <= 128 && vd % 8 == 0;
 }
 
 static int decode_checks(const void* q, int q_stride, const void* kpool, const void* vpool, int T,
-                         int nh, int nkv, int hd, int splits) {
-  if (hd != 64 && hd != 128)
-    MB_FAIL("mb_attention_decode: heads of %d values are not supported (64 or 128)", hd);
+                         int nh, int nkv, int hd, int vd, int splits) {
+  if (!head_sizes_ok(hd, vd))
+    MB_FAIL("mb_attention_decode: heads of %d and %d values are not supported (multiples of 8, at "
+            "most 128)", hd, vd);
   if (nkv <= 0 || nh % nkv) MB_FAIL("mb_attention_decode: %d heads on %d KV heads", nh, nkv);
   if (splits <= 0 || splits > 65535) MB_FAIL("mb_attention_decode: %d splits", splits);
   if (((uintptr_t)kpool & 15) || ((uintptr_t)vpool & 15))
@@ -434,6 +469,20 @@ static int decode_checks(const void* q, int q_stride, const void* kpool, const v
   return 0;
 }
 
+// GO for the kernel's sizes: 64 and 128 as they are, others rounded up
+#define HEAD_SIZES_CAP(CAP_)                                                                   \
+  if (hd == 128 && vd == 128) GO(128, 128, true, CAP_)                                         \
+  else if (hd == 64 && vd == 64) GO(64, 64, true, CAP_)                                        \
+  else if (hd <= 64 && vd <= 64) GO(64, 64, false, CAP_)                                       \
+  else if (vd <= 64) GO(128, 64, false, CAP_)                                                  \
+  else GO(128, 128, false, CAP_)
+#define HEAD_SIZES                                                                             \
+  if (softcap > 0.f) {                                                                         \
+    HEAD_SIZES_CAP(true)                                                                       \
+  } else {                                                                                     \
+    HEAD_SIZES_CAP(false)                                                                      \
+  }
+
 // in_clusters: the splits of a (token, group) form a cluster and are merged through their
 // shared memory (no scratch, no second kernel); else through part_o / part_ml
 static int decode_launch(const void* q, int q_stride, void* out, int out_stride,
@@ -441,48 +490,45 @@ static int decode_launch(const void* q, int q_stride, void* out, int out_stride,
                          int max_pages, int ring_pages, const int* tok_slot, const int* tok_pos,
                          int T, int nh, int nkv, int hd, int window, float scale, int splits,
                          float* part_o, float* part_ml, int in_clusters, int* error,
-                         cudaStream_t s, const float* sink = nullptr, float softcap = 0.f,
-                         const void* gate = nullptr, int gate_stride = 0,
-                         const float* slopes = nullptr, int keep_first = 0) {
+                         cudaStream_t s, const float* sink, float softcap, const void* gate,
+                         int gate_stride, int gate_dim, const float* slopes, int keep_first,
+                         int vd) {
   const int G = nh / nkv, subs = (G + 15) / 16;
   const float log2e = 1.4426950408889634f;
   const float scale_log2 = softcap > 0.f ? 2.f * log2e * scale / softcap : scale * log2e;
   const float cap_log2 = softcap * log2e;
   dim3 grid(splits, nkv * subs, T), mgrid(T, nh);
-#define GO(HD_, CAP_)                                                                          \
+#define GO(D_, V_, X_, CAP_)                                                                   \
   {                                                                                            \
-    constexpr int smem = DEC_STAGES * 2 * MB_PAGE * HD_ * 2 + 64;                              \
+    const int smem = (int)decode_room(hd, vd, V_) + 64;                                        \
     static bool configured = false;                                                            \
     if (!configured) {                                                                         \
-      cudaError_t e = cudaFuncSetAttribute(attn_decode_kernel<HD_, CAP_>,                      \
-                                           cudaFuncAttributeMaxDynamicSharedMemorySize, smem); \
+      cudaError_t e = cudaFuncSetAttribute(attn_decode_kernel<D_, V_, X_, CAP_>,               \
+                                           cudaFuncAttributeMaxDynamicSharedMemorySize,        \
+                                           (int)decode_room(D_, V_, V_) + DEC_SLACK + 64);     \
       if (e != cudaSuccess) MB_FAIL("mb_attention_decode: %s", cudaGetErrorString(e));         \
       configured = true;                                                                       \
     }                                                                                          \
     if (in_clusters && splits > 1) {                                                           \
-      mb_launch_clusters(attn_decode_kernel<HD_, CAP_>, grid, dim3((DEC_WARPS + 1) * 32),      \
+      mb_launch_clusters(attn_decode_kernel<D_, V_, X_, CAP_>, grid, dim3((DEC_WARPS + 1) * 32), \
                          smem, s, splits, (const bf16*)q, q_stride, (const bf16*)kpool,        \
                          (const bf16*)vpool, page_table, max_pages, ring_pages, tok_slot,      \
                          tok_pos, nh, nkv, window, scale_log2, part_o, part_ml, (bf16*)out,    \
                          out_stride, 1, error, sink, cap_log2, (const bf16*)gate, gate_stride, \
-                         slopes, keep_first);                                                  \
+                         gate_dim, slopes, keep_first, hd, vd);                                \
     } else {                                                                                   \
-      mb_launch(attn_decode_kernel<HD_, CAP_>, grid, dim3((DEC_WARPS + 1) * 32), smem, s,      \
+      mb_launch(attn_decode_kernel<D_, V_, X_, CAP_>, grid, dim3((DEC_WARPS + 1) * 32), smem, s, \
                 (const bf16*)q, q_stride, (const bf16*)kpool, (const bf16*)vpool, page_table,  \
                 max_pages, ring_pages, tok_slot, tok_pos, nh, nkv, window, scale_log2, part_o, \
                 part_ml, (bf16*)out, out_stride, in_clusters, error, sink, cap_log2,           \
-                (const bf16*)gate, gate_stride, slopes, keep_first);                           \
+                (const bf16*)gate, gate_stride, gate_dim, slopes, keep_first, hd, vd);         \
       if (!in_clusters)                                                                        \
-        mb_launch(attn_merge_kernel<HD_>, mgrid, dim3(HD_), 0, s, (const float*)part_o,        \
+        mb_launch(attn_merge_kernel, mgrid, dim3(vd), 0, s, (const float*)part_o,              \
                   (const float*)part_ml, splits, (bf16*)out, out_stride, nh,                   \
-                  (const bf16*)gate, gate_stride);                                             \
+                  (const bf16*)gate, gate_stride, gate_dim, vd);                               \
     }                                                                                          \
   }
-  if (softcap > 0.f) {
-    if (hd == 64) GO(64, true) else GO(128, true)
-  } else {
-    if (hd == 64) GO(64, false) else GO(128, false)
-  }
+  HEAD_SIZES
 #undef GO
   MB_CHECK_LAUNCH("mb_attention_decode");
 }
@@ -501,17 +547,19 @@ MB_EXPORT int mb_attention_decode(const void* q, int q_stride, void* out, int ou
                                   int hd, int window, float scale, int splits, float* scratch,
                                   long long scratch_floats, int* error, const float* sink,
                                   float softcap, const void* gate, int gate_stride,
-                                  const float* slopes, int keep_first, void* stream) {
+                                  int gate_dim, const float* slopes, int keep_first, int vd,
+                                  void* stream) {
   if (T <= 0) return 0;
-  if (decode_checks(q, q_stride, kpool, vpool, T, nh, nkv, hd, splits)) return -1;
-  const long long need = mb_attention_decode_scratch(T, nh, hd, splits);
+  if (vd <= 0) vd = hd;
+  if (decode_checks(q, q_stride, kpool, vpool, T, nh, nkv, hd, vd, splits)) return -1;
+  const long long need = mb_attention_decode_scratch(T, nh, vd, splits);
   if (scratch == nullptr || scratch_floats < need)
     MB_FAIL("mb_attention_decode: %lld floats of scratch, %lld needed", scratch_floats, need);
   return decode_launch(q, q_stride, out, out_stride, kpool, vpool, page_table, max_pages,
                        ring_pages, tok_slot, tok_pos, T, nh, nkv, hd, window, scale, splits,
-                       scratch, scratch + (size_t)T * nh * splits * hd, 0, error,
-                       (cudaStream_t)stream, sink, softcap, gate, gate_stride, slopes,
-                       keep_first);
+                       scratch, scratch + (size_t)T * nh * splits * vd, 0, error,
+                       (cudaStream_t)stream, sink, softcap, gate, gate_stride, gate_dim, slopes,
+                       keep_first, vd);
 }
 
 // The same with the splits of a (token, group of heads) as the CTAs of one thread-block
@@ -526,9 +574,11 @@ MB_EXPORT int mb_attention_decode_clusters(const void* q, int q_stride, void* ou
                                            int nh, int nkv, int hd, int window, float scale,
                                            int splits, int* error, const float* sink,
                                            float softcap, const void* gate, int gate_stride,
-                                           const float* slopes, int keep_first, void* stream) {
+                                           int gate_dim, const float* slopes, int keep_first,
+                                           int vd, void* stream) {
   if (T <= 0) return 0;
-  if (decode_checks(q, q_stride, kpool, vpool, T, nh, nkv, hd, splits)) return -1;
+  if (vd <= 0) vd = hd;
+  if (decode_checks(q, q_stride, kpool, vpool, T, nh, nkv, hd, vd, splits)) return -1;
   if (splits > MB_DECODE_CLUSTER_SPLITS)
     MB_FAIL("mb_attention_decode_clusters: %d splits (a cluster holds at most %d)", splits,
             MB_DECODE_CLUSTER_SPLITS);
@@ -536,7 +586,7 @@ MB_EXPORT int mb_attention_decode_clusters(const void* q, int q_stride, void* ou
   return decode_launch(q, q_stride, out, out_stride, kpool, vpool, page_table, max_pages,
                        ring_pages, tok_slot, tok_pos, T, nh, nkv, hd, window, scale, splits,
                        nullptr, nullptr, 1, error, (cudaStream_t)stream, sink, softcap, gate,
-                       gate_stride, slopes, keep_first);
+                       gate_stride, gate_dim, slopes, keep_first, vd);
 }
 
 // ------------------------------------------------------------------ prefill
@@ -553,7 +603,7 @@ MB_EXPORT int mb_attention_decode_clusters(const void* q, int q_stride, void* ou
 // asynchronous copies, two pages ahead of the page in work. The rows of a tile are padded in
 // shared memory (keys to a pitch of 2 HD + 64 bytes, values to 2 HD + 16), which makes every
 // fragment read of qk_page_smem / pv_page_smem free of bank conflicts.
-template <int HD, bool CAP>
+template <int DB, int VB, bool EXACT, bool CAP>
 __global__ void __launch_bounds__(DEC_WARPS * 32, 2)
 attn_prefill_kernel(const bf16* __restrict__ q, int q_stride, bf16* __restrict__ out,
                     int out_stride, const bf16* __restrict__ kpool,
@@ -561,14 +611,15 @@ attn_prefill_kernel(const bf16* __restrict__ q, int q_stride, bf16* __restrict__
                     int max_pages, int ring_pages, const int* __restrict__ seq_start,
                     const int* __restrict__ seq_past, const int* __restrict__ seq_slot, int nh,
                     int nkv, int window, float scale_log2, const float* __restrict__ sink,
-                    float cap_log2, const bf16* __restrict__ gate, int gate_stride,
-                    const float* __restrict__ slopes, int keep_first) {
+                    float cap_log2, const bf16* __restrict__ gate, int gate_stride, int gate_dim,
+                    const float* __restrict__ slopes, int keep_first, int dim_rt, int vd_rt) {
   mb_grid_wait();
   mb_grid_launch_next();
-  constexpr int CH = HD / 32, DB = HD / 64;
-  constexpr int KP = HD * 2 + 64, VP = HD * 2 + 16;     // row pitches in bytes
+  constexpr int CH = DB / 32, OB = VB / 64;
+  constexpr int KP = DB * 2 + 64, VP = VB * 2 + 16;     // row pitches in bytes
   constexpr uint32_t STAGE = MB_PAGE * (KP + VP);
-  constexpr int CHUNKS = HD / 8;                        // 16-byte chunks of a row
+  const int dim = EXACT ? DB : dim_rt, vd = EXACT ? VB : vd_rt;
+  const int kch = dim / 8, vch = vd / 8;                // 16-byte chunks of a row
   extern __shared__ __align__(128) uint8_t pre_smem[];
   const uint32_t tiles = smem_u32(pre_smem);
 
@@ -590,6 +641,11 @@ attn_prefill_kernel(const bf16* __restrict__ q, int q_stride, bf16* __restrict__
   const int n_pages = kp + cta_last / MB_PAGE - page0 + 1;
   auto page_at = [&](int i) { return i < kp ? i : page0 + i - kp; };
 
+  if (!EXACT) {   // what rows are rounded up by stays zero
+    for (int e = threadIdx.x; e < (int)(PRE_STAGES * STAGE / 16); e += DEC_WARPS * 32)
+      *(uint4*)(pre_smem + 16 * e) = make_uint4(0, 0, 0, 0);
+    __syncthreads();
+  }
   auto issue = [&](int i) {  // page i of the CTA into stage i % PRE_STAGES
     if (i < n_pages) {
       const int p = page_at(i);
@@ -597,14 +653,19 @@ attn_prefill_kernel(const bf16* __restrict__ q, int q_stride, bf16* __restrict__
       int page = MB_INDEX_OK(entry < max_pages, 1, slot, p, max_pages)
                      ? page_table[(size_t)slot * max_pages + entry] : 0;
       if (!MB_INDEX_OK(page >= 0, 2, slot, entry, page)) page = 0;
-      const bf16* ksrc = kpool + ((size_t)page * nkv + g) * MB_PAGE * HD;
-      const bf16* vsrc = vpool + ((size_t)page * nkv + g) * MB_PAGE * HD;
-      const uint32_t kd = tiles + (i % PRE_STAGES) * STAGE, vd = kd + MB_PAGE * KP;
-      for (int e = threadIdx.x; e < MB_PAGE * CHUNKS; e += DEC_WARPS * 32) {
-        const int row = e / CHUNKS, ch = e % CHUNKS;
-        cp_async16(kd + row * KP + ch * 16, ksrc + row * HD + ch * 8);
-        cp_async16(vd + row * VP + ch * 16, vsrc + row * HD + ch * 8);
+      const bf16* ksrc = kpool + ((size_t)page * nkv + g) * MB_PAGE * dim;
+      const bf16* vsrc = vpool + ((size_t)page * nkv + g) * MB_PAGE * vd;
+      const uint32_t kd = tiles + (i % PRE_STAGES) * STAGE, vdst = kd + MB_PAGE * KP;
+      for (int e = threadIdx.x; e < MB_PAGE * kch; e += DEC_WARPS * 32) {
+        const int row = e / kch, ch = e - row * kch;
+        cp_async16(kd + row * KP + ch * 16, ksrc + row * dim + ch * 8);
+        if (EXACT && DB == VB) cp_async16(vdst + row * VP + ch * 16, vsrc + row * vd + ch * 8);
       }
+      if (!(EXACT && DB == VB))
+        for (int e = threadIdx.x; e < MB_PAGE * vch; e += DEC_WARPS * 32) {
+          const int row = e / vch, ch = e - row * vch;
+          cp_async16(vdst + row * VP + ch * 16, vsrc + row * vd + ch * 8);
+        }
     }
     cp_async_commit();
   };
@@ -624,8 +685,9 @@ attn_prefill_kernel(const bf16* __restrict__ q, int q_stride, bf16* __restrict__
 
   uint4 qa[CH], qb[CH];
   {
-    const bf16* qrow = q + (size_t)(start + ra) * q_stride + (size_t)h * HD;
-    load_q<HD>(has_a ? qrow : nullptr, has_b ? qrow + (size_t)8 * q_stride : nullptr, c, qa, qb);
+    const bf16* qrow = q + (size_t)(start + ra) * q_stride + (size_t)h * dim;
+    load_q<DB>(has_a ? qrow : nullptr, has_b ? qrow + (size_t)8 * q_stride : nullptr, c, qa, qb,
+               dim);
   }
   const float sl = slopes ? slopes[h] * 1.4426950408889634f : 0.f;   // the distance bias
   float m0 = -INFINITY, m1 = -INFINITY, l0 = 0.f, l1 = 0.f;
@@ -636,9 +698,9 @@ attn_prefill_kernel(const bf16* __restrict__ q, int q_stride, bf16* __restrict__
     m0 = m1 = sink[h] * 1.4426950408889634f;
     l0 = l1 = c == 0 ? 1.f : 0.f;
   }
-  float o[DB][8][4];
+  float o[OB][8][4];
 #pragma unroll
-  for (int db = 0; db < DB; ++db)
+  for (int db = 0; db < OB; ++db)
 #pragma unroll
     for (int j = 0; j < 8; ++j)
 #pragma unroll
@@ -655,7 +717,7 @@ attn_prefill_kernel(const bf16* __restrict__ q, int q_stride, bf16* __restrict__
       const uint32_t ks = tiles + (i % PRE_STAGES) * STAGE, vs = ks + MB_PAGE * KP;
       const int key0 = p * MB_PAGE;
       float sc[8][4];
-      qk_page_smem<HD, KP>(qa, qb, ks, r, c, sc);
+      qk_page_smem<DB, KP>(qa, qb, ks, r, c, sc);
       float mx0 = -INFINITY, mx1 = -INFINITY;
 #pragma unroll
       for (int u = 0; u < 8; ++u) {
@@ -698,7 +760,7 @@ attn_prefill_kernel(const bf16* __restrict__ q, int q_stride, bf16* __restrict__
       l0 = l0 * c0 + s0;
       l1 = l1 * c1 + s1;
 #pragma unroll
-      for (int db = 0; db < DB; ++db)
+      for (int db = 0; db < OB; ++db)
 #pragma unroll
         for (int j = 0; j < 8; ++j) {
           o[db][j][0] *= c0;
@@ -706,7 +768,7 @@ attn_prefill_kernel(const bf16* __restrict__ q, int q_stride, bf16* __restrict__
           o[db][j][2] *= c1;
           o[db][j][3] *= c1;
         }
-      pv_page_smem<HD, VP>(sc, vs, r, c, o);
+      pv_page_smem<VB, VP>(sc, vs, r, c, o);
     }
   }
   cp_async_wait<0>();
@@ -715,11 +777,40 @@ attn_prefill_kernel(const bf16* __restrict__ q, int q_stride, bf16* __restrict__
   l0 += __shfl_xor_sync(0xffffffffu, l0, 2);
   l1 += __shfl_xor_sync(0xffffffffu, l1, 1);
   l1 += __shfl_xor_sync(0xffffffffu, l1, 2);
-  const float i0 = (has_a ? gate_of(gate, gate_stride, start + ra, h) : 1.0f) / l0;
-  const float i1 = (has_b ? gate_of(gate, gate_stride, start + rb, h) : 1.0f) / l1;
+  const bool per_head = gate != nullptr && gate_dim == 0;
+  const float i0 = (per_head && has_a ? gate_of(gate, gate_stride, 0, start + ra, h, 0) : 1.0f) / l0;
+  const float i1 = (per_head && has_b ? gate_of(gate, gate_stride, 0, start + rb, h, 0) : 1.0f) / l1;
   // a thread holds the dims db*64 + 16c .. + 15 of its two rows
 #pragma unroll
-  for (int db = 0; db < DB; ++db) {
+  for (int db = 0; db < OB; ++db) {
+    const int d = db * 64 + 16 * c;
+    bf16* oa = out + (size_t)(start + ra) * out_stride + (size_t)h * vd + d;
+    bf16* ob = oa + (size_t)8 * out_stride;
+    if (gate_dim > 0) {   // a gate for every value: the outputs stay in float32 up to here
+      const bf16* ga = gate + (size_t)(start + ra) * gate_stride + (size_t)h * gate_dim + d;
+      const bf16* gb = ga + (size_t)8 * gate_stride;
+#pragma unroll
+      for (int half = 0; half < 2; ++half) {
+        if (d + 8 * half >= vd) continue;
+        float a[8], b[8];
+#pragma unroll
+        for (int j = 0; j < 8; ++j) {
+          a[j] = o[db][j][half] * i0;
+          b[j] = o[db][j][2 + half] * i1;
+        }
+        if (has_a) {
+          gate8(ga + 8 * half, a);
+          *(uint4*)(oa + 8 * half) = make_uint4(pack_bf16(a[0], a[1]), pack_bf16(a[2], a[3]),
+                                                pack_bf16(a[4], a[5]), pack_bf16(a[6], a[7]));
+        }
+        if (has_b) {
+          gate8(gb + 8 * half, b);
+          *(uint4*)(ob + 8 * half) = make_uint4(pack_bf16(b[0], b[1]), pack_bf16(b[2], b[3]),
+                                                pack_bf16(b[4], b[5]), pack_bf16(b[6], b[7]));
+        }
+      }
+      continue;
+    }
     uint32_t w[4][4];  // [row a lo, row a hi, row b lo, row b hi][4 registers of 2 bf16]
 #pragma unroll
     for (int j = 0; j < 8; j += 2) {
@@ -728,16 +819,10 @@ attn_prefill_kernel(const bf16* __restrict__ q, int q_stride, bf16* __restrict__
       w[2][j >> 1] = pack_bf16(o[db][j][2] * i1, o[db][j + 1][2] * i1);
       w[3][j >> 1] = pack_bf16(o[db][j][3] * i1, o[db][j + 1][3] * i1);
     }
-    if (has_a) {
-      uint4* dst = (uint4*)(out + (size_t)(start + ra) * out_stride + (size_t)h * HD + db * 64 + 16 * c);
-      dst[0] = make_uint4(w[0][0], w[0][1], w[0][2], w[0][3]);
-      dst[1] = make_uint4(w[1][0], w[1][1], w[1][2], w[1][3]);
-    }
-    if (has_b) {
-      uint4* dst = (uint4*)(out + (size_t)(start + rb) * out_stride + (size_t)h * HD + db * 64 + 16 * c);
-      dst[0] = make_uint4(w[2][0], w[2][1], w[2][2], w[2][3]);
-      dst[1] = make_uint4(w[3][0], w[3][1], w[3][2], w[3][3]);
-    }
+    if (has_a && d < vd) *(uint4*)oa = make_uint4(w[0][0], w[0][1], w[0][2], w[0][3]);
+    if (has_a && d + 8 < vd) *(uint4*)(oa + 8) = make_uint4(w[1][0], w[1][1], w[1][2], w[1][3]);
+    if (has_b && d < vd) *(uint4*)ob = make_uint4(w[2][0], w[2][1], w[2][2], w[2][3]);
+    if (has_b && d + 8 < vd) *(uint4*)(ob + 8) = make_uint4(w[3][0], w[3][1], w[3][2], w[3][3]);
   }
 }
 
@@ -750,11 +835,17 @@ MB_EXPORT int mb_attention_prefill(const void* q, int q_stride, void* out, int o
                                    const int* seq_past, const int* seq_slot, int B, int max_new,
                                    int nh, int nkv, int hd, int window, float scale, int* error,
                                    const float* sink, float softcap, const void* gate,
-                                   int gate_stride, const float* slopes, int keep_first,
-                                   void* stream) {
+                                   int gate_stride, int gate_dim, const float* slopes,
+                                   int keep_first, int vd, void* stream) {
   if (B <= 0 || max_new <= 0) return 0;
-  if (hd != 64 && hd != 128)
-    MB_FAIL("mb_attention_prefill: heads of %d values are not supported (64 or 128)", hd);
+  if (vd <= 0) vd = hd;
+  if (!head_sizes_ok(hd, vd))
+    MB_FAIL("mb_attention_prefill: heads of %d and %d values are not supported (multiples of 8, at "
+            "most 128)", hd, vd);
+  if (((uintptr_t)kpool & 15) || ((uintptr_t)vpool & 15))
+    MB_FAIL("mb_attention_prefill: the cache pools are not 16-byte aligned");
+  if (gate != nullptr && gate_dim > 0 && (((uintptr_t)gate & 15) || (gate_stride & 7) || gate_dim != vd))
+    MB_FAIL("mb_attention_prefill: the gate's rows are not 16-byte aligned (stride %d)", gate_stride);
   if (nkv <= 0 || nh % nkv) MB_FAIL("mb_attention_prefill: %d heads on %d KV heads", nh, nkv);
   if (((uintptr_t)q & 15) || (q_stride & 7) || ((uintptr_t)out & 15) || (out_stride & 7))
     MB_FAIL("mb_attention_prefill: q or out is not 16-byte aligned (strides %d, %d)", q_stride,
@@ -765,27 +856,23 @@ MB_EXPORT int mb_attention_prefill(const void* q, int q_stride, void* out, int o
   const float log2e = 1.4426950408889634f;
   const float scale_log2 = softcap > 0.f ? 2.f * log2e * scale / softcap : scale * log2e;
   const float cap_log2 = softcap * log2e;
-#define GO(HD_, CAP_)                                                                          \
+#define GO(D_, V_, X_, CAP_)                                                                   \
   {                                                                                            \
-    constexpr int smem = PRE_STAGES * MB_PAGE * (4 * HD_ + 80);                                \
+    constexpr int smem = PRE_STAGES * MB_PAGE * (2 * D_ + 2 * V_ + 80);                        \
     static bool configured = false;                                                            \
     if (!configured) {                                                                         \
-      cudaError_t e = cudaFuncSetAttribute(attn_prefill_kernel<HD_, CAP_>,                     \
+      cudaError_t e = cudaFuncSetAttribute(attn_prefill_kernel<D_, V_, X_, CAP_>,              \
                                            cudaFuncAttributeMaxDynamicSharedMemorySize, smem); \
       if (e != cudaSuccess) MB_FAIL("mb_attention_prefill: %s", cudaGetErrorString(e));        \
       configured = true;                                                                       \
     }                                                                                          \
-    mb_launch(attn_prefill_kernel<HD_, CAP_>, grid, dim3(DEC_WARPS * 32), smem, s,             \
+    mb_launch(attn_prefill_kernel<D_, V_, X_, CAP_>, grid, dim3(DEC_WARPS * 32), smem, s,      \
               (const bf16*)q, q_stride, (bf16*)out, out_stride, (const bf16*)kpool,            \
               (const bf16*)vpool, page_table, max_pages, ring_pages, seq_start, seq_past,      \
               seq_slot, nh, nkv, window, scale_log2, sink, cap_log2, (const bf16*)gate,        \
-              gate_stride, slopes, keep_first);                                                \
+              gate_stride, gate_dim, slopes, keep_first, hd, vd);                              \
   }
-  if (softcap > 0.f) {
-    if (hd == 64) GO(64, true) else GO(128, true)
-  } else {
-    if (hd == 64) GO(64, false) else GO(128, false)
-  }
+  HEAD_SIZES
 #undef GO
   (void)error;
   MB_CHECK_LAUNCH("mb_attention_prefill");
@@ -834,6 +921,6 @@ MB_EXPORT int mb_attention_decode_static(const void* q, int q_stride, void* out,
   return mb_attention_decode(q, q_stride, out, out_stride, kpool, vpool, page_table, max_pages,
                              ring_pages, tok_slot, tok_pos, T, nh, nkv, hd, window,
                              scale, splits, g_static_scratch_ptr[device],
-                             MB_ATTENTION_DECODE_STATIC_FLOATS, error, nullptr, 0.f, nullptr, 0,
-                             nullptr, 0, stream);
+                             MB_ATTENTION_DECODE_STATIC_FLOATS, error, nullptr, 0.f, nullptr, 0, 0,
+                             nullptr, 0, 0, stream);
 }

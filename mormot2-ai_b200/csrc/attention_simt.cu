@@ -25,7 +25,7 @@ attention_simt_kernel(const T* __restrict__ q, int q_stride, T* __restrict__ out
                       const int* __restrict__ tok_seq, const int* __restrict__ tok_pos,
                       const int* __restrict__ seq_slot, int nh, int nkv, int hd, int window,
                       float scale, int vd, const float* __restrict__ sink, float softcap,
-                      const T* __restrict__ gate, int gate_stride,
+                      const T* __restrict__ gate, int gate_stride, int gate_dim,
                       const float* __restrict__ slopes, int keep_first) {
   extern __shared__ __align__(16) float qs[];  // ATT_WARPS x hd
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -112,9 +112,18 @@ attention_simt_kernel(const T* __restrict__ q, int q_stride, T* __restrict__ out
     }
   }
   }
-  // a gate per head: the head's output times the sigmoid of the token's logit for this head
-  const float inv = (gate ? 1.0f / (1.0f + expf(-to_f32<T>(gate[(size_t)t * gate_stride + h])))
-                          : 1.0f) / l;
+  // a gate per head: the head's output times the sigmoid of the token's logit for this head;
+  // or one per value
+  const float inv = (gate && gate_dim == 0
+                         ? sigmoid_f32(to_f32<T>(gate[(size_t)t * gate_stride + h])) : 1.0f) / l;
+  if (gate && gate_dim > 0) {
+    const T* gp = gate + (size_t)t * gate_stride + (size_t)h * gate_dim;
+#pragma unroll
+    for (int d = 0; d < ATT_MAX_D; ++d) {
+      const int i = VEC ? 4 * lane + 128 * (d / 4) + d % 4 : lane + 32 * d;
+      if (i < vd) acc[d] *= sigmoid_f32(to_f32<T>(gp[i]));
+    }
+  }
   T* op = out + (size_t)t * out_stride + (size_t)h * vd;
   if (VEC) {
 #pragma unroll
@@ -146,7 +155,7 @@ attention_shared_kernel(const T* __restrict__ q, int q_stride, T* __restrict__ o
                         const int* __restrict__ tok_seq, const int* __restrict__ tok_pos,
                         const int* __restrict__ seq_slot, int nh, int nkv, int hd, int window,
                         float scale, int vd, const float* __restrict__ sink, float softcap,
-                        const T* __restrict__ gate, int gate_stride,
+                        const T* __restrict__ gate, int gate_stride, int gate_dim,
                         const float* __restrict__ slopes, int keep_first) {
   extern __shared__ __align__(16) float sm[];
   const int pitch = hd + 4, pieces = hd / 4, vpitch = vd + 4, vpieces = vd / 4;
@@ -228,9 +237,18 @@ attention_shared_kernel(const T* __restrict__ q, int q_stride, T* __restrict__ o
     }
   }
   }
-  // a gate per head: the head's output times the sigmoid of the token's logit for this head
-  const float inv = (gate ? 1.0f / (1.0f + expf(-to_f32<T>(gate[(size_t)t * gate_stride + h])))
-                          : 1.0f) / l;
+  // a gate per head: the head's output times the sigmoid of the token's logit for this head;
+  // or one per value
+  const float inv = (gate && gate_dim == 0
+                         ? sigmoid_f32(to_f32<T>(gate[(size_t)t * gate_stride + h])) : 1.0f) / l;
+  if (gate && gate_dim > 0) {
+    const T* gp = gate + (size_t)t * gate_stride + (size_t)h * gate_dim;
+#pragma unroll
+    for (int d = 0; d < ATT_MAX_D; ++d) {
+      const int i = 4 * lane + 128 * (d / 4) + d % 4;
+      if (i < vd) acc[d] *= sigmoid_f32(to_f32<T>(gp[i]));
+    }
+  }
   T* op = out + (size_t)t * out_stride + (size_t)h * vd;
 #pragma unroll
   for (int d = 0; d < ATT_MAX_D / 4; ++d) {
@@ -246,7 +264,8 @@ attention_shared_kernel(const T* __restrict__ q, int q_stride, T* __restrict__ o
 // out + t * out_stride + h * vd. `vd`: the size of a value row (0: hd). `sink`: float32 [nh]
 // or null, one more term exp(sink[h]) in every softmax denominator of head h. `softcap` > 0:
 // every score s (after the scale) becomes softcap * tanh(s / softcap). `gate` (may be null):
-// head h's output of token t is multiplied by sigmoid(gate[t * gate_stride + h]). `slopes`:
+// head h's output of token t is multiplied by sigmoid(gate[t * gate_stride + h]), or, with
+// `gate_dim` > 0, its value d by sigmoid(gate[t * gate_stride + h * gate_dim + d]). `slopes`:
 // float32 [nh] or null: slopes[h] * (query's position - key's position) is taken off every
 // score of head h after the cap. `keep_first` > 0: with a window, the first keep_first
 // positions of a sequence stay visible to every later one.
@@ -256,7 +275,7 @@ MB_EXPORT int mb_attention_simt(const void* q, int q_stride, void* out, int out_
                                 const int* tok_seq, const int* tok_pos, const int* seq_slot,
                                 int T, int nh, int nkv, int hd, int window, float scale,
                                 int vd, const float* sink, float softcap, const void* gate,
-                                int gate_stride, const float* slopes, int keep_first,
+                                int gate_stride, int gate_dim, const float* slopes, int keep_first,
                                 void* stream) {
   if (T <= 0) return 0;
   if (vd <= 0) vd = hd;
@@ -286,7 +305,7 @@ MB_EXPORT int mb_attention_simt(const void* q, int q_stride, void* out, int out_
     attention_shared_kernel<T_><<<grid, ATT_WARPS * 32, shared, s>>>(                         \
         (const T_*)q, q_stride, (T_*)out, out_stride, (const T_*)kpool, (const T_*)vpool,     \
         page_table, max_pages, ring_pages, tok_seq, tok_pos, seq_slot, nh, nkv, hd, window,   \
-        scale, vd, sink, softcap, (const T_*)gate, gate_stride, slopes, keep_first);                                                             \
+        scale, vd, sink, softcap, (const T_*)gate, gate_stride, gate_dim, slopes, keep_first);                                                             \
   }
     if (dtype == MB_F32) GOS(float) else GOS(__nv_bfloat16)
 #undef GOS
@@ -296,7 +315,7 @@ MB_EXPORT int mb_attention_simt(const void* q, int q_stride, void* out, int out_
   attention_simt_kernel<T_, V_><<<grid, ATT_WARPS * 32, smem, s>>>(                           \
       (const T_*)q, q_stride, (T_*)out, out_stride, (const T_*)kpool, (const T_*)vpool,       \
       page_table, max_pages, ring_pages, tok_seq, tok_pos, seq_slot, nh, nkv, hd, window, scale, \
-      vd, sink, softcap, (const T_*)gate, gate_stride, slopes, keep_first)
+      vd, sink, softcap, (const T_*)gate, gate_stride, gate_dim, slopes, keep_first)
   if (dtype == MB_F32) {
     if (vec) GO(float, true); else GO(float, false);
   } else {

@@ -1,5 +1,5 @@
 // Causal prefill attention over the paged cache on the fifth-generation tensor cores, for
-// bfloat16 heads of 128 values: S = Q·Kᵀ and O += P·V are tcgen05.mma instructions with their
+// bfloat16 heads of 128 values (value rows of 128 or 64): S = Q·Kᵀ and O += P·V are tcgen05.mma instructions with their
 // accumulators in tensor memory, the tiles of Q, K and V come by TMA (128-byte swizzle), the
 // softmax runs in float32 on four warps that read S from tensor memory, one row a thread.
 //
@@ -9,7 +9,7 @@
 //               (K ahead of V: its stage is free again after the first product);
 //   warp 1      issues S = Q·Kᵀ (128 x 64) two pages ahead into one of two S buffers in tensor
 //               memory, and when P of a page is ready O += P·V (128 x 128) with P as the
-//               operand that lies in tensor memory;
+//               operand that lies in tensor memory (128 x 64 for value rows of 64);
 //   warps 2-5   read S, mask it (causal bound and window by position), keep the row maximum
 //               and sum, and write P = exp2(S - max) as bfloat16 over the S they have just read
 //               (the second product takes it from there), so that the softmax of a page never
@@ -34,16 +34,17 @@ typedef __nv_bfloat16 bf16;
 #define AT_V_STAGES 2
 #define AT_THREADS 192
 #define AT_Q_BYTES (AT_ROWS * AT_HD * 2)    // 32 KB: two 128 x 64 halves
-#define AT_KV_BYTES (MB_PAGE * AT_HD * 2)   // 16 KB: two 64 x 64 halves
+#define AT_KV_BYTES (MB_PAGE * AT_HD * 2)   // 16 KB: two 64 x 64 halves (a page's values: VD / 64)
 // no slack for alignment: two CTAs must fit in one SM; the kernel checks that its dynamic
 // shared memory starts on a 1024-byte boundary (it does when there is no static shared memory)
 #define AT_SMEM (AT_Q_BYTES + (AT_K_STAGES + AT_V_STAGES) * AT_KV_BYTES + 256)
 #define AT_TMEM_COLS 256                    // two S buffers of 64 columns, O: 128 columns
 
 // CAP: the scores are capped, s <- c tanh(s scale / c): `scale_log2` is then 2 log2(e) scale / c
-// and `cap_log2` = c log2(e). `gate` (may be null): head h of token t at
-// gate[t * gate_stride + h], a logit whose sigmoid multiplies the head's output.
-template <bool CAP>
+// and `cap_log2` = c log2(e). `gate` (may be null): logits whose sigmoid multiplies the output,
+// one for a head (head h of token t at gate[t * gate_stride + h]) or, with `gate_dim` > 0, one for
+// every value (at gate[t * gate_stride + h * gate_dim + d]). VD: the size of a value row.
+template <int VD, bool CAP>
 __global__ void __launch_bounds__(AT_THREADS, 2)
 attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ,
                        const __grid_constant__ CUtensorMap tmK,
@@ -53,7 +54,8 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ,
                        const int* __restrict__ seq_past, const int* __restrict__ seq_slot, int nh,
                        int nkv, int window, float scale_log2, int* __restrict__ error,
                        const float* __restrict__ sink, float cap_log2,
-                       const bf16* __restrict__ gate, int gate_stride) {
+                       const bf16* __restrict__ gate, int gate_stride, int gate_dim) {
+  constexpr int V_BYTES = MB_PAGE * VD * 2;
   extern __shared__ __align__(1024) uint8_t at_smem[];
   const uint32_t raw = smem_u32(at_smem);
   if (raw & 1023u) {  // swizzled tiles need it; never seen, but a wrong result must not follow
@@ -63,7 +65,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ,
   const uint32_t sQ = raw;
   const uint32_t sK = sQ + AT_Q_BYTES;                  // [stage][16 KB]
   const uint32_t sV = sK + AT_K_STAGES * AT_KV_BYTES;
-  const uint32_t bars = sV + AT_V_STAGES * AT_KV_BYTES;
+  const uint32_t bars = sV + AT_V_STAGES * V_BYTES;
   const uint32_t q_full = bars, k_full0 = bars + 8, k_empty0 = k_full0 + 8 * AT_K_STAGES;
   const uint32_t v_full0 = k_empty0 + 8 * AT_K_STAGES, v_empty0 = v_full0 + 8 * AT_V_STAGES;
   const uint32_t s_full0 = v_empty0 + 8 * AT_V_STAGES;  // one for each of the two S buffers
@@ -143,9 +145,11 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ,
         if (j + 2 < n_pages) load_k(j + 2);
         const int st = j % AT_V_STAGES, y = row_of(j);
         mbar_wait(v_empty0 + 8 * st, ((j / AT_V_STAGES) & 1) ^ 1, error, 10);
-        mbar_expect_tx(v_full0 + 8 * st, AT_KV_BYTES);
-        tma_load_2d(sV + st * AT_KV_BYTES, &tmV, 0, y, v_full0 + 8 * st);
-        tma_load_2d(sV + st * AT_KV_BYTES + AT_KV_BYTES / 2, &tmV, 64, y, v_full0 + 8 * st);
+        mbar_expect_tx(v_full0 + 8 * st, V_BYTES);
+#pragma unroll
+        for (int half = 0; half < VD / 64; ++half)
+          tma_load_2d(sV + st * V_BYTES + half * (MB_PAGE * 128), &tmV, 64 * half, y,
+                      v_full0 + 8 * st);
       }
     }
   } else if (warp == 1) {
@@ -179,11 +183,11 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ,
         tc_fence_after_sync();
         const uint32_t tP = tS + 64 * (j & 1);
 #pragma unroll
-        for (int half = 0; half < 2; ++half)
+        for (int half = 0; half < VD / 64; ++half)
 #pragma unroll
           for (int k = 0; k < MB_PAGE / 16; ++k) {
             const uint64_t db = umma_desc_mn128(
-                sV + st * AT_KV_BYTES + half * (AT_KV_BYTES / 2) + k * 2048, AT_KV_BYTES / 2);
+                sV + st * V_BYTES + half * (MB_PAGE * 128) + k * 2048, MB_PAGE * 128);
             umma_bf16_ts(tO + half * 64, tP + 8 * k, db, idesc_o, (j | k) != 0);
           }
         umma_commit(v_empty0 + 8 * st);  // V of this page has been read
@@ -245,7 +249,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ,
           mbar_wait(o_done0 + 8 * ((j - 1) & 1), ((j - 1) >> 1) & 1, error, 17);
           tc_fence_after_sync();
 #pragma unroll 1
-          for (int c0 = 0; c0 < AT_HD; c0 += 16) {
+          for (int c0 = 0; c0 < VD; c0 += 16) {
             float o[16];
             tmem_ld16(tO + lane_addr + c0, o);
 #pragma unroll
@@ -295,17 +299,31 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ,
     if (sink != nullptr)
       l += exp2f(sink[h] * 1.4426950408889634f - (m_ref == -INFINITY ? 0.f : m_ref));
     float inv = 1.0f / l;
-    if (gate != nullptr && row0 + row < n_new)
+    if (gate != nullptr && gate_dim == 0 && row0 + row < n_new)
       inv *= sigmoid_f32(__bfloat162float(gate[(size_t)(start + row0 + row) * gate_stride + h]));
+    // a gate for every value: this thread's row of logits
+    const bf16* gates = gate != nullptr && gate_dim > 0 && row0 + row < n_new
+                            ? gate + (size_t)(start + row0 + row) * gate_stride + (size_t)h * gate_dim
+                            : nullptr;
     // A thread holds one row of O; written from there, a warp's store would touch 32 rows with
     // 16 bytes each. Q's shared memory is free now (every product is done): the warp lays its
-    // 32 rows of 256 bytes there (16-byte piece p of row r at p ^ (r & 7): no bank conflicts
-    // either way) and writes them out two whole rows at a time.
-    const uint32_t stage = sQ + (uint32_t)q * (32 * AT_HD * 2);
+    // 32 rows of 256 bytes (or 128) there (16-byte piece p of row r at p ^ (r & 7): no bank
+    // conflicts either way) and writes them out several whole rows at a time.
+    const uint32_t stage = sQ + (uint32_t)q * (32 * VD * 2);
 #pragma unroll 1
-    for (int c0 = 0; c0 < AT_HD; c0 += 16) {
+    for (int c0 = 0; c0 < VD; c0 += 16) {
       float o[16];
       tmem_ld16(tO + lane_addr + c0, o);
+      if (gates != nullptr) {
+        const uint4 ga = *(const uint4*)(gates + c0), gb = *(const uint4*)(gates + c0 + 8);
+        const uint32_t gw[8] = {ga.x, ga.y, ga.z, ga.w, gb.x, gb.y, gb.z, gb.w};
+#pragma unroll
+        for (int i = 0; i < 8; ++i) {
+          const float2 gv = __bfloat1622float2(*(const __nv_bfloat162*)&gw[i]);
+          o[2 * i] *= sigmoid_f32(gv.x);
+          o[2 * i + 1] *= sigmoid_f32(gv.y);
+        }
+      }
       uint32_t w[8];
 #pragma unroll
       for (int i = 0; i < 8; ++i) {
@@ -313,19 +331,20 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ,
         w[i] = *reinterpret_cast<uint32_t*>(&v);
       }
       const int pc = c0 >> 3;
-      st_shared_v4(stage + lane * (AT_HD * 2) + ((pc ^ (lane & 7)) << 4),
+      st_shared_v4(stage + lane * (VD * 2) + ((pc ^ (lane & 7)) << 4),
                    make_uint4(w[0], w[1], w[2], w[3]));
-      st_shared_v4(stage + lane * (AT_HD * 2) + (((pc + 1) ^ (lane & 7)) << 4),
+      st_shared_v4(stage + lane * (VD * 2) + (((pc + 1) ^ (lane & 7)) << 4),
                    make_uint4(w[4], w[5], w[6], w[7]));
     }
     __syncwarp();
-    const int pc = lane & 15;
+    constexpr int PIECES = VD / 8, AT_ONCE = 32 / PIECES;   // 16-byte pieces a row, rows a store
+    const int pc = lane % PIECES;
 #pragma unroll 4
-    for (int i = 0; i < 16; ++i) {
-      const int r = 2 * i + (lane >> 4);
+    for (int i = 0; i < 32 / AT_ONCE; ++i) {
+      const int r = AT_ONCE * i + lane / PIECES;
       if (row0 + q * 32 + r < n_new) {
-        const uint4 v = ld_shared_v4(stage + r * (AT_HD * 2) + ((pc ^ (r & 7)) << 4));
-        *(uint4*)(out + (size_t)(start + row0 + q * 32 + r) * out_stride + (size_t)h * AT_HD +
+        const uint4 v = ld_shared_v4(stage + r * (VD * 2) + ((pc ^ (r & 7)) << 4));
+        *(uint4*)(out + (size_t)(start + row0 + q * 32 + r) * out_stride + (size_t)h * VD +
                   8 * pc) = v;
       }
     }
@@ -335,9 +354,10 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ,
   if (warp == 1) tmem_dealloc(tmem, AT_TMEM_COLS);
 }
 
-// out[t, h, :] for the new tokens of B sequences over the cache, heads of 128 values.
+// out[t, h, :] for the new tokens of B sequences over the cache, heads of 128 values with value
+// rows of `vd` (0: 128; or 64).
 // q: [T, q_cols] bfloat16 with head h of token t at q + t * q_stride + h * 128 (the fused qkv
-// rows serve); kpool / vpool: [pool_rows, 128] with pool_rows = pages * kv_heads * 64.
+// rows serve); kpool / vpool: [pool_rows, 128 / vd] with pool_rows = pages * kv_heads * 64.
 // `error`: a device word that receives 9..19 if a wait in the kernel ran out.
 MB_EXPORT int mb_attention_prefill_tc(const void* q, int q_stride, int q_cols, void* out,
                                       int out_stride, const void* kpool, const void* vpool,
@@ -346,9 +366,13 @@ MB_EXPORT int mb_attention_prefill_tc(const void* q, int q_stride, int q_cols, v
                                       const int* seq_slot, int B, int T, int max_new, int nh,
                                       int nkv, int hd, int window, float scale, int* error,
                                       const float* sink, float softcap, const void* gate,
-                                      int gate_stride, void* stream) {
+                                      int gate_stride, int gate_dim, int vd, void* stream) {
   if (B <= 0 || max_new <= 0) return 0;
-  if (hd != AT_HD) MB_FAIL("mb_attention_prefill_tc: heads of %d values (128 only)", hd);
+  if (vd <= 0) vd = hd;
+  if (hd != AT_HD || (vd != 128 && vd != 64))
+    MB_FAIL("mb_attention_prefill_tc: heads of %d and %d values (128, and 128 or 64)", hd, vd);
+  if (gate != nullptr && gate_dim > 0 && (((uintptr_t)gate & 15) || (gate_stride & 7) || gate_dim != vd))
+    MB_FAIL("mb_attention_prefill_tc: the gate's rows are not 16-byte aligned (stride %d)", gate_stride);
   if (nkv <= 0 || nh % nkv) MB_FAIL("mb_attention_prefill_tc: %d heads on %d KV heads", nh, nkv);
   if (((uintptr_t)out & 15) || (out_stride & 7))
     MB_FAIL("mb_attention_prefill_tc: out is not 16-byte aligned (stride %d)", out_stride);
@@ -358,27 +382,33 @@ MB_EXPORT int mb_attention_prefill_tc(const void* q, int q_stride, int q_cols, v
   CUtensorMap tmQ, tmK, tmV;
   if (!mb_make_map_bf16(&tmQ, q, T, q_cols, q_stride, AT_ROWS, "mb_attention_prefill_tc q")) return -1;
   if (!mb_make_map_bf16(&tmK, kpool, pool_rows, hd, hd, MB_PAGE, "mb_attention_prefill_tc k")) return -1;
-  if (!mb_make_map_bf16(&tmV, vpool, pool_rows, hd, hd, MB_PAGE, "mb_attention_prefill_tc v")) return -1;
+  if (!mb_make_map_bf16(&tmV, vpool, pool_rows, vd, vd, MB_PAGE, "mb_attention_prefill_tc v")) return -1;
   const int tiles = (max_new + AT_ROWS - 1) / AT_ROWS;
   if (tiles > 65535) MB_FAIL("mb_attention_prefill_tc: %d new tokens in one sequence", max_new);
   dim3 grid(nh, tiles, B);
   const float log2e = 1.4426950408889634f;
-#define GO(CAP_, SCALE_)                                                                       \
+#define GO(VD_, CAP_, SCALE_)                                                                  \
   {                                                                                            \
     static bool configured = false;                                                            \
     if (!configured) {                                                                         \
-      cudaError_t e = cudaFuncSetAttribute(attn_prefill_tc_kernel<CAP_>,                       \
+      cudaError_t e = cudaFuncSetAttribute(attn_prefill_tc_kernel<VD_, CAP_>,                  \
                                            cudaFuncAttributeMaxDynamicSharedMemorySize,        \
                                            AT_SMEM);                                           \
       if (e != cudaSuccess) MB_FAIL("mb_attention_prefill_tc: %s", cudaGetErrorString(e));     \
       configured = true;                                                                       \
     }                                                                                          \
-    mb_launch(attn_prefill_tc_kernel<CAP_>, grid, dim3(AT_THREADS), AT_SMEM,                   \
+    mb_launch(attn_prefill_tc_kernel<VD_, CAP_>, grid, dim3(AT_THREADS), AT_SMEM,              \
               (cudaStream_t)stream, tmQ, tmK, tmV, (bf16*)out, out_stride, page_table,         \
               max_pages, ring_pages, seq_start, seq_past, seq_slot, nh, nkv, window, SCALE_,   \
-              error, sink, softcap * log2e, (const bf16*)gate, gate_stride);                   \
+              error, sink, softcap * log2e, (const bf16*)gate, gate_stride, gate_dim);         \
   }
-  if (softcap > 0.f) GO(true, 2.f * log2e * scale / softcap) else GO(false, scale * log2e)
+  if (vd == 128) {
+    if (softcap > 0.f) GO(128, true, 2.f * log2e * scale / softcap)
+    else GO(128, false, scale * log2e)
+  } else {
+    if (softcap > 0.f) GO(64, true, 2.f * log2e * scale / softcap)
+    else GO(64, false, scale * log2e)
+  }
 #undef GO
   MB_CHECK_LAUNCH("mb_attention_prefill_tc");
 }

@@ -52,6 +52,7 @@ SOURCES = {
     "moe_tc": "moe_tc.cu",
     "latent_mma": "latent_mma.cu",
     "streams": "streams.cu",
+    "norm_step": "norm_step.cu",
     "recurrent": "recurrent.cu",
     "linear_state": "linear_state.cu",
     "attention_diff": "attention_diff.cu",

@@ -17,8 +17,9 @@
 // added up in split order by a second kernel (deterministic, no atomics) or by the caller's
 // next kernel.
 //
-// Epilogues: store (bfloat16 or float32), add into the float32 residual, and SwiGLU for a
-// weight whose rows alternate gate, up, gate, up ...: out[:, i] = silu(y[:, 2i]) * y[:, 2i+1].
+// Epilogues: store (bfloat16 or float32), add into the float32 residual, and SwiGLU (or another
+// gated form) for a weight whose rows alternate gate, up, gate, up ...:
+// out[:, i] = silu(y[:, 2i]) * y[:, 2i+1].
 //
 // Warp roles in a CTA of 192 threads: warp 0 loads (one elected lane), warp 1 allocates TMEM
 // and issues the MMAs (one elected lane), warps 2-5 read the accumulator and store.
@@ -26,6 +27,8 @@
 // This replaces the reference's `gemm8` / `linear8` (tools/cuda/linear.cu:418-606 of the
 // reference project), which multiply in float32 on the CUDA cores.
 #include "tc_common.cuh"
+
+#include <string.h>
 
 MB_DEFINE_LAST_ERROR
 
@@ -41,7 +44,10 @@ MB_EXPORT int mb_gemm_tc_last_launches() { return g_last_launches; }
 // act(gate) * up with act = SiLU or the tanh form of GELU. In these two modes nothing is split,
 // and the pointer that otherwise names the partial sums may name bfloat16 biases instead, one
 // per weight row (gate and up alternating like the rows), which are added before the activation.
-enum { TC_STORE = 0, TC_ADD = 1, TC_PARTIAL = 2, TC_SWIGLU = 3, TC_GEGLU = 4 };
+// TC_CLAMPED is the clamped form: g' = min(gate, limit), u' = clamp(up, -limit, limit),
+// g' sigmoid(1.702 g') (u' + 1); the pitch that otherwise belongs to the partial sums then carries
+// the limit's bits.
+enum { TC_STORE = 0, TC_ADD = 1, TC_PARTIAL = 2, TC_SWIGLU = 3, TC_GEGLU = 4, TC_CLAMPED = 5 };
 
 #define TC_BM 128
 #define TC_BK 64
@@ -70,8 +76,13 @@ __device__ __forceinline__ void store_out(void* C, int c_dtype, size_t idx, floa
 __device__ __forceinline__ float silu_mul(float g, float u) {
   return __fdividef(g, 1.0f + __expf(-g)) * u;
 }
-// the same for either activation; gelu_tanh(g) = g * sigmoid(2 sqrt(2/pi) (g + 0.044715 g^3))
-__device__ __forceinline__ float gated_mul(float g, float u, int mode) {
+// the same for any of the activations; gelu_tanh(g) = g * sigmoid(2 sqrt(2/pi) (g + 0.044715 g^3))
+__device__ __forceinline__ float gated_mul(float g, float u, int mode, float limit) {
+  if (mode == TC_CLAMPED) {
+    g = fminf(g, limit);
+    u = fminf(fmaxf(u, -limit), limit);
+    return __fdividef(g, 1.0f + __expf(-1.702f * g)) * (u + 1.0f);
+  }
   if (mode == TC_GEGLU) {
     const float z = 1.5957691216057308f * (g + 0.044715f * g * g * g);
     return __fdividef(g, 1.0f + __expf(-z)) * u;
@@ -93,6 +104,9 @@ __device__ __forceinline__ void unary16(float* v, int act) {
     }
   }
 }
+__device__ __forceinline__ float limit_of(long long partial_ld) {
+  return __uint_as_float((unsigned)partial_ld);
+}
 __device__ __forceinline__ float pair_bias(const float* part, int row) {
   return part ? __bfloat162float(((const __nv_bfloat16*)part)[row]) : 0.f;
 }
@@ -106,6 +120,7 @@ __device__ __forceinline__ void store_row16(const float* v, void* C, int c_dtype
   if (mode >= TC_SWIGLU) {
     // columns 2i and 2i+1 are gate and up of output feature (b0 + 2i) / 2
     __nv_bfloat16* p = (__nv_bfloat16*)C + (size_t)a * ldc + (b0 >> 1);
+    const float limit = limit_of(partial_ld);
     float w[16];
 #pragma unroll
     for (int j = 0; j < 16; ++j) w[j] = v[j] + (b0 + j < rowsB ? pair_bias(part, b0 + j) : 0.f);
@@ -113,12 +128,12 @@ __device__ __forceinline__ void store_row16(const float* v, void* C, int c_dtype
       __nv_bfloat162 h[4];
 #pragma unroll
       for (int j = 0; j < 4; ++j)
-        h[j] = __floats2bfloat162_rn(gated_mul(w[4 * j], w[4 * j + 1], mode),
-                                     gated_mul(w[4 * j + 2], w[4 * j + 3], mode));
+        h[j] = __floats2bfloat162_rn(gated_mul(w[4 * j], w[4 * j + 1], mode, limit),
+                                     gated_mul(w[4 * j + 2], w[4 * j + 3], mode, limit));
       *(uint4*)p = *(uint4*)&h[0];
     } else {
       for (int j = 0; j < 16 && b0 + j + 1 < rowsB; j += 2)
-        p[j >> 1] = __float2bfloat16_rn(gated_mul(w[j], w[j + 1], mode));
+        p[j >> 1] = __float2bfloat16_rn(gated_mul(w[j], w[j + 1], mode, limit));
     }
   } else if (mode == TC_PARTIAL) {
     float* p = part + (size_t)a * partial_ld + b0;
@@ -165,6 +180,7 @@ __device__ __forceinline__ void staged_rows(uint32_t taddr, uint32_t stage_w, in
                                             long long partial_ld, int act) {
   const int acc_cols = mode >= TC_SWIGLU ? 128 : (c_dtype == MB_BF16 && mode == TC_STORE ? 64 : 32);
   const uint32_t mine = stage_w + lane * 128;
+  const float limit = limit_of(partial_ld);   // of the clamped gated form
 #pragma unroll 1
   for (int c0 = 0; c0 < width; c0 += acc_cols) {
     if (n0 + c0 >= N) break;
@@ -185,8 +201,8 @@ __device__ __forceinline__ void staged_rows(uint32_t taddr, uint32_t stage_w, in
         __nv_bfloat162 h[4];
 #pragma unroll
         for (int j = 0; j < 4; ++j)
-          h[j] = __floats2bfloat162_rn(gated_mul(v[4 * j], v[4 * j + 1], mode),
-                                       gated_mul(v[4 * j + 2], v[4 * j + 3], mode));
+          h[j] = __floats2bfloat162_rn(gated_mul(v[4 * j], v[4 * j + 1], mode, limit),
+                                       gated_mul(v[4 * j + 2], v[4 * j + 3], mode, limit));
         st_shared_v4(mine + ((g ^ (lane & 7)) << 4), *(uint4*)&h[0]);
       } else if (acc_cols == 64) {
         __nv_bfloat162 h[8];
@@ -414,7 +430,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ 
             const int bb = n0 + c0 + j;
             if (mine && !(lane & 1) && bb < rowsB)
               ((__nv_bfloat16*)C)[(size_t)bb * ldc + (a >> 1)] =
-                  __float2bfloat16_rn(gated_mul(own, up, mode));
+                  __float2bfloat16_rn(gated_mul(own, up, mode, limit_of(partial_ld)));
           }
           continue;
         }
@@ -641,6 +657,15 @@ static int pair_capacity(int sms) {
 }
 MB_EXPORT int mb_gemm_tc_pairs(int sms) { return pair_capacity(sms); }
 
+// set by mb_gemm_tc_gated around its call: the biases of a gated epilogue (see the modes)
+static thread_local const void* g_pair_bias = nullptr;
+static thread_local float g_pair_limit = 0.f;   // and the limit of the clamped form
+static long long limit_bits() {
+  unsigned bits;
+  memcpy(&bits, &g_pair_limit, sizeof(bits));
+  return (long long)bits;
+}
+
 template <typename... KArgs, typename... Args>
 static cudaError_t mb_launch_pair(void (*kernel)(KArgs...), dim3 grid, dim3 block, size_t smem,
                                   cudaStream_t stream, Args... args) {
@@ -679,7 +704,8 @@ static int launch_pair(const CUtensorMap& tmA, const CUtensorMap& tmB, void* C, 
   const int grid = 2 * (num_tiles < pairs ? num_tiles : pairs);
   mb_launch_pair(gemm_tc_pair_kernel<BN>, dim3(grid), dim3(TC_THREADS), Tc2Cfg<BN>::SMEM, s, tmA,
                  tmB, C, c_dtype, ldc, M, N, K, kb_per_split, mode, partial, (long long)M * N,
-                 (long long)N, tiles_m, tiles_n, num_tiles, error);
+                 (mode & 255) >= TC_SWIGLU ? limit_bits() : (long long)N, tiles_m, tiles_n,
+                 num_tiles, error);
   cudaError_t le = cudaGetLastError();
   if (le != cudaSuccess) MB_FAIL("mb_gemm_tc (pairs): %s", cudaGetErrorString(le));
   return 0;
@@ -770,9 +796,6 @@ MB_EXPORT int mb_gemm_tc_supported(const void* A, int lda, const void* W, int M,
 // (1 load, 2 MMA, 3 epilogue). `sms`: the number of SMs of the device. `defer`: when K was split
 // (mb_gemm_tc_last_splits() > 1) the partial sums stay in the workspace as [splits][M][N] and C
 // is not touched: the caller's next kernel adds them up.
-// set by mb_gemm_tc_gated around its call: the biases of a gated epilogue (see the modes)
-static thread_local const void* g_pair_bias = nullptr;
-
 MB_EXPORT int mb_gemm_tc(const void* A, int lda, const void* W, void* C, int c_dtype, int ldc,
                          int M, int N, int K, int epilogue, float* workspace,
                          long long workspace_floats, int defer, int* error, int sms,
@@ -787,7 +810,8 @@ MB_EXPORT int mb_gemm_tc(const void* A, int lda, const void* W, void* C, int c_d
   if (act != 0 && (epilogue != TC_STORE || (act != 1 && act != 2 && act != 4)))
     MB_FAIL("mb_gemm_tc: activation %d with epilogue %d", act, epilogue);
   if (act) workspace = nullptr;
-  if (epilogue != TC_STORE && epilogue != TC_ADD && epilogue != TC_SWIGLU && epilogue != TC_GEGLU)
+  if (epilogue != TC_STORE && epilogue != TC_ADD && epilogue != TC_SWIGLU && epilogue != TC_GEGLU &&
+      epilogue != TC_CLAMPED)
     MB_FAIL("mb_gemm_tc: epilogue %d", epilogue);
   if (epilogue == TC_ADD && c_dtype != MB_F32) MB_FAIL("mb_gemm_tc: the residual is float32");
   if (epilogue >= TC_SWIGLU && (c_dtype != MB_BF16 || (N & 1)))
@@ -907,7 +931,7 @@ MB_EXPORT int mb_gemm_tc(const void* A, int lda, const void* W, void* C, int c_d
   }
   const int mode = p.splits > 1 ? TC_PARTIAL : (epilogue | (act << 8));
   float* partial = p.splits > 1 ? workspace : (float*)g_pair_bias;
-  const long long pstride = (long long)M * N, pld = N;
+  const long long pstride = (long long)M * N, pld = epilogue >= TC_SWIGLU ? limit_bits() : N;
   int rc;
 #define GO(BN_, SW_)                                                                        \
   rc = launch_tc<BN_, SW_>(tmA, tmB, C, c_dtype, ldc, rowsA, rowsB, K, p, mode, partial,    \
@@ -932,16 +956,19 @@ MB_EXPORT int mb_gemm_tc(const void* A, int lda, const void* W, void* C, int c_d
 }
 
 // C[M, N / 2] = act(gate + b_gate) * (up + b_up) for a weight [N, K] whose rows alternate gate
-// and up; act 0: SiLU, 1: the tanh form of GELU; pair_bias: bfloat16 [N], alternating like the
-// rows, or null. C is bfloat16.
+// and up; act 0: SiLU, 1: the tanh form of GELU, 2: the clamped form with `limit` (see the modes);
+// pair_bias: bfloat16 [N], alternating like the rows, or null. C is bfloat16.
 MB_EXPORT int mb_gemm_tc_gated(const void* A, int lda, const void* W, void* C, int ldc, int M,
-                               int N, int K, int act, const void* pair_bias, int* error, int sms,
-                               void* stream) {
-  if (act != 0 && act != 1) MB_FAIL("mb_gemm_tc_gated: activation %d", act);
+                               int N, int K, int act, const void* pair_bias, float limit, int* error,
+                               int sms, void* stream) {
+  if (act < 0 || act > 2) MB_FAIL("mb_gemm_tc_gated: activation %d", act);
   g_pair_bias = pair_bias;
-  const int rc = mb_gemm_tc(A, lda, W, C, MB_BF16, ldc, M, N, K, act == 1 ? TC_GEGLU : TC_SWIGLU,
-                            nullptr, 0, 0, error, sms, stream);
+  g_pair_limit = limit;
+  const int rc = mb_gemm_tc(A, lda, W, C, MB_BF16, ldc, M, N, K,
+                            act == 2 ? TC_CLAMPED : (act == 1 ? TC_GEGLU : TC_SWIGLU), nullptr, 0,
+                            0, error, sms, stream);
   g_pair_bias = nullptr;
+  g_pair_limit = 0.f;
   return rc;
 }
 

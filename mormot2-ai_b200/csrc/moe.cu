@@ -100,14 +100,17 @@ __device__ __forceinline__ void route_token(const float* __restrict__ zr, int pa
   if (sg && lane == 0) *sg = 1.0f / (1.0f + expf(-route_logit(zr, parts, part_stride, shared_col)));
 }
 
-// The other scoring: s = softmax(z) over all E columns; the choice goes by s + corr (the lower
-// index on a tie), the weights are the chosen s times wscale, not renormalized. Up to 256
-// columns (a lane keeps eight).
+// The other scorings: s = softmax(z) over all E columns, or s = sigmoid(z) column by column
+// (`sigmoid`); the choice goes by s + corr (the lower index on a tie), the weights are the chosen
+// s times wscale, not renormalized. Up to 256 columns (a lane keeps eight).
+// `groups` > 1: the columns are that many equal groups of neighbours; a group's score is the sum
+// of its two largest choice scores, and only columns of the `keep` best groups (the lower group on
+// a tie) can be chosen. At most 32 groups (lane g keeps group g's score).
 __device__ __forceinline__ void route_token_scored(const float* __restrict__ zr, int parts,
                                                    size_t part_stride, int E, int top,
                                                    const float* __restrict__ corr, float wscale,
                                                    int* __restrict__ ids, float* __restrict__ w,
-                                                   int lane) {
+                                                   int lane, bool sigmoid, int groups, int keep) {
   float sc[8], ch[8];
   float mx = -INFINITY;
 #pragma unroll
@@ -116,19 +119,60 @@ __device__ __forceinline__ void route_token_scored(const float* __restrict__ zr,
     sc[j] = i < E ? route_logit(zr, parts, part_stride, i) : -INFINITY;
     mx = fmaxf(mx, sc[j]);
   }
-  mx = warp_max(mx);
-  float sum = 0.f;
+  if (sigmoid) {
 #pragma unroll
-  for (int j = 0; j < 8; ++j) {
-    sc[j] = lane + 32 * j < E ? expf(sc[j] - mx) : 0.f;
-    sum += sc[j];
+    for (int j = 0; j < 8; ++j) sc[j] = lane + 32 * j < E ? sigmoid_f32(sc[j]) : 0.f;
+  } else {
+    mx = warp_max(mx);
+    float sum = 0.f;
+#pragma unroll
+    for (int j = 0; j < 8; ++j) {
+      sc[j] = lane + 32 * j < E ? expf(sc[j] - mx) : 0.f;
+      sum += sc[j];
+    }
+    sum = warp_sum(sum);
+#pragma unroll
+    for (int j = 0; j < 8; ++j) sc[j] = sc[j] / sum;
   }
-  sum = warp_sum(sum);
 #pragma unroll
   for (int j = 0; j < 8; ++j) {
     const int i = lane + 32 * j;
-    sc[j] = sc[j] / sum;
     ch[j] = i < E ? sc[j] + (corr ? corr[i] : 0.f) : -INFINITY;
+  }
+  if (groups > 1) {
+    const int size = E / groups;
+    float mine = -INFINITY;
+    for (int g = 0; g < groups; ++g) {
+      float a = -INFINITY, b = -INFINITY;    // this lane's two largest of the group
+#pragma unroll
+      for (int j = 0; j < 8; ++j) {
+        const int i = lane + 32 * j;
+        if (i >= g * size && i < (g + 1) * size) {
+          b = fmaxf(b, fminf(a, ch[j]));
+          a = fmaxf(a, ch[j]);
+        }
+      }
+#pragma unroll
+      for (int o = 16; o > 0; o >>= 1) {
+        const float oa = __shfl_xor_sync(0xffffffffu, a, o);
+        const float ob = __shfl_xor_sync(0xffffffffu, b, o);
+        b = fmaxf(fmaxf(b, ob), fminf(a, oa));
+        a = fmaxf(a, oa);
+      }
+      if (lane == g) mine = size > 1 ? a + b : a;
+    }
+    // a group is open when fewer than `keep` groups are ahead of it
+    int ahead = 0;
+    for (int g = 0; g < groups; ++g) {
+      const float v = __shfl_sync(0xffffffffu, mine, g);
+      ahead += v > mine || (v == mine && g < lane);
+    }
+    const unsigned open = __ballot_sync(0xffffffffu, lane < groups && ahead < keep);
+#pragma unroll
+    for (int j = 0; j < 8; ++j) {
+      const int i = lane + 32 * j;
+      if (i < E && !((open >> (i / size)) & 1u)) ch[j] = -INFINITY;
+    }
   }
   float last_v = INFINITY, mine = 0.f;
   int last_i = -1;
@@ -140,7 +184,7 @@ __device__ __forceinline__ void route_token_scored(const float* __restrict__ zr,
       const int i = lane + 32 * j;
       const float v = ch[j];
       const bool open = i < E && (v < last_v || (v == last_v && i > last_i));
-      if (open && (v > best || (v == best && i < best_i))) {
+      if (open && v > -INFINITY && (v > best || (v == best && i < best_i))) {
         best = v;
         best_i = i;
         best_s = sc[j];
@@ -173,32 +217,44 @@ __global__ void __launch_bounds__(128)
 moe_route_kernel(const float* __restrict__ z, int ldz, int parts, size_t part_stride, int E,
                  int top, int shared_col, int* __restrict__ ids, float* __restrict__ w,
                  float* __restrict__ sg, int T, int mode, const float* __restrict__ corr,
-                 float wscale) {
+                 float wscale, int groups, int keep) {
   mb_grid_wait();
   mb_grid_launch_next();
   const int lane = threadIdx.x & 31;
   const int t = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
   if (t >= T) return;
-  if (mode == 1) {
+  if (mode != 0) {
     route_token_scored(z + (size_t)t * ldz, parts, part_stride, E, top, corr, wscale,
-                       ids + (size_t)t * top, w + (size_t)t * top, lane);
+                       ids + (size_t)t * top, w + (size_t)t * top, lane, mode == 2, groups, keep);
     return;
   }
   route_token(z + (size_t)t * ldz, parts, part_stride, E, top, shared_col, ids + (size_t)t * top,
               w + (size_t)t * top, sg ? sg + t : nullptr, lane);
 }
 
+// mode 0: softmax over the chosen logits; 1: scores by a softmax over all; 2: by a sigmoid each
+static int route_groups(const char* who, int mode, int E, int top, int groups, int keep) {
+  if (mode < 0 || mode > 2) MB_FAIL("%s: scoring %d", who, mode);
+  if (groups <= 1) return 0;
+  if (mode == 0 || groups > 32 || E % groups || keep < 1 || keep > groups ||
+      top > keep * (E / groups))
+    MB_FAIL("%s: %d of %d columns from %d of %d groups", who, top, E, keep, groups);
+  return 0;
+}
+
 MB_EXPORT int mb_moe_route(const float* z, int ldz, int parts, long long part_stride, int E,
                            int top, int shared_col, int* ids, float* w, float* sg, int T,
-                           int mode, const float* corr, float wscale, void* stream) {
+                           int mode, const float* corr, float wscale, int groups, int keep,
+                           void* stream) {
   if (T <= 0) return 0;
-  if (mode == 1 && (E > 256 || sg != nullptr))
+  if (route_groups("mb_moe_route", mode, E, top, groups, keep)) return -1;
+  if (mode != 0 && (E > 256 || sg != nullptr))
     MB_FAIL("mb_moe_route: scores over all of %d columns (at most 256, no gate column)", E);
   if (top <= 0 || top > 32 || top > E) MB_FAIL("mb_moe_route: %d of %d experts", top, E);
   if ((sg != nullptr) != (shared_col >= 0)) MB_FAIL("mb_moe_route: the shared gate and its column");
   if (parts < 1) MB_FAIL("mb_moe_route: %d parts", parts);
   mb_launch(moe_route_kernel, dim3((T + 3) / 4), dim3(128), 0, (cudaStream_t)stream, z, ldz,
-            parts, (size_t)part_stride, E, top, shared_col, ids, w, sg, T, mode, corr, wscale);
+            parts, (size_t)part_stride, E, top, shared_col, ids, w, sg, T, mode, corr, wscale, groups, keep);
   MB_CHECK_LAUNCH("mb_moe_route");
 }
 
@@ -215,7 +271,7 @@ moe_plan_kernel(int* __restrict__ ids, int A, int E, int bm, int max_tiles,
                 int* __restrict__ plan, const float* __restrict__ z, int ldz, int parts,
                 size_t part_stride, int top, int shared_col, float* __restrict__ w,
                 float* __restrict__ sg, int mode, const float* __restrict__ corr, float wscale,
-                int E_route, const int* __restrict__ table, const int* __restrict__ tok_ids,
+                int groups, int keep, int E_route, const int* __restrict__ table, const int* __restrict__ tok_ids,
                 int V) {
   mb_grid_wait();
   mb_grid_launch_next();
@@ -223,9 +279,10 @@ moe_plan_kernel(int* __restrict__ ids, int A, int E, int bm, int max_tiles,
   if (z != nullptr) {
     const int T = A / top, lane = threadIdx.x & 31;
     for (int t = threadIdx.x >> 5; t < T; t += blockDim.x >> 5) {
-      if (mode == 1)
+      if (mode != 0)
         route_token_scored(z + (size_t)t * ldz, parts, part_stride, E_route, top, corr, wscale,
-                           ids + (size_t)t * top, w + (size_t)t * top, lane);
+                           ids + (size_t)t * top, w + (size_t)t * top, lane, mode == 2, groups,
+                           keep);
       else
         route_token(z + (size_t)t * ldz, parts, part_stride, E_route, top, shared_col,
                     ids + (size_t)t * top, w + (size_t)t * top, sg ? sg + t : nullptr, lane);
@@ -278,7 +335,7 @@ MB_EXPORT int mb_moe_plan(int* ids, int A, int E, int bm, int max_tiles, int* pl
   if (max_tiles < (A + bm - 1) / bm + E) MB_FAIL("mb_moe_plan: room for %d tiles", max_tiles);
   mb_launch(moe_plan_kernel, dim3(1), dim3(1024), (size_t)2 * E * sizeof(int),
             (cudaStream_t)stream, ids, A, E, bm, max_tiles, plan, (const float*)nullptr, 0, 1,
-            (size_t)0, 1, -1, (float*)nullptr, (float*)nullptr, 0, (const float*)nullptr, 1.0f, E,
+            (size_t)0, 1, -1, (float*)nullptr, (float*)nullptr, 0, (const float*)nullptr, 1.0f, 1, 1, E,
             (const int*)nullptr, (const int*)nullptr, 0);
   MB_CHECK_LAUNCH("mb_moe_plan");
 }
@@ -293,7 +350,7 @@ MB_EXPORT int mb_moe_table_plan(const int* table, int V, int top, const int* tok
   mb_launch(moe_plan_kernel, dim3(1), dim3(1024), (size_t)2 * E * sizeof(int),
             (cudaStream_t)stream, (int*)nullptr, A, E, bm, max_tiles, plan, (const float*)nullptr, 0,
             1, (size_t)0, top, -1, (float*)nullptr, (float*)nullptr, 0, (const float*)nullptr, 1.0f,
-            E, table, tok_ids, V);
+            1, 1, E, table, tok_ids, V);
   MB_CHECK_LAUNCH("mb_moe_table_plan");
 }
 
@@ -301,10 +358,11 @@ MB_EXPORT int mb_moe_table_plan(const int* table, int V, int top, const int* tok
 MB_EXPORT int mb_moe_route_plan(const float* z, int ldz, int parts, long long part_stride, int E,
                                 int top, int shared_col, int* ids, float* w, float* sg, int T,
                                 int bm, int max_tiles, int* plan, int mode, const float* corr,
-                                float wscale, int E_route, void* stream) {
+                                float wscale, int groups, int keep, int E_route, void* stream) {
   if (T <= 0) return 0;
   if (E_route < E) MB_FAIL("mb_moe_route_plan: %d routed columns for %d experts", E_route, E);
-  if (mode == 1 && (E_route > 256 || sg != nullptr))
+  if (route_groups("mb_moe_route_plan", mode, E_route, top, groups, keep)) return -1;
+  if (mode != 0 && (E_route > 256 || sg != nullptr))
     MB_FAIL("mb_moe_route_plan: scores over all of %d columns (at most 256, no gate column)", E_route);
   if (T > 64) MB_FAIL("mb_moe_route_plan: %d tokens (at most 64)", T);
   if (top <= 0 || top > 32 || top > E_route) MB_FAIL("mb_moe_route_plan: %d of %d experts", top, E_route);
@@ -314,7 +372,7 @@ MB_EXPORT int mb_moe_route_plan(const float* z, int ldz, int parts, long long pa
   if (max_tiles < (A + bm - 1) / bm + E) MB_FAIL("mb_moe_route_plan: room for %d tiles", max_tiles);
   mb_launch(moe_plan_kernel, dim3(1), dim3(1024), (size_t)2 * E * sizeof(int),
             (cudaStream_t)stream, ids, A, E, bm, max_tiles, plan, z, ldz, parts,
-            (size_t)part_stride, top, shared_col, w, sg, mode, corr, wscale, E_route,
+            (size_t)part_stride, top, shared_col, w, sg, mode, corr, wscale, groups, keep, E_route,
             (const int*)nullptr, (const int*)nullptr, 0);
   MB_CHECK_LAUNCH("mb_moe_route_plan");
 }

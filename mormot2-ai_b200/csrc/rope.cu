@@ -759,3 +759,180 @@ MB_EXPORT int mb_maps_norm_rope_store(const void* rows, int in_dtype, int parts,
 #undef GO
   MB_CHECK_LAUNCH("mb_maps_norm_rope_store");
 }
+
+// ------------------------------------------------------------------ heads without a norm
+// Rows [q | k | v | gates] of a product (or its float32 split sums [parts][T][ld], added up in
+// split order) for attention that norms neither q nor k: the first rot_dim values of every q and k
+// head turn, pair (i, i + rot_dim / 2), cosine and sine times `amp`; q goes to q_out (rows of q_ld
+// values; it may be the product's row itself), k and v into the cache.
+// `first` [T, nkv * vd] (or null) is what values are blended with across layers: without `lam` it
+// receives this layer's values, with it (one float32 on the device) the values become
+// (1 - lam) v + lam first before they are stored. `gate_out` (or null) [T, gate_n]: receives the
+// gate_n columns behind v (of split sums; a product's own row is read where it lies).
+// V neighbouring values a thread (8: everything on 16-byte boundaries; 1: any sizes).
+template <typename T, int V> struct RsVec {
+  static __device__ __forceinline__ void load(const T* p, float* v) {
+#pragma unroll
+    for (int i = 0; i < V; ++i) v[i] = to_f32<T>(p[i]);
+  }
+  static __device__ __forceinline__ void store(T* p, const float* v) {
+#pragma unroll
+    for (int i = 0; i < V; ++i) p[i] = from_f32<T>(v[i]);
+  }
+};
+template <> struct RsVec<__nv_bfloat16, 8> {
+  static __device__ __forceinline__ void load(const __nv_bfloat16* p, float* v) {
+    unpack8(*(const uint4*)p, v);
+  }
+  static __device__ __forceinline__ void store(__nv_bfloat16* p, const float* v) {
+    *(uint4*)p = pack8(v);
+  }
+};
+template <> struct RsVec<float, 8> {
+  static __device__ __forceinline__ void load(const float* p, float* v) {
+    const float4 a = *(const float4*)p, b = *(const float4*)(p + 4);
+    v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w;
+    v[4] = b.x; v[5] = b.y; v[6] = b.z; v[7] = b.w;
+  }
+  static __device__ __forceinline__ void store(float* p, const float* v) {
+    *(float4*)p = make_float4(v[0], v[1], v[2], v[3]);
+    *(float4*)(p + 4) = make_float4(v[4], v[5], v[6], v[7]);
+  }
+};
+
+template <typename TI, typename TO, int V>
+__global__ void __launch_bounds__(256)
+rope_store_kernel(const TI* rows, int parts, size_t part_stride, int ld,
+                  const float* __restrict__ inv_freq, int rot_dim, float amp,
+                  const int* __restrict__ tok_slot, const int* __restrict__ tok_pos,
+                  const int* __restrict__ page_table, int max_pages, int ring_pages,
+                  TO* __restrict__ kpool, TO* __restrict__ vpool, TO* q_out, int q_ld,
+                  TO* __restrict__ first, const float* __restrict__ lam, TO* __restrict__ gate_out,
+                  int gate_n, int nh, int nkv, int dim, int vd) {
+  extern __shared__ float rs_angles[];   // [rot_dim / 2] cosines, then sines
+  const int half = rot_dim >> 1;
+  float* cs = rs_angles;
+  float* sn = cs + half;
+  const int t = blockIdx.x;
+  // ahead of the wait: what does not depend on the kernel before
+  const int pos = tok_pos[t], slot = tok_slot[t];
+  for (int i = threadIdx.x; i < half; i += blockDim.x) {
+    float s, c;
+    sincosf(inv_freq[i] * (float)pos, &s, &c);
+    cs[i] = c * amp;
+    sn[i] = s * amp;
+  }
+  const float l = lam ? *lam : 0.f;
+  __syncthreads();
+  mb_grid_wait();
+  mb_grid_launch_next();
+  const TI* row = rows + (size_t)t * ld;
+  auto read = [&](int col, float* v) {
+    RsVec<TI, V>::load(row + col, v);
+    for (int p = 1; p < parts; ++p) {
+      float a[V];
+      RsVec<TI, V>::load(row + (size_t)p * part_stride + col, a);
+#pragma unroll
+      for (int i = 0; i < V; ++i) v[i] += a[i];
+    }
+  };
+  // a head of q or k: pairs of V values that turn together, then V values at a time that pass
+  const int pairs = half / V, per_head = pairs + (dim - rot_dim) / V;
+  const int n_heads = (nh + nkv) * per_head, per_v = vd / V, n_v = nkv * per_v;
+  const int total = n_heads + n_v + (gate_out ? gate_n / V : 0);
+  for (int n = blockIdx.y * blockDim.x + threadIdx.x; n < total; n += gridDim.y * blockDim.x) {
+    if (n < n_heads) {
+      const int head = n / per_head, i = n - head * per_head;
+      TO* dst;
+      if (head < nh) {
+        dst = q_out + (size_t)t * q_ld + (size_t)head * dim;
+      } else {
+        dst = kpool + kv_row(page_table, max_pages, ring_pages, slot, pos, nkv, head - nh) * dim;
+      }
+      float a[V];
+      if (i < pairs) {
+        float b[V];
+        read(head * dim + i * V, a);
+        read(head * dim + half + i * V, b);
+#pragma unroll
+        for (int j = 0; j < V; ++j) {
+          const float c = cs[i * V + j], s = sn[i * V + j], u = a[j], w = b[j];
+          a[j] = u * c - w * s;
+          b[j] = w * c + u * s;
+        }
+        RsVec<TO, V>::store(dst + i * V, a);
+        RsVec<TO, V>::store(dst + half + i * V, b);
+      } else {
+        const int at = rot_dim + (i - pairs) * V;
+        read(head * dim + at, a);
+        RsVec<TO, V>::store(dst + at, a);
+      }
+    } else if (n < n_heads + n_v) {
+      const int m = n - n_heads, g = m / per_v, at = (m - g * per_v) * V;
+      float v[V];
+      read((nh + nkv) * dim + g * vd + at, v);
+      if (first) {
+        TO* f = first + ((size_t)t * nkv + g) * vd + at;
+        if (lam) {
+          float o[V];
+          RsVec<TO, V>::load(f, o);
+#pragma unroll
+          for (int j = 0; j < V; ++j) v[j] = (1.0f - l) * v[j] + l * o[j];
+        } else {
+          RsVec<TO, V>::store(f, v);
+        }
+      }
+      RsVec<TO, V>::store(
+          vpool + kv_row(page_table, max_pages, ring_pages, slot, pos, nkv, g) * vd + at, v);
+    } else {
+      const int at = (n - n_heads - n_v) * V;
+      float v[V];
+      read((nh + nkv) * dim + nkv * vd + at, v);
+      RsVec<TO, V>::store(gate_out + (size_t)t * gate_n + at, v);
+    }
+  }
+}
+
+MB_EXPORT int mb_rope_store(const void* rows, int in_dtype, int parts, long long part_stride, int ld,
+                            const float* inv_freq, int rot_dim, float amp, const int* tok_slot,
+                            const int* tok_pos, const int* page_table, int max_pages,
+                            int ring_pages, void* kpool, void* vpool, void* q_out, int q_ld,
+                            int dtype, void* first, const float* lam, void* gate_out, int gate_n,
+                            int T, int nh, int nkv, int dim, int vd, void* stream) {
+  if (T <= 0) return 0;
+  if (rot_dim < 0 || rot_dim > dim || (rot_dim & 1) || (rot_dim > 0 && inv_freq == nullptr))
+    MB_FAIL("mb_rope_store: %d of %d values rotate", rot_dim, dim);
+  if (nh <= 0 || nkv <= 0 || nh % nkv || parts < 1 || dim <= 0 || vd <= 0)
+    MB_FAIL("mb_rope_store: %d heads on %d KV heads, %d parts", nh, nkv, parts);
+  if (ld < (nh + nkv) * dim + nkv * vd + (gate_out ? gate_n : 0) || q_ld < nh * dim)
+    MB_FAIL("mb_rope_store: row pitches of %d and %d", ld, q_ld);
+  if (in_dtype == MB_BF16 && dtype != MB_BF16)
+    MB_FAIL("mb_rope_store: bfloat16 rows for float32 activations");
+  if (lam != nullptr && first == nullptr) MB_FAIL("mb_rope_store: nothing to blend with");
+  if (rot_dim > 8192) MB_FAIL("mb_rope_store: %d rotating values", rot_dim);
+  cudaStream_t s = (cudaStream_t)stream;
+  const uintptr_t bits = (uintptr_t)rows | (uintptr_t)kpool | (uintptr_t)vpool | (uintptr_t)q_out |
+                         (uintptr_t)first | (uintptr_t)gate_out;
+  const bool wide = dim % 8 == 0 && vd % 8 == 0 && (rot_dim / 2) % 8 == 0 && ld % 8 == 0 &&
+                    q_ld % 8 == 0 && part_stride % 8 == 0 && (!gate_out || gate_n % 8 == 0) &&
+                    (bits & 15) == 0;
+  const int V = wide ? 8 : 1;
+  const int items = (nh + nkv) * (dim - rot_dim / 2) / V + nkv * vd / V + (gate_out ? gate_n / V : 0);
+  // few tokens: an item a thread; many: a block walks its token's items, the angles once
+  const int threads = items >= 256 ? 256 : (items > 64 ? 128 : 64);
+  const int most = (items + threads - 1) / threads;
+  dim3 grid(T, T <= 64 ? most : (most + 3) / 4);
+  const size_t smem = (size_t)rot_dim * sizeof(float);
+#define GO(TI_, TO_, V_)                                                                        \
+  mb_launch(rope_store_kernel<TI_, TO_, V_>, grid, dim3(threads), smem, s, (const TI_*)rows,    \
+            parts, (size_t)part_stride, ld, inv_freq, rot_dim, amp, tok_slot, tok_pos,          \
+            page_table, max_pages, ring_pages, (TO_*)kpool, (TO_*)vpool, (TO_*)q_out, q_ld,     \
+            (TO_*)first, lam, (TO_*)gate_out, gate_n, nh, nkv, dim, vd)
+#define GO_V(TI_, TO_) { if (wide) GO(TI_, TO_, 8); else GO(TI_, TO_, 1); }
+  if (dtype == MB_F32) GO_V(float, float)
+  else if (in_dtype == MB_F32) GO_V(float, __nv_bfloat16)
+  else GO_V(__nv_bfloat16, __nv_bfloat16)
+#undef GO_V
+#undef GO
+  MB_CHECK_LAUNCH("mb_rope_store");
+}

@@ -171,16 +171,18 @@ class Runtime:
 
     def attention(self, q, q_stride, out, step, line, nh, nkv, hd, window, scale, vd=0,
                   sink=None, softcap=0.0, gate=None, gate_stride=0, slopes=None,
-                  keep_first=0) -> None:
+                  keep_first=0, gate_dim=0) -> None:
         """``vd``: the size of a value row where it differs from ``hd``; ``sink``: float32
         [nh], one more term of every softmax denominator; ``softcap`` > 0: a cap
         c tanh(s / c) on the scaled scores; ``gate``: one logit per (token, head) whose sigmoid
-        multiplies the head's output; ``slopes``: float32 [nh], taken off the scores times the
+        multiplies the head's output, or, with ``gate_dim`` (the size of a value row), one per
+        value; ``slopes``: float32 [nh], taken off the scores times the
         distance; ``keep_first``: positions at a sequence's start that a window never loses."""
-        if self.fast_kernels and (not vd or vd == hd):
+        if self.fast_kernels:
             from ..parts import attention_fast
             if attention_fast.run(self, q, q_stride, out, step, line, nh, nkv, hd, window, scale,
-                                  sink, softcap, gate, gate_stride, slopes, keep_first):
+                                  sink, softcap, gate, gate_stride, slopes, keep_first, vd,
+                                  gate_dim):
                 return
         K.attention_simt(q, q_stride, out, step, line, nh, nkv, hd, window, scale, vd, sink,
-                         softcap, gate, gate_stride, slopes, keep_first)
+                         softcap, gate, gate_stride, slopes, keep_first, gate_dim)

@@ -82,9 +82,9 @@ CLASS_OF = {"mb_gemm_tc": "products", "mb_gemm_simt": "products",
             "mb_token_shift": "recurrence", "mb_wkv_scan": "recurrence",
             "mb_mlstm_scan": "recurrence", "mb_tanh": "recurrence",
             "mb_retention_scan": "recurrence", "mb_retention_chunked": "recurrence",
-            "mb_norm_add": "norms", "mb_cast_rows": "norms",
+            "mb_norm_add": "norms", "mb_cast_rows": "norms", "mb_norm_step": "norms",
             "mb_unary_act": "activation", "mb_softcap": "activation",
-            "mb_pass_input": "embedding", "mb_wide_qk_norm": "rotary",
+            "mb_pass_input": "embedding", "mb_wide_qk_norm": "rotary", "mb_rope_store": "rotary",
             "mb_short_conv": "recurrence", "mb_linear_state_scan": "recurrence"}
 
 
@@ -457,6 +457,76 @@ def pass_concat(x: torch.Tensor, terms, table: torch.Tensor, ids: torch.Tensor, 
           [_vp, _vp, _i, _vp, _i, _i, _vp, _f, _vp, _vp, _i, _i, _i, _vp],
           _ptr(x), _c.cast(arr, _vp), n, _ptr(table), code_of(table.dtype), table.shape[0],
           _ptr(ids), float(scale), _ptr(vector), _ptr(both), code_of(both.dtype), T, H, _stream())
+
+
+def norm_step(x: torch.Tensor, y: Optional[torch.Tensor] = None, out_norm=None,
+              h: Optional[torch.Tensor] = None, in_norm=None, rows: Optional[torch.Tensor] = None,
+              n_rows: Optional[int] = None) -> None:
+    """x [T, H] float32 += out_norm(y), then h = in_norm(x); either half may be missing. ``y``
+    float32 [T, H] or [parts, T, H] (the parts may lie in any order in memory): a sublayer's
+    output, added up here. A norm is (w [H], b [H] or None, "layer" or "rms", eps). ``rows``:
+    without y, only these rows are normed (gathered)."""
+    T, H = x.shape
+    _contig(x, "x")
+    assert x.dtype == torch.float32
+    R = n_rows if n_rows is not None else (rows.numel() if rows is not None else T)
+    parts, part_stride, row_stride = 1, 0, H
+    if y is not None:
+        assert y.dtype == torch.float32 and y.shape[-2:] == (T, H) and y.stride(-1) == 1
+        row_stride = y.stride(-2)
+        if y.dim() == 3:
+            parts, part_stride = y.shape[0], y.stride(0)
+    args = []
+    for norm in (out_norm, in_norm):
+        if norm is None:
+            args += [None, None, 0, 0, 0.0]
+            continue
+        w, b, kind, eps = norm
+        assert kind in ("layer", "rms") and w.numel() == H
+        assert b is None or (b.numel() == H and b.dtype == w.dtype)
+        args += [_ptr(w), _ptr(b), 1 if code_of(w.dtype) == BF16 else 0,
+                 1 if kind == "layer" else 0, float(eps)]
+    if h is not None:
+        assert h.shape == (R, H) and h.is_contiguous()
+    _call("norm_step", "mb_norm_step",
+          [_vp, _vp, _i, _ll, _ll, _vp, _vp, _i, _i, _f, _vp, _vp, _i, _i, _f, _vp, _i, _vp, _i, _i,
+           _vp],
+          _ptr(x), _ptr(y), parts, part_stride, row_stride, *args, _ptr(h),
+          code_of(h.dtype) if h is not None else F32, _ptr(rows), R, H, _stream())
+
+
+def rope_store(rows: torch.Tensor, inv_freq: Optional[torch.Tensor], rot_dim: int,
+               amplitude: float, step, line, nh: int, nkv: int, dim: int, vd: int,
+               q_out: torch.Tensor, first: Optional[torch.Tensor] = None,
+               lam: Optional[torch.Tensor] = None,
+               gate_out: Optional[torch.Tensor] = None) -> None:
+    """From the rows [q | k | v | gates] of a product (``rows`` [T, width], or float32 [parts, T,
+    width]: its split sums): q and k rotated (no norm; cosine and sine times ``amplitude``), q
+    into ``q_out`` [T, >= nh * dim] (it may be the rows themselves), k and v into the cache line.
+    ``first`` [T, nkv * vd]: receives the values, or, with ``lam`` (one float32 on the device),
+    is what they are blended with: (1 - lam) v + lam first. ``gate_out`` [T, n]: receives the n
+    columns behind v."""
+    T = q_out.shape[0]
+    parts, stride = (1, 0) if rows.dim() == 2 else (rows.shape[0], rows.stride(0))
+    assert rows.shape[-2] == T and rows.stride(-1) == 1 and q_out.stride(1) == 1
+    assert rows.dim() == 2 or rows.dtype == torch.float32
+    assert line.head_dim == dim and line.kv_heads == nkv
+    assert q_out.dtype == line.k.dtype == line.v.dtype
+    for t in (first, gate_out):
+        assert t is None or (t.dtype == q_out.dtype and t.is_contiguous() and t.shape[0] == T)
+    assert first is None or first.shape[1] == nkv * vd
+    assert lam is None or (lam.dtype == torch.float32 and lam.numel() == 1)
+    if rot_dim > 0 and (inv_freq is None or inv_freq.dtype != torch.float32
+                        or inv_freq.numel() < rot_dim // 2):
+        raise KernelError(f"a rotation of {rot_dim} values without its frequencies")
+    _call("rope", "mb_rope_store",
+          [_vp, _i, _i, _ll, _i, _vp, _i, _f, _vp, _vp, _vp, _i, _i, _vp, _vp, _vp, _i, _i, _vp,
+           _vp, _vp, _i, _i, _i, _i, _i, _i, _vp],
+          _ptr(rows), code_of(rows.dtype), parts, stride, rows.stride(-2), _ptr(inv_freq), rot_dim,
+          float(amplitude), _ptr(step.tok_slot), _ptr(step.tok_pos), _ptr(line.page_table),
+          line.max_pages, line.ring_pages, _ptr(line.k), _ptr(line.v), _ptr(q_out),
+          q_out.stride(0), code_of(q_out.dtype), _ptr(first), _ptr(lam), _ptr(gate_out),
+          gate_out.shape[1] if gate_out is not None else 0, T, nh, nkv, dim, vd, _stream())
 
 
 def wide_qk_norm(qkv: torch.Tensor, qw: int, kw: int, wq: torch.Tensor, wk: torch.Tensor,
@@ -837,24 +907,27 @@ def _parts_of(z: torch.Tensor):
     return z.shape[0], z.stride(0), z.stride(1)
 
 
-ROUTE_SOFTMAX_OF_CHOSEN, ROUTE_SOFTMAX_OF_ALL = 0, 1
+ROUTE_SOFTMAX_OF_CHOSEN, ROUTE_SOFTMAX_OF_ALL, ROUTE_SIGMOID = 0, 1, 2
 
 
 def moe_route(z: torch.Tensor, experts: int, top: int, shared_col: int, ids: torch.Tensor,
               w: torch.Tensor, sg: Optional[torch.Tensor], mode: int = 0,
-              correction: Optional[torch.Tensor] = None, scale: float = 1.0) -> None:
+              correction: Optional[torch.Tensor] = None, scale: float = 1.0,
+              groups: int = 1, keep: int = 1) -> None:
     """Per row of z (float32 router logits, [T, N] or the split sums [parts, T, N] of the
     router's product): the ``top`` largest of the first ``experts`` columns into ``ids`` and
-    the softmax over them into ``w``; ``sg`` = sigmoid of column ``shared_col``."""
+    the softmax over them into ``w``; ``sg`` = sigmoid of column ``shared_col``. ``mode``: other
+    scores (a softmax over all columns, a sigmoid each), chosen with ``correction`` added and
+    weighted without it; then only columns of the ``keep`` best of ``groups`` can be chosen."""
     parts, stride, ldz = _parts_of(z)
     assert ids.dtype == torch.int32 and w.dtype == torch.float32
     assert correction is None or (correction.dtype == torch.float32
                                   and correction.numel() == experts)
     _call("moe", "mb_moe_route",
-          [_vp, _i, _i, _ll, _i, _i, _i, _vp, _vp, _vp, _i, _i, _vp, _f, _vp],
+          [_vp, _i, _i, _ll, _i, _i, _i, _vp, _vp, _vp, _i, _i, _vp, _f, _i, _i, _vp],
           _ptr(z), ldz, parts, stride, experts, top, shared_col if sg is not None else -1,
-          _ptr(ids), _ptr(w), _ptr(sg), z.shape[-2], mode, _ptr(correction), float(scale),
-          _stream())
+          _ptr(ids), _ptr(w), _ptr(sg), z.shape[-2], mode, _ptr(correction), float(scale), groups,
+          keep, _stream())
 
 
 def moe_plan(ids: torch.Tensor, experts: int, bm: int, max_tiles: int,
@@ -880,7 +953,8 @@ def moe_table_plan(table: torch.Tensor, tok_ids: torch.Tensor, experts: int, bm:
 def moe_route_plan(z: torch.Tensor, experts: int, top: int, shared_col: int, ids: torch.Tensor,
                    w: torch.Tensor, sg: Optional[torch.Tensor], bm: int, max_tiles: int,
                    plan: torch.Tensor, mode: int = 0, correction: Optional[torch.Tensor] = None,
-                   scale: float = 1.0, routed: Optional[int] = None) -> None:
+                   scale: float = 1.0, routed: Optional[int] = None, groups: int = 1,
+                   keep: int = 1) -> None:
     """``moe_route`` and ``moe_plan`` as one kernel, for a step of at most 64 tokens.
     ``routed``: the columns that the router chooses among (``experts`` of them have lists;
     those after them are identity experts)."""
@@ -888,10 +962,11 @@ def moe_route_plan(z: torch.Tensor, experts: int, top: int, shared_col: int, ids
     assert ids.dtype == torch.int32 and w.dtype == torch.float32
     assert plan.dtype == torch.int32 and plan.numel() >= 2 + experts + ids.numel() + 2 * max_tiles
     _call("moe", "mb_moe_route_plan",
-          [_vp, _i, _i, _ll, _i, _i, _i, _vp, _vp, _vp, _i, _i, _i, _vp, _i, _vp, _f, _i, _vp],
+          [_vp, _i, _i, _ll, _i, _i, _i, _vp, _vp, _vp, _i, _i, _i, _vp, _i, _vp, _f, _i, _i, _i, _vp],
           _ptr(z), ldz, parts, stride, experts, top, shared_col if sg is not None else -1,
           _ptr(ids), _ptr(w), _ptr(sg), z.shape[-2], bm, max_tiles, _ptr(plan), mode,
-          _ptr(correction), float(scale), routed if routed is not None else experts, _stream())
+          _ptr(correction), float(scale), groups, keep,
+          routed if routed is not None else experts, _stream())
 
 
 def moe_gemm(src: torch.Tensor, w: torch.Tensor, out: torch.Tensor, plan: torch.Tensor,
@@ -1102,12 +1177,14 @@ def attention_simt(q: torch.Tensor, q_stride: int, out: torch.Tensor, step, line
                    window: int, scale: float, vd: int = 0,
                    sink: Optional[torch.Tensor] = None, softcap: float = 0.0,
                    gate: Optional[torch.Tensor] = None, gate_stride: int = 0,
-                   slopes: Optional[torch.Tensor] = None, keep_first: int = 0) -> None:
+                   slopes: Optional[torch.Tensor] = None, keep_first: int = 0,
+                   gate_dim: int = 0) -> None:
     """``vd``: the size of a value row when it differs from ``hd``. ``sink``: float32 [nh],
     one more term exp(sink[h]) in the softmax denominators of head h. ``softcap`` > 0: scores
     become softcap * tanh(score / softcap). ``gate``: logits of q's type, head h of token t at
-    ``gate[t * gate_stride + h]``; the head's output is multiplied by their sigmoid.
-    ``slopes``: float32 [nh]; slopes[h] * (distance of key and query) is taken off head h's
+    ``gate[t * gate_stride + h]``; the head's output is multiplied by their sigmoid. With
+    ``gate_dim`` (the size of a value row) there is one for every value of the head, at
+    ``gate[t * gate_stride + h * gate_dim + d]``. ``slopes``: float32 [nh]; slopes[h] * (distance of key and query) is taken off head h's
     scores after the cap. ``keep_first``: with a window, the first so many positions of a
     sequence stay visible (the line must then keep all pages, not a ring)."""
     T = out.shape[0]
@@ -1118,12 +1195,12 @@ def attention_simt(q: torch.Tensor, q_stride: int, out: torch.Tensor, step, line
     assert keep_first == 0 or line.ring_pages == 0
     _call("attention_simt", "mb_attention_simt",
           [_vp, _i, _vp, _i, _vp, _vp, _i, _vp, _i, _i, _vp, _vp, _vp, _i, _i, _i, _i, _i, _f,
-           _i, _vp, _f, _vp, _i, _vp, _i, _vp],
+           _i, _vp, _f, _vp, _i, _i, _vp, _i, _vp],
           _ptr(q), q_stride, _ptr(out), out.stride(0), _ptr(line.k), _ptr(line.v),
           code_of(out.dtype), _ptr(line.page_table), line.max_pages, line.ring_pages,
           _ptr(step.tok_seq), _ptr(step.tok_pos), _ptr(step.seq_slot), T, nh, nkv, hd,
           window, float(scale), vd or hd, _ptr(sink), float(softcap), _ptr(gate), gate_stride,
-          _ptr(slopes), int(keep_first), _stream())
+          int(gate_dim), _ptr(slopes), int(keep_first), _stream())
 
 
 # ------------------------------------------------------------------------------ sampling
@@ -1190,10 +1267,11 @@ def gemm_tc(a: torch.Tensor, w: torch.Tensor, c: torch.Tensor, add: bool,
 
 
 def gemm_tc_gated(a: torch.Tensor, w: torch.Tensor, c: torch.Tensor, act: int,
-                  pair_bias: Optional[torch.Tensor], error: torch.Tensor, sms: int) -> None:
+                  pair_bias: Optional[torch.Tensor], error: torch.Tensor, sms: int,
+                  limit: float = 0.0) -> None:
     """c [M, N / 2] = act(gate + bias) * (up + bias) for a bfloat16 weight [N, K] whose rows
     alternate gate and up (``pair_bias`` [N] bfloat16 alternates likewise, or None), in the
-    epilogue of the tensor-core product."""
+    epilogue of the tensor-core product. ``limit``: of ACT_CLAMPED_SWISH."""
     M, Kd = a.shape
     N = w.shape[0]
     assert a.dtype == w.dtype == c.dtype == torch.bfloat16 and w.shape[1] == Kd
@@ -1201,9 +1279,9 @@ def gemm_tc_gated(a: torch.Tensor, w: torch.Tensor, c: torch.Tensor, act: int,
     _contig(w, "the weight")
     if pair_bias is not None:
         assert pair_bias.dtype == torch.bfloat16 and pair_bias.numel() == N
-    _call("gemm_tc", "mb_gemm_tc_gated", [_vp, _i, _vp, _vp, _i, _i, _i, _i, _i, _vp, _vp, _i, _vp],
+    _call("gemm_tc", "mb_gemm_tc_gated", [_vp, _i, _vp, _vp, _i, _i, _i, _i, _i, _vp, _f, _vp, _i, _vp],
           _ptr(a), a.stride(0), _ptr(w), _ptr(c), c.stride(0), M, N, Kd, act, _ptr(pair_bias),
-          _ptr(error), sms, _stream())
+          float(limit), _ptr(error), sms, _stream())
 
 
 def wait_selftest(error: torch.Tensor, code: int, tries: int = 2048) -> bool:
@@ -1246,10 +1324,11 @@ def attention_decode(q: torch.Tensor, q_stride: int, out: torch.Tensor, step, li
                      error: Optional[torch.Tensor] = None,
                      sink: Optional[torch.Tensor] = None, softcap: float = 0.0,
                      gate: Optional[torch.Tensor] = None, gate_stride: int = 0,
-                     slopes: Optional[torch.Tensor] = None, keep_first: int = 0) -> None:
+                     slopes: Optional[torch.Tensor] = None, keep_first: int = 0,
+                     gate_dim: int = 0, vd: int = 0) -> None:
     """Attention of single tokens (a decode step) over the paged cache on the tensor cores; the
-    pages of a sequence are dealt out over ``splits`` CTAs. ``softcap``, ``gate``, ``slopes``
-    and ``keep_first`` as for ``attention_simt``."""
+    pages of a sequence are dealt out over ``splits`` CTAs. ``softcap``, ``gate``, ``gate_dim``,
+    ``slopes``, ``keep_first`` and ``vd`` as for ``attention_simt``."""
     T = out.shape[0]
     _contig(out, "out")
     assert q.dtype == torch.bfloat16 and out.dtype == torch.bfloat16
@@ -1257,12 +1336,13 @@ def attention_decode(q: torch.Tensor, q_stride: int, out: torch.Tensor, step, li
     assert gate is None or gate.dtype == torch.bfloat16
     _call("attention_mma", "mb_attention_decode",
           [_vp, _i, _vp, _i, _vp, _vp, _vp, _i, _i, _vp, _vp, _i, _i, _i, _i, _i, _f, _i,
-           _vp, _ll, _vp, _vp, _f, _vp, _i, _vp, _i, _vp],
+           _vp, _ll, _vp, _vp, _f, _vp, _i, _i, _vp, _i, _i, _vp],
           _ptr(q), q_stride, _ptr(out), out.stride(0), _ptr(line.k), _ptr(line.v),
           _ptr(line.page_table), line.max_pages, line.ring_pages, _ptr(step.tok_slot),
           _ptr(step.tok_pos), T, nh, nkv, hd, window, float(scale),
           splits, _ptr(scratch), scratch.numel(), _ptr(error), _ptr(sink), float(softcap),
-          _ptr(gate), gate_stride, _ptr(slopes), int(keep_first), _stream(), launches=2)
+          _ptr(gate), gate_stride, int(gate_dim), _ptr(slopes), int(keep_first), int(vd),
+          _stream(), launches=2)
 
 
 def attention_decode_clusters(q: torch.Tensor, q_stride: int, out: torch.Tensor, step, line, nh,
@@ -1271,7 +1351,7 @@ def attention_decode_clusters(q: torch.Tensor, q_stride: int, out: torch.Tensor,
                               sink: Optional[torch.Tensor] = None, softcap: float = 0.0,
                               gate: Optional[torch.Tensor] = None, gate_stride: int = 0,
                               slopes: Optional[torch.Tensor] = None,
-                              keep_first: int = 0) -> None:
+                              keep_first: int = 0, gate_dim: int = 0, vd: int = 0) -> None:
     """``attention_decode`` with the splits of a (token, group of heads) as one thread-block
     cluster that merges through its shared memory: no scratch, one kernel; at most 8 splits."""
     T = out.shape[0]
@@ -1280,12 +1360,12 @@ def attention_decode_clusters(q: torch.Tensor, q_stride: int, out: torch.Tensor,
     assert gate is None or gate.dtype == torch.bfloat16
     _call("attention_mma", "mb_attention_decode_clusters",
           [_vp, _i, _vp, _i, _vp, _vp, _vp, _i, _i, _vp, _vp, _i, _i, _i, _i, _i, _f, _i,
-           _vp, _vp, _f, _vp, _i, _vp, _i, _vp],
+           _vp, _vp, _f, _vp, _i, _i, _vp, _i, _i, _vp],
           _ptr(q), q_stride, _ptr(out), out.stride(0), _ptr(line.k), _ptr(line.v),
           _ptr(line.page_table), line.max_pages, line.ring_pages, _ptr(step.tok_slot),
           _ptr(step.tok_pos), T, nh, nkv, hd, window, float(scale), splits, _ptr(error),
-          _ptr(sink), float(softcap), _ptr(gate), gate_stride, _ptr(slopes), int(keep_first),
-          _stream())
+          _ptr(sink), float(softcap), _ptr(gate), gate_stride, int(gate_dim), _ptr(slopes),
+          int(keep_first), int(vd), _stream())
 
 
 def attention_prefill(q: torch.Tensor, q_stride: int, out: torch.Tensor, step, line, nh, nkv,
@@ -1293,7 +1373,8 @@ def attention_prefill(q: torch.Tensor, q_stride: int, out: torch.Tensor, step, l
                       error: Optional[torch.Tensor] = None,
                       sink: Optional[torch.Tensor] = None, softcap: float = 0.0,
                       gate: Optional[torch.Tensor] = None, gate_stride: int = 0,
-                      slopes: Optional[torch.Tensor] = None, keep_first: int = 0) -> None:
+                      slopes: Optional[torch.Tensor] = None, keep_first: int = 0,
+                      gate_dim: int = 0, vd: int = 0) -> None:
     """Causal attention of every sequence's new tokens over the paged cache on the tensor
     cores (the cache already holds their keys and values)."""
     _contig(out, "out")
@@ -1301,19 +1382,20 @@ def attention_prefill(q: torch.Tensor, q_stride: int, out: torch.Tensor, step, l
     assert gate is None or gate.dtype == torch.bfloat16
     _call("attention_mma", "mb_attention_prefill",
           [_vp, _i, _vp, _i, _vp, _vp, _vp, _i, _i, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _f,
-           _vp, _vp, _f, _vp, _i, _vp, _i, _vp],
+           _vp, _vp, _f, _vp, _i, _i, _vp, _i, _i, _vp],
           _ptr(q), q_stride, _ptr(out), out.stride(0), _ptr(line.k), _ptr(line.v),
           _ptr(line.page_table), line.max_pages, line.ring_pages, _ptr(step.seq_start),
           _ptr(step.seq_past), _ptr(step.seq_slot), step.B, step.max_new, nh, nkv, hd, window,
           float(scale), _ptr(error), _ptr(sink), float(softcap), _ptr(gate), gate_stride,
-          _ptr(slopes), int(keep_first), _stream())
+          int(gate_dim), _ptr(slopes), int(keep_first), int(vd), _stream())
 
 
 def attention_prefill_tc(q: torch.Tensor, q_stride: int, out: torch.Tensor, step, line, nh, nkv,
                          hd, window: int, scale: float, error: torch.Tensor,
                          sink: Optional[torch.Tensor] = None, softcap: float = 0.0,
-                         gate: Optional[torch.Tensor] = None, gate_stride: int = 0) -> None:
-    """The prefill attention on tcgen05 (heads of 128 values): S and O in tensor memory, Q, K
+                         gate: Optional[torch.Tensor] = None, gate_stride: int = 0,
+                         gate_dim: int = 0, vd: int = 0) -> None:
+    """The prefill attention on tcgen05 (heads of 128 values, value rows of 128 or 64): S and O in tensor memory, Q, K
     and V tiles by TMA."""
     _contig(out, "out")
     assert q.dtype == torch.bfloat16 and out.dtype == torch.bfloat16 and q.stride(1) == 1
@@ -1321,9 +1403,9 @@ def attention_prefill_tc(q: torch.Tensor, q_stride: int, out: torch.Tensor, step
     pool_rows = line.k.shape[0] * line.k.shape[1] * line.k.shape[2]
     _call("attention_tc", "mb_attention_prefill_tc",
           [_vp, _i, _i, _vp, _i, _vp, _vp, _ll, _vp, _i, _i, _vp, _vp, _vp, _i, _i, _i, _i, _i,
-           _i, _i, _f, _vp, _vp, _f, _vp, _i, _vp],
+           _i, _i, _f, _vp, _vp, _f, _vp, _i, _i, _i, _vp],
           _ptr(q), q_stride, nh * hd, _ptr(out), out.stride(0), _ptr(line.k), _ptr(line.v),
           pool_rows, _ptr(line.page_table), line.max_pages, line.ring_pages,
           _ptr(step.seq_start), _ptr(step.seq_past), _ptr(step.seq_slot), step.B, q.shape[0],
           step.max_new, nh, nkv, hd, window, float(scale), _ptr(error), _ptr(sink),
-          float(softcap), _ptr(gate), gate_stride, _stream())
+          float(softcap), _ptr(gate), gate_stride, int(gate_dim), int(vd), _stream())

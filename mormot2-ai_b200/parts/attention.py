@@ -20,7 +20,11 @@ n positions of a sequence stay visible to all later ones (the cache line then ke
 page instead of a ring); ``head_norm`` = "whole_rows": q and k are each normed over their
 whole projection at once, with weights of that width; ``values`` = "keys_as_projected": there
 is no value projection, a token's values are its keys as they leave the projection (before any
-norm or rotation).
+norm or rotation); ``gate`` = "value" with ``names["g"]``: a logit for every value of the
+concatenated heads instead of one per head; ``value_mix``: values are blended across layers, the
+first layer that takes part ("first") keeps its values of the step, every later one ("blend")
+stores (1 − l) v + l v_first with a learned number l (``names["vmix"]``). These two, and an
+encoding whose cosine and sine carry a factor, come without norms of q and k.
 """
 from __future__ import annotations
 
@@ -84,13 +88,31 @@ class GqaAttention(Part):
         self.unit_after = self.head_norm == "unit_after_rotation"
         if self.unit_after and ("q_norm" in self.names or self.head_norm_eps is None):
             raise ConfigError("a unit norm after the rotation has an eps and no weights")
-        self.gate_n = self.nh if "g" in self.names else 0
+        self.gate_per = p.get("gate", "head")
+        if self.gate_per not in ("head", "value"):
+            raise ConfigError(f"a gate per \"{self.gate_per}\" (head, value)")
+        self.gate_n = 0
+        if "g" in self.names:
+            self.gate_n = self.nh if self.gate_per == "head" else self.ow
+        self.gate_dim = self.vd if self.gate_n and self.gate_per == "value" else 0
+        self.value_mix = p.get("value_mix")
+        if self.value_mix not in (None, "first", "blend"):
+            raise ConfigError(f"values mixed as \"{self.value_mix}\" (first, blend)")
+        self.amplitude = float(getattr(self.position, "amplitude", 1.0))
+        # q, k and v as they leave the projection, apart from the rotation and the blend
+        self.bare = bool(self.gate_dim or self.value_mix or self.amplitude != 1.0)
+        if self.bare and ("q_norm" in self.names or self.unit_after or self.v_from_k):
+            raise ConfigError("a gate per value, values mixed across layers or an amplified "
+                              "rotation with norms of q and k or with values from keys")
         # the gates' columns stand behind q (k, v) in the projection's rows: rows of zeros after
         # them keep those rows a multiple of 16 bytes wide, which the tensor-core kernels ask for
         self.gate_w = self.gate_n
         if self.gate_n and self.qw % 8 == 0 and (self.kvw + self.vw) % 8 == 0:
             self.gate_w = (self.gate_n + 7) // 8 * 8
         self.shared_kv = bool(p.get("shared_kv", False))
+        if self.bare and self.shared_kv:
+            raise ConfigError("a gate per value, values mixed across layers or an amplified "
+                              "rotation with another layer's keys and values")
 
     can_store = True      # forward(..., store=True) writes its output into x instead of adding
 
@@ -106,7 +128,9 @@ class GqaAttention(Part):
                 out.append(TensorNeed(n["v"], (self.vw, self.hidden)))
         out.append(TensorNeed(n["o"], (self.hidden, self.ow)))
         if self.gate_n:
-            out.append(TensorNeed(n["g"], (self.nh, self.hidden)))
+            out.append(TensorNeed(n["g"], (self.gate_n, self.hidden)))
+        if self.value_mix:      # the first layer's number is stored but never used
+            out.append(TensorNeed(n["vmix"], (), "fraction", optional=self.value_mix == "first"))
         if "sink" in n:
             out.append(TensorNeed(n["sink"], (self.nh,), "bias"))
         if "q_norm" in n:
@@ -124,7 +148,7 @@ class GqaAttention(Part):
         plain = (self.vd == self.hd and "sink" not in self.names and not self.softcap
                  and not self.gate_n and not self.unit_after and self.sink_value is None
                  and self.distance_exponent is None and not self.whole_rows
-                 and not self.v_from_k and not self.keep_first)
+                 and not self.v_from_k and not self.keep_first and not self.bare)
         if self.sink_value is not None:
             self.sink = torch.full((self.nh,), float(self.sink_value), dtype=torch.float32,
                                    device=rt.device)
@@ -179,6 +203,8 @@ class GqaAttention(Part):
         self.k_norm = weights.get(n.get("k_norm", ""))
         if "sink" in n:
             self.sink = weights[n["sink"]].to(torch.float32).contiguous()
+        if self.value_mix == "blend":     # stays on the device
+            self.lam = weights[n["vmix"]].to(torch.float32).reshape(1).contiguous()
 
     @property
     def q_only(self) -> Linear:
@@ -210,7 +236,12 @@ class GqaAttention(Part):
                     and self.vd == self.hd and not self.gate_n and not self.whole_rows
                     and not self.v_from_k)
         more = {"slopes": self.slopes, "keep_first": self.keep_first}
-        qkv = self.qkv(h, defer=True) if split_ok else None
+        if self.bare and not writes_cache:
+            raise ConfigError("a gate per value, values mixed across layers or an amplified "
+                              "rotation with a borrowed cache line")
+        qkv = self.qkv(h, defer=True) if (split_ok or self.bare and self.qkv is not None) else None
+        if self.bare and isinstance(qkv, Pending):
+            return self._bare(qkv.partial, None, inv_freq, rot_dim, T, step, line, x, store, more)
         if isinstance(qkv, Pending):
             # the kernel that norms and rotates q and k adds the split sums up as it reads them
             q = torch.empty((T, self.qw), dtype=self.rt.dtype, device=h.device)
@@ -238,6 +269,8 @@ class GqaAttention(Part):
             self.split[1](h, out=qkv[:, self.qw:self.qw + self.kvw])
             if not self.v_from_k:
                 self.split[2](h, out=qkv[:, self.qw + self.kvw:])
+        if self.bare:
+            return self._bare(qkv, qkv, inv_freq, rot_dim, T, step, line, x, store, more)
         q_norm, k_norm = self.q_norm, self.k_norm
         if self.whole_rows or self.v_from_k:
             if not writes_cache:
@@ -256,6 +289,35 @@ class GqaAttention(Part):
                           softcap=self.softcap,
                           gate=qkv[:, heads_width:] if self.gate_n else None, gate_stride=width,
                           **more)
+        return self._project(attn, x, store)
+
+    def _bare(self, rows, in_place, inv_freq, rot_dim, T, step, line, x, store, more):
+        """From the product's rows [q | k | v | gates] (``in_place``: the same rows, in which q
+        is rotated and the gates are read; None: ``rows`` are split sums)."""
+        dev, dt = rows.device, self.rt.dtype
+        first = lam = gate_out = gate = None
+        if self.value_mix == "first":
+            first = torch.empty((T, self.vw), dtype=dt, device=dev)
+            step.memo["first_values"] = first
+        elif self.value_mix == "blend":
+            first, lam = step.memo.get("first_values"), self.lam
+            if first is None or first.shape != (T, self.vw):
+                raise ConfigError("values are blended with those of a layer that has not run "
+                                  "or has others of another size")
+        q = in_place
+        if q is None:
+            q = torch.empty((T, self.qw), dtype=dt, device=dev)
+            if self.gate_n:
+                gate = gate_out = torch.empty((T, self.gate_n), dtype=dt, device=dev)
+        elif self.gate_n:
+            gate = q[:, self.qw + self.kvw + self.vw:]
+        K.rope_store(rows, inv_freq, rot_dim, self.amplitude, step, line, self.nh, self.nkv,
+                     self.hd, self.vd, q, first, lam, gate_out)
+        attn = torch.empty((T, self.ow), dtype=dt, device=dev)
+        self.rt.attention(q, q.stride(0), attn, step, line, self.nh, self.nkv, self.hd, self.window,
+                          self.scale, vd=self.vd, sink=self.sink, softcap=self.softcap, gate=gate,
+                          gate_stride=gate.stride(0) if gate is not None else 0,
+                          gate_dim=self.gate_dim, **more)
         return self._project(attn, x, store)
 
     def _project(self, attn, x, store: bool):

@@ -8,7 +8,7 @@ import torch
 from .. import kernels as K
 from ..cache.pages import pages_for
 
-FAST_HEAD_DIMS = (64, 128)
+FAST_HEAD_MOST = 128        # query/key and value sizes: multiples of 8 up to this
 MAX_DECODE_SPLITS = 8       # the splits of a sequence are one thread-block cluster
 
 
@@ -48,23 +48,28 @@ def decode_many_splits(step, nh: int, nkv: int, sms: int) -> int:
 
 def run(rt, q, q_stride, out, step, line, nh, nkv, hd, window, scale, sink=None,
         softcap: float = 0.0, gate=None, gate_stride: int = 0, slopes=None,
-        keep_first: int = 0) -> bool:
+        keep_first: int = 0, vd: int = 0, gate_dim: int = 0) -> bool:
     """True if a fast kernel took the call; False: the caller uses the general kernel.
     ``sink``: float32 [nh], one more term exp(sink[h]) in every softmax denominator.
     ``softcap`` > 0: scores become softcap * tanh(score / softcap); ``gate``: bfloat16 logits,
     head h of token t at ``gate[t * gate_stride + h]``, whose sigmoid multiplies the head's
-    output. ``slopes`` (float32 [nh], a bias slopes[h] * distance taken off the scores) and
+    output, or with ``gate_dim`` (the size of a value row) one for every value. ``vd``: the size
+    of a value row (0: ``hd``). ``slopes`` (float32 [nh], a bias slopes[h] * distance taken off the scores) and
     ``keep_first`` (positions at a sequence's start that a window never loses) are served by
     the ``mma.sync`` kernels; the tcgen05 prefill kernel does not take them."""
-    if hd not in FAST_HEAD_DIMS or q.dtype != torch.bfloat16 or q_stride % 8 or q.data_ptr() % 16:
+    vd = vd or hd
+    if (max(hd, vd) > FAST_HEAD_MOST or hd % 8 or vd % 8 or q.dtype != torch.bfloat16
+            or q_stride % 8 or q.data_ptr() % 16):
+        return False
+    if gate is not None and gate_dim and (gate_stride % 8 or gate.data_ptr() % 16):
         return False
     if scale <= 0 or (gate is not None and gate.dtype != torch.bfloat16):
         return False
-    more = (softcap, gate, gate_stride, slopes, keep_first)
+    more = (softcap, gate, gate_stride, slopes, keep_first, gate_dim, vd)
     plain_mask = slopes is None and not keep_first
     if step.decode:
         many = decode_many_splits(step, nh, nkv, rt.sms) if window == 0 else 0
-        if many > MAX_DECODE_SPLITS and step.T * nh * many * (hd + 2) <= rt.attention_scratch.numel():
+        if many > MAX_DECODE_SPLITS and step.T * nh * many * (vd + 2) <= rt.attention_scratch.numel():
             K.attention_decode(q, q_stride, out, step, line, nh, nkv, hd, window, scale, many,
                                rt.attention_scratch, rt.error_word, sink, *more)
             return True
@@ -74,10 +79,10 @@ def run(rt, q, q_stride, out, step, line, nh, nkv, hd, window, scale, sink=None,
         return True
     if out.stride(0) % 8 or out.data_ptr() % 16:
         return False
-    if hd == 128 and q.stride(1) == 1 and plain_mask:
+    if hd == 128 and vd in (64, 128) and q.stride(1) == 1 and plain_mask:
         # S and O in tensor memory, tiles by TMA (csrc/attention_tc.cu)
         K.attention_prefill_tc(q, q_stride, out, step, line, nh, nkv, hd, window, scale,
-                               rt.error_word, sink, softcap, gate, gate_stride)
+                               rt.error_word, sink, softcap, gate, gate_stride, gate_dim, vd)
         return True
     K.attention_prefill(q, q_stride, out, step, line, nh, nkv, hd, window, scale,
                         rt.error_word, sink, *more)

@@ -23,6 +23,11 @@ which it is handed on as pending) reads. With ``side`` the block then adds an in
 from the token: e = columns [col0, col0 + dim) of the row of a second embedding table,
 t = P (act(G x) * e), x += norm_side(t).
 
+``sandwich_residual``: norms on both sides of a sublayer: x += norm_mixer_out(mixer(
+norm_mixer(x))); x += norm_ff_out(feed_forward(norm_ff(x))). A sublayer's output stays beside the
+residual (stored, as split sums, or as the rows of a token's experts) until the next norm reads the
+residual: one kernel adds the output up, norms it, adds it into x and norms x (``NormedOutput``).
+
 ``parallel_residual``: both sublayers read one norm of the residual and are added at once, each
 times a vector and all times a constant:
 h = norm_input(x); x += factor * (scales_mixer * mixer(h) + scales_ff * feed_forward(h)). The
@@ -304,6 +309,76 @@ class OutputNormResidualBlock(Part):
         return ReadyInput(h) if h is not x else None
 
 
+class NormedOutput:
+    """A sublayer's output that is still to be normed and added: x += norm(y), y float32 [T, H] or
+    [parts, T, H] (the parts may lie in any order in memory)."""
+
+    def __init__(self, y, norm):
+        self.y, self.norm = y, norm
+
+    def settle(self, x) -> None:
+        from .. import kernels as K
+        K.norm_step(x, self.y, self.norm.terms())
+
+
+class SandwichResidualBlock(Part):
+    capturable = True
+    accepts_pending = True
+
+    def __init__(self, spec, prefix: str = "", mixer=None, feed_forward=None, norms=None):
+        super().__init__(spec, prefix)
+        self.mixer, self.feed_forward, self.norms = mixer, feed_forward, norms
+        self.with_ff = bool(spec.params.get("feed_forward", True))
+        for q in ("mixer", "mixer_out") + (("feed_forward", "feed_forward_out") if self.with_ff else ()):
+            if not hasattr(norms.get(q), "terms"):
+                raise ConfigError(f"norms on both sides of a sublayer: \"{q}\" is missing or "
+                                  "cannot be one (layernorm, rmsnorm)")
+
+    def libraries(self, rt):
+        return ["norm_step"]
+
+    def bind(self, weights, rt) -> None:
+        self.rt = rt
+
+    def _operand(self, which, x, pending):
+        """norm(x) in the activation type, after what is pending has been added into x."""
+        from .. import kernels as K
+        h = torch.empty(x.shape, dtype=self.rt.dtype, device=x.device)
+        if isinstance(pending, NormedOutput):
+            K.norm_step(x, pending.y, pending.norm.terms(), h, self.norms[which].terms())
+            return h
+        if pending is not None:
+            settle(x, pending)
+        K.norm_step(x, h=h, in_norm=self.norms[which].terms())
+        return h
+
+    def _sublayer(self, part, h, args):
+        """The sublayer's output as float32 [T, hidden] or [parts, T, hidden]."""
+        if hasattr(part, "forward_parts"):
+            y = part.forward_parts(h, *args)
+            if y is not None:
+                return y
+        y = torch.empty((h.shape[0], h.shape[1]), dtype=torch.float32, device=h.device)
+        if getattr(part, "can_store", False):
+            pending = part.forward(h, y, *args, store=True)
+            return pending.partial if pending is not None else y
+        y.zero_()
+        pending = part.forward(h, y, *args)
+        if pending is not None:
+            settle(y, pending)
+        return y
+
+    def forward(self, x, step, line, state, writes_cache: bool, pending=None):
+        h = self._operand("mixer", x, pending)
+        y = self._sublayer(self.mixer, h, (step, line, state, writes_cache))
+        pending = NormedOutput(y, self.norms["mixer_out"])
+        if not self.with_ff:
+            return pending
+        h = self._operand("feed_forward", x, pending)
+        y = self._sublayer(self.feed_forward, h, (step,))
+        return NormedOutput(y, self.norms["feed_forward_out"])
+
+
 class ParallelResidualBlock(Part):
     capturable = True
     accepts_pending = True
@@ -356,5 +431,6 @@ class ParallelResidualBlock(Part):
 
 BLOCKS.register("prenorm_residual", PreNormResidualBlock)
 BLOCKS.register("parallel_residual", ParallelResidualBlock)
+BLOCKS.register("sandwich_residual", SandwichResidualBlock)
 BLOCKS.register("output_norm_residual", OutputNormResidualBlock)
 BLOCKS.register("hyper_connections", HyperConnectionsBlock)

@@ -1,7 +1,8 @@
 """Feed-forwards without routing.
 
 ``gated_mlp``: x += W_d (act(W_g h + b_g) * (W_u h + b_u)) + b_d with ``activation`` "silu" or
-"gelu_tanh" and optional biases. Gate and up are one product. In bfloat16 their rows
+"gelu_tanh" (or "clamped_swish" with ``limit``: g' sigmoid(1.702 g') (u' + 1) with
+g' = min(W_g h, limit) and u' = W_u h cut to [−limit, limit]) and optional biases. Gate and up are one product. In bfloat16 their rows
 alternate and the product's epilogue adds the biases and applies the activation (as the
 SwiGLU feed-forward does for SiLU without biases); b_d is placed in the residual rows, which
 the last product then accumulates onto, by the norm before the feed-forward where that norm
@@ -71,6 +72,7 @@ class SwiGluFfn(Part):
 
 class GatedMlp(Part):
     capturable = True
+    can_store = True      # forward(..., store=True) writes its output into x instead of adding
 
     def __init__(self, spec, prefix: str = ""):
         super().__init__(spec, prefix)
@@ -81,6 +83,7 @@ class GatedMlp(Part):
             raise ConfigError(f"activation \"{p['activation']}\" is not known "
                               f"(known: {', '.join(sorted(K.ACTIVATIONS))})")
         self.act = K.ACTIVATIONS[p["activation"]]
+        self.limit = float(p.get("limit", 0.0))
         self.bias = bool(p.get("bias", False))
         self.names = {k: prefix + v for k, v in p["names"].items()}
 
@@ -114,7 +117,8 @@ class GatedMlp(Part):
             pairs = torch.stack([g, u], dim=1).reshape(2 * self.inter, self.hidden)
             pair_bias = (torch.stack(self.biases[:2], dim=1).reshape(-1).contiguous()
                          if self.biases is not None else None)
-            self.gate_up = Linear(pairs, rt, swiglu=True, activation=self.act, pair_bias=pair_bias)
+            self.gate_up = Linear(pairs, rt, swiglu=True, activation=self.act, pair_bias=pair_bias,
+                                  limit=self.limit)
             self.fused = self.gate_up.fast is not None
         if not self.fused:
             self.gate_up = Linear(torch.cat([g, u], dim=0), rt)  # gate rows, then up rows
@@ -126,9 +130,16 @@ class GatedMlp(Part):
         # what the norm before this feed-forward may add into the residual for it
         self.residual_bias = self.biases[2] if (self.fused and self.biases is not None) else None
 
-    def forward(self, h, x, step, bias_placed: bool = False):
-        """``bias_placed``: the norm before already added ``residual_bias`` into x."""
+    def forward(self, h, x, step, bias_placed: bool = False, store: bool = False,
+                settled: bool = False):
+        """``bias_placed``: the norm before already added ``residual_bias`` into x. ``store``: x
+        receives the output instead of a sum onto it, or the split sums are returned and x is
+        left as it is. ``settled``: nothing is left pending."""
         from .linear import Pending
+        if store and self.biases is not None:
+            x.zero_()
+            self.forward(h, x, step, settled=True)
+            return None
         if self.fused:
             act = self.gate_up(h)
             if self.residual_bias is not None and not bias_placed:
@@ -139,8 +150,11 @@ class GatedMlp(Part):
             if self.biases is not None:
                 K.gated_act(gu, act, self.act, self.biases[0], self.biases[1], x, self.biases[2])
             else:
-                K.gated_act(gu, act, self.act)
-        out = self.down(act, add_into=x, defer=True)
+                K.gated_act(gu, act, self.act, limit=self.limit)
+        if store:
+            out = self.down(act, out=x, defer="any")
+        else:
+            out = self.down(act, add_into=x, defer=not settled)
         return out if isinstance(out, Pending) else None
 
 

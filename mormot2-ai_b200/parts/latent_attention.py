@@ -46,6 +46,8 @@ class LatentAttention(Part):
         if min(self.nh, self.dim, self.vd, self.kvr, self.qr) <= 0 or self.rd < 0:
             raise ConfigError(f"latent attention with sizes {p}")
 
+    can_store = True      # forward(..., store=True) writes its output into x instead of adding
+
     def libraries(self, rt) -> List[str]:
         return ["latent", "latent_mma"] if rt.fast_kernels else ["latent"]
 
@@ -99,7 +101,7 @@ class LatentAttention(Part):
             for key in ["dq", "dkv", "uk"] + (["g"] if self.gated else []):
                 weights.pop(n[key], None)
 
-    def forward(self, h, x, step, line, state, writes_cache: bool):
+    def forward(self, h, x, step, line, state, writes_cache: bool, store: bool = False):
         T, dev, dt = h.shape[0], h.device, self.rt.dtype
         nh, dim, rd, vd, kvr, qr = self.nh, self.dim, self.rd, self.vd, self.kvr, self.qr
         inv_freq, rot_dims = (self.position.frequencies() if self.position is not None
@@ -128,7 +130,10 @@ class LatentAttention(Part):
         self.rt.latent_attention(ql, ol, step, line, nh, kvr, rd, self.window, self.scale)
         heads = torch.empty((T, nh * vd), dtype=dt, device=dev)
         K.heads_gemm(ol, kvr, self.uv, heads, vd, gate=gate)
-        out = self.o(heads, add_into=x, defer=True)
+        if store:       # stored into x, or left pending (x is then not touched)
+            out = self.o(heads, out=x, defer="any")
+        else:
+            out = self.o(heads, add_into=x, defer=True)
         return out if isinstance(out, Pending) else None
 
 

@@ -27,12 +27,14 @@ class Pending:
 
 class Linear:
     def __init__(self, weight: torch.Tensor, rt, swiglu: bool = False, activation: int = 0,
-                 pair_bias: Optional[torch.Tensor] = None, unary: Optional[int] = None):
+                 pair_bias: Optional[torch.Tensor] = None, unary: Optional[int] = None,
+                 limit: float = 0.0):
         """``swiglu``: the weight is [2 * out, in] with rows that alternate gate and up (row 2i
         the gate, row 2i + 1 the up projection of output i) and the product is followed by
         out = silu(gate) * up in the kernel's epilogue. ``activation`` (``kernels.ACT_*``)
         other than SiLU, or ``pair_bias`` ([2 * out], alternating like the rows, added before
-        the activation): only the tensor-core kernel has that epilogue. ``unary``
+        the activation; ``limit``: of the clamped form): only the tensor-core kernel has that
+        epilogue. ``unary``
         (``kernels.ACT_*``): the stored product is act(a · Wᵀ), in the tensor-core kernel's
         epilogue or by a kernel after the exact product; such a product is never added into a
         residual or left as split sums."""
@@ -50,7 +52,7 @@ class Linear:
             from .linear_fast import FastLinear
             self.fast = FastLinear.maybe(self.weight, rt, swiglu)
             if self.fast is not None and swiglu and not self.plain_swiglu:
-                self.fast.gated = (activation, pair_bias)
+                self.fast.gated = (activation, pair_bias, limit)
             if self.fast is not None:
                 self.fast.unary = unary
 

@@ -16,7 +16,7 @@ class FastLinear:
     def __init__(self, weight: torch.Tensor, rt, swiglu: bool):
         self.weight, self.rt, self.swiglu = weight, rt, swiglu
         self.unary = None       # an activation of the stored product, in the epilogue
-        self.gated = None       # (activation, pair bias) of a gated epilogue that is not plain SwiGLU
+        self.gated = None       # (activation, pair bias, limit) of a gated epilogue that is not plain SwiGLU
 
     @classmethod
     def maybe(cls, weight: torch.Tensor, rt, swiglu: bool) -> Optional["FastLinear"]:
@@ -51,7 +51,7 @@ class FastLinear:
         if self.swiglu:
             if self.gated is not None:
                 K.gemm_tc_gated(a, self.weight, out, self.gated[0], self.gated[1], rt.error_word,
-                                rt.sms)
+                                rt.sms, limit=self.gated[2])
                 return True
             K.gemm_tc(a, self.weight, out, False, rt.workspace, rt.error_word, rt.sms, swiglu=True)
             return True

@@ -14,7 +14,10 @@ fixed order. Nothing is read back to the host, so a decode pass stays a CUDA gra
 
 Options that a design may name. ``weights = "softmax_of_all"``: s = softmax(z) over every
 router output; the choice goes by s + ``correction`` (a stored vector), the weights are the
-chosen s times ``route_scale``, not renormalized. ``identity`` = n: the last n router outputs
+chosen s times ``route_scale``, not renormalized. ``weights = "sigmoid"``: the same with
+s = sigmoid(z). ``groups`` with ``keep_groups`` (with either): the experts are that many equal
+groups of neighbours, a group's score is the sum of its two largest s + ``correction``, and only
+experts of the best ``keep_groups`` groups can be chosen. ``identity`` = n: the last n router outputs
 are identity experts without tensors, whose output is the input h times the weight.
 ``activation = "clamped_swish"`` with ``limit``: g = min(W_g h, limit),
 u = clamp(W_u h, −limit, limit), g · sigmoid(1.702 g) · (u + 1) (the shared expert has a
@@ -86,7 +89,7 @@ class RoutedExperts(Part):
         if not 0 < self.top <= min(self.experts + int(p.get("identity", 0)), 32):
             raise ConfigError(f"{self.top} of {self.experts} experts per token")
         modes = {"softmax_of_chosen": K.ROUTE_SOFTMAX_OF_CHOSEN,
-                 "softmax_of_all": K.ROUTE_SOFTMAX_OF_ALL}
+                 "softmax_of_all": K.ROUTE_SOFTMAX_OF_ALL, "sigmoid": K.ROUTE_SIGMOID}
         if p.get("weights", "softmax_of_chosen") not in modes:
             raise ConfigError(f"expert weights \"{p['weights']}\" are not known "
                               f"(known: {', '.join(sorted(modes))})")
@@ -97,11 +100,18 @@ class RoutedExperts(Part):
         self.limit = float(p.get("limit", 0.0))
         self.shared_limit = float(p.get("shared_limit", self.limit))
         self.shared_gate = bool(p.get("shared_gate", True))
-        if self.mode == K.ROUTE_SOFTMAX_OF_ALL and (self.routed > 256 or self.shared_gate
-                                                    and int(p.get("shared_size", 0))):
+        scored = self.mode != K.ROUTE_SOFTMAX_OF_CHOSEN
+        if scored and (self.routed > 256 or self.shared_gate and int(p.get("shared_size", 0))):
             raise ConfigError("scores over all router outputs: at most 256 outputs, and a "
                               "shared expert without a gate")
-        if self.identity and self.mode != K.ROUTE_SOFTMAX_OF_ALL:
+        self.groups = int(p.get("groups", 1))
+        self.keep_groups = int(p.get("keep_groups", self.groups))
+        if self.groups > 1 and (not scored or self.groups > 32 or self.routed % self.groups
+                                or not 1 <= self.keep_groups <= self.groups
+                                or self.top > self.keep_groups * (self.routed // self.groups)):
+            raise ConfigError(f"{self.top} of {self.routed} experts from {self.keep_groups} of "
+                              f"{self.groups} groups")
+        if self.identity and not scored:
             raise ConfigError("identity experts come with scores over all router outputs")
         if self.top > self.routed:
             raise ConfigError(f"{self.top} of {self.routed} experts per token")
@@ -183,7 +193,18 @@ class RoutedExperts(Part):
             self.shared_up = Linear(both, rt, swiglu=self.shared_fused)
             self.shared_down = Linear(weights[self.n_shared + l["down"]], rt)
 
-    def forward(self, h, x, step, store: bool = False):
+    def forward_parts(self, h, step):
+        """The output as the rows of a token's choices [top, T, hidden] float32, which the caller
+        adds up in order; None for a part that has more to add (a shared expert, identity
+        experts)."""
+        if self.shared_size or self.identity:
+            return None
+        y, _, _ = self._chosen(h, step)
+        return y.view(h.shape[0], self.top, self.hidden).transpose(0, 1)
+
+    def _chosen(self, h, step, sg=None):
+        """The chosen experts' rows y [T * top, hidden] (row t * top + k, weighted), their ids and
+        weights [T, top]; ``sg`` [T] receives the shared expert's gate."""
         T, dev = h.shape[0], h.device
         E, top = self.experts, self.top
         A = T * top
@@ -191,22 +212,28 @@ class RoutedExperts(Part):
         z = _sums(self.router(h, out_dtype=torch.float32, defer=True))
         ids = torch.empty((T, top), dtype=torch.int32, device=dev)
         w = torch.empty((T, top), dtype=torch.float32, device=dev)
-        sg = (torch.empty((T,), dtype=torch.float32, device=dev)
-              if self.shared_size and self.shared_gate else None)
         bm = tile_rows(self.rt, self.w_up, T, A, E, self.hidden, self.inter)
         max_tiles = (A + bm - 1) // bm + E
         plan = torch.empty((2 + E + A + 2 * max_tiles,), dtype=torch.int32, device=dev)
         R = self.routed
         if T <= 64:          # the router's choice and the lists in one kernel
             K.moe_route_plan(z, E, top, R, ids, w, sg, bm, max_tiles, plan, self.mode,
-                             self.correction, self.route_scale, R)
+                             self.correction, self.route_scale, R, self.groups, self.keep_groups)
         else:
-            K.moe_route(z, R, top, R, ids, w, sg, self.mode, self.correction, self.route_scale)
+            K.moe_route(z, R, top, R, ids, w, sg, self.mode, self.correction, self.route_scale,
+                        self.groups, self.keep_groups)
             K.moe_plan(ids, E, bm, max_tiles, plan)
         if self.probe is not None:
             self.probe(self, step, ids)
         y = expert_products(self.rt, h, self.w_up, self.w_down, plan, bm, max_tiles, top, self.act,
                             limit=self.limit, weight=w)
+        return y, ids, w
+
+    def forward(self, h, x, step, store: bool = False):
+        T, dev, E, top = h.shape[0], h.device, self.experts, self.top
+        sg = (torch.empty((T,), dtype=torch.float32, device=dev)
+              if self.shared_size and self.shared_gate else None)
+        y, ids, w = self._chosen(h, step, sg)
         shared = None
         if self.shared_size:
             if self.shared_fused:

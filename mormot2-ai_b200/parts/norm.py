@@ -7,7 +7,11 @@ Dynamic Tanh: y = tanh(alpha · x) · w + b with a learned scalar alpha: a norm 
 mean and no variance, value by value in float32.
 
 Layer norm: y = (x − mean) / sqrt(var + eps) · w with the variance as the mean of the squared
-deviations and no bias, in float32. Over a residual of several streams it norms their sum."""
+deviations, in float32; with ``bias`` + b, stored as ``<name>.b``. Over a residual of several
+streams it norms their sum (without a bias).
+
+RMSNorm and layer norm also stand on what a sublayer gives back (``terms()`` names their
+weights for the kernel that does both sides of such a step, ``csrc/norm_step.cu``)."""
 from __future__ import annotations
 
 from typing import Dict, List, Optional
@@ -58,6 +62,10 @@ class RmsNorm(Part):
         K.rmsnorm(x, self.weight, self.eps, out, rows, R,
                   pending.partial if pending is not None else None)
         return out
+
+    def terms(self):
+        """(weight, bias or None, kind, eps) as ``kernels.norm_step`` takes a norm."""
+        return self.weight, None, "rms", self.eps
 
     def add_normed(self, y: torch.Tensor, x: torch.Tensor, h: Optional[torch.Tensor] = None) -> None:
         """x += w · y / rms(y) for a sublayer's output y [T, size] float32 (or its split sums
@@ -110,24 +118,43 @@ class LayerNorm(Part):
         self.size = int(spec.params["size"])
         self.eps = float(spec.params["eps"])
         self.name = prefix + spec.params["name"]
+        self.has_bias = bool(spec.params.get("bias", False))
+        self.optional = bool(spec.params.get("optional", False))   # may be absent (and unused)
         self.weight: Optional[torch.Tensor] = None
+        self.bias: Optional[torch.Tensor] = None
 
     def libraries(self, rt) -> List[str]:
-        return ["streams"]
+        return ["streams", "norm_step"] if not self.has_bias else ["norm_step"]
 
     def tensors(self) -> List[TensorNeed]:
-        return [TensorNeed(self.name, (self.size,), "vector")]
+        out = [TensorNeed(self.name, (self.size,), "vector", optional=self.optional)]
+        if self.has_bias:
+            out.append(TensorNeed(self.name + ".b", (self.size,), "bias", optional=self.optional))
+        return out
 
     def bind(self, weights: Dict[str, torch.Tensor], rt) -> None:
-        self.weight = weights[self.name]
         self.rt = rt
+        if self.optional and self.name not in weights:
+            return
+        self.weight = weights[self.name]
+        if self.has_bias:
+            self.bias = weights[self.name + ".b"]
+            if self.bias.dtype != self.weight.dtype:
+                self.weight, self.bias = self.weight.float(), self.bias.float()
+
+    def terms(self):
+        """(weight, bias or None, kind, eps) as ``kernels.norm_step`` takes a norm."""
+        return self.weight, self.bias, "layer", self.eps
 
     def forward(self, x: torch.Tensor, rows: Optional[torch.Tensor] = None,
                 n_rows: Optional[int] = None) -> torch.Tensor:
         """x: the float32 residual [T, size], or [streams, T, size], whose sum is normed."""
         R = n_rows if n_rows is not None else (rows.numel() if rows is not None else x.shape[-2])
         out = torch.empty((R, self.size), dtype=self.rt.dtype, device=x.device)
-        K.stream_step(x, read=(None, self.weight, self.eps, out, rows, R))
+        if self.has_bias:
+            K.norm_step(x, h=out, in_norm=self.terms(), rows=rows, n_rows=R)
+        else:
+            K.stream_step(x, read=(None, self.weight, self.eps, out, rows, R))
         return out
 
 
