@@ -1,7 +1,7 @@
 """Measures decoding and prefill of the Qwen3-8B shape with random weights on one B200.
 
     python bench.py [--gpus 1] [--steps K] [--warmup W] [--impl ours|reference]
-    python bench.py --design busavik|fimudra|sezopel|laralix|lotirax [--sizes small,mid]   (another workload, see below)
+    python bench.py --design busavik|fimudra|sezopel|laralix|lotirax|tenusun [--sizes small,mid]   (another workload, see below)
 
 A step is one decode step of a batch of 8 sequences whose context reaches 4,096 at the end of
 the timed steps. ``value`` is decoded tokens a second with the steps running back to back on
@@ -29,7 +29,10 @@ keys and values, retention, normed sublayer outputs, an input from the token aft
 ``--design laralix`` for the Laralix design (windowed attention with a distance bias beside the
 gated delta rule, attention whose values are its keys beside gated linear attention, latent
 attention with neighbours turned), ``--design lotirax`` for the Lotirax design (windowed
-differential attention, sublayers side by side, experts that a table names, looped layers).
+differential attention, sublayers side by side, experts that a table names, looped layers),
+``--design tenusun`` for the Tenusun design (latent attention in a window beside attention with
+values blended across layers and a gate per value, norms on both sides of every sublayer, experts
+chosen by sigmoid scores among groups).
 """
 import argparse
 import json
@@ -522,6 +525,80 @@ def lotirax_shapes(name):
     return LotiraxConfig.from_dict(doc), twin
 
 
+def tenusun_shapes(name):
+    """A Tenusun configuration whose layers have the sizes of a real model's (latent attention in a
+    window of 1,024 positions with a clamped gated feed-forward and attention over everything with
+    routed experts, in turn) and the Qwen3 configuration of equal width, head count, KV heads, key
+    size, feed-forward size and windows: the closest model of this library."""
+    from mormot2_ai_b200 import Qwen3Config, TenusunConfig
+    sizes = {
+        # width, heads, kv heads, dim, vdim, rot, latent: dim, rot, vdim, q rank, kv rank; ff,
+        # experts, groups, keep, top, expert ff
+        "small": (1024, 8, 2, 128, 64, 64, 64, 32, 64, 384, 256, 2816, 16, 4, 2, 4, 704),
+        "mid": (4096, 32, 8, 128, 128, 64, 128, 64, 128, 1536, 512, 11008, 32, 8, 4, 4, 2752),
+    }[name]
+    w, h, kv, dim, vd, rot, ld, lr, lv, qr, kvr, ff, ne, gc, gk, top, eff = sizes
+    vocab, window = 32768, 1024
+    lat = {"type": "latent_attention",
+           "mixer": {"heads": h, "dim": ld, "rot_dim": lr, "vdim": lv, "q_rank": qr, "kv_rank": kvr,
+                     "scale": (ld + lr) ** -0.5, "mask": {"size": window},
+                     "rot": {"base": 1e6, "dims": lr}},
+           "mlp": {"kind": "dense", "ff": ff, "limit": 7.0}}
+    att = {"type": "attention",
+           "mixer": {"heads": h, "kv_heads": kv, "dim": dim, "vdim": vd, "scale": dim ** -0.5,
+                     "v_mix": True,
+                     "rot": {"base": 1e6, "dims": rot,
+                             "scaling": {"factor": 4.0, "original": 4096, "fast": 32.0, "slow": 1.0}}},
+           "mlp": {"kind": "moe", "expert": {"ff": eff},
+                   "router": {"experts": ne, "top": top, "groups": {"count": gc, "keep": gk}}}}
+    doc = {"architecture": "Tenusun", "vocab": vocab, "width": w, "norm": {"eps": 1e-6},
+           "embedding": {"scale": float(w) ** 0.5}, "layers": [lat, att, lat, att]}
+    twin = Qwen3Config(vocab_size=vocab, hidden_size=w, num_hidden_layers=4,
+                       num_attention_heads=h, num_key_value_heads=kv, head_dim=dim,
+                       intermediate_size=ff, max_position_embeddings=40960,
+                       rms_norm_eps=1e-6, rope_theta=1e6, tie_word_embeddings=True,
+                       layer_windows=(window, 0, window, 0))
+    return TenusunConfig.from_dict(doc), twin
+
+
+def tenusun_work(cfg, tokens, batch, held, experts_read=None):
+    """As ``busavik_work`` for the Tenusun family: attention counts both products over the pairs
+    that the windows leave (a decode step the rows inside them, once), latent attention what its
+    kernel does (every head scores rows of kv_rank + rot_dim values and sums rows of kv_rank)."""
+    out = {"prefill_flops": {"attention": 0.0, "products": 0.0},
+           "decode_bytes": {"attention": 0.0, "products": 0.0}}
+    w = cfg.width
+    for layer in cfg.layers:
+        m, mlp = layer["mixer"], layer.get("mlp")
+        h, dim, vd = m["heads"], m["dim"], m["vdim"]
+        size = (m.get("mask") or {}).get("size") or 0
+        pairs = windowed_pairs(tokens, size)
+        seen = min(held / batch, size) if size else held / batch
+        if layer["type"] == "latent_attention":
+            rd, kvr, qr = m["rot_dim"], m["kv_rank"], m["q_rank"]
+            run = (qr + kvr + rd) * w + h * (dim + rd) * qr + h * (dim + vd) * kvr + h * vd * w
+            out["prefill_flops"]["attention"] += 2 * h * (kvr + rd + kvr) * pairs
+            out["decode_bytes"]["attention"] += 2 * batch * seen * (kvr + rd)
+        else:
+            kv = m["kv_heads"]
+            run = (h * dim + kv * (dim + vd) + 2 * h * vd) * w
+            out["prefill_flops"]["attention"] += 2 * h * (dim + vd) * pairs
+            out["decode_bytes"]["attention"] += 2 * batch * seen * kv * (dim + vd)
+        read = run
+        if mlp and mlp["kind"] == "dense":
+            run += 3 * w * mlp["ff"]
+            read += 3 * w * mlp["ff"]
+        elif mlp:
+            one, e, top = 3 * w * mlp["expert"]["ff"], mlp["router"]["experts"], mlp["router"]["top"]
+            run += top * one + e * w
+            read += (min(e, batch * top) if experts_read is None else experts_read) * one + e * w
+        out["prefill_flops"]["products"] += 2 * tokens * run
+        out["decode_bytes"]["products"] += 2 * read
+    out["prefill_flops"]["products"] += 2 * cfg.vocab * w
+    out["decode_bytes"]["products"] += 2 * cfg.vocab * w
+    return out
+
+
 def lotirax_work(cfg, tokens, batch, held, experts_read=None):
     """As ``busavik_work`` for the Lotirax family: attention counts both products of both maps
     over the pairs that the windows leave (a decode step the keys and values inside them, once),
@@ -709,6 +786,8 @@ def busavik_work(cfg, tokens, batch, held, experts_read=None):
         return laralix_work(cfg, tokens, batch, held)
     if getattr(cfg, "ARCHITECTURE", "") == "Lotirax":
         return lotirax_work(cfg, tokens, batch, held, experts_read)
+    if getattr(cfg, "ARCHITECTURE", "") == "Tenusun":
+        return tenusun_work(cfg, tokens, batch, held, experts_read)
     pairs = tokens * (tokens + 1) / 2
     out = {"prefill_flops": {"attention": 0.0, "products": 0.0},
            "decode_bytes": {"attention": 0.0, "products": 0.0}}
@@ -764,7 +843,8 @@ def busavik_bench(a):
     points = {}
     for size in [v for v in a.sizes.split(",") if v]:
         shapes = {"fimudra": fimudra_shapes, "sezopel": sezopel_shapes,
-                  "laralix": laralix_shapes, "lotirax": lotirax_shapes}.get(a.design, busavik_shapes)
+                  "laralix": laralix_shapes, "lotirax": lotirax_shapes,
+                  "tenusun": tenusun_shapes}.get(a.design, busavik_shapes)
         for family, cfg in zip((a.design, "qwen3"), shapes(size)):
             eng = Engine.from_random(cfg, seed=5, std=0.02, max_tokens=batch * ctx + tokens,
                                      max_context=max(ctx, tokens), max_slots=batch,
@@ -794,8 +874,9 @@ def busavik_bench(a):
                         int(ids[ids < real].unique().numel()))
             dshares = {}
             for k in range(6):
-                # a table of experts is read by token ids: different ones in the batch
-                apart = 97 if a.design == "lotirax" else 0
+                # a table of experts is read by token ids, and equal tokens choose alike: different
+                # ones in the batch
+                apart = 97 if a.design in ("lotirax", "tenusun") else 0
                 _, sh, _ = eng.timed_step([Entry(s, [1 + k + apart * i])
                                            for i, s in enumerate(slots)])
                 if k >= 2:
@@ -847,8 +928,8 @@ def main():
     ap.add_argument("--only-prefill", type=int, nargs="?", const=PREFILL_TOKENS, default=0,
                     help="only a prefill of this many tokens (for profiles; prints a short line)")
     ap.add_argument("--design", default="", choices=["", "busavik", "fimudra", "sezopel", "laralix",
-                                                          "lotirax"],
-                    help="busavik, fimudra, sezopel, laralix, lotirax: instead of the default workload, prefill and decode "
+                                                          "lotirax", "tenusun"],
+                    help="busavik, fimudra, sezopel, laralix, lotirax, tenusun: instead of the default workload, prefill and decode "
                          "of that design at layer sizes of real models beside the Qwen3 model of "
                          "equal size (prints its own JSON line)")
     ap.add_argument("--sizes", default="small,mid", help="with --design: which layer sizes")

@@ -161,24 +161,62 @@ def clamped_dense(h, w, p, limit, rnd=exact):
 
 def choose(z, correction, top, count, keep) -> Tuple[List[int], List[float]]:
     """The experts of one token's router logits z [E] and their weights (ties: the lower)."""
+    chosen, weights, _ = choose_with_margin(z, correction, top, count, keep)
+    return chosen, weights
+
+
+def choose_with_margin(z, correction, top, count, keep):
+    """Also how close the call was: the least that a choice score (or a group's score) lies above
+    the first one left out."""
     s = sigmoid(z)
     score = s + correction
     size = len(z) // count
     totals = [sum(sorted(score[g * size:(g + 1) * size])[-2:]) for g in range(count)]
-    kept = sorted(range(count), key=lambda g: (-totals[g], g))[:keep]
-    open_to = [e for e in range(len(z)) if e // size in kept]
-    chosen = sorted(open_to, key=lambda e: (-score[e], e))[:top]
-    return chosen, [float(s[e]) for e in chosen]
+    groups = sorted(range(count), key=lambda g: (-totals[g], g))
+    kept = groups[:keep]
+    ranked = sorted((e for e in range(len(z)) if e // size in kept), key=lambda e: (-score[e], e))
+    chosen = ranked[:top]
+    margin = np.inf
+    if keep < count:
+        margin = min(margin, totals[groups[keep - 1]] - totals[groups[keep]])
+    if top < len(ranked):
+        margin = min(margin, score[ranked[top - 1]] - score[ranked[top]])
+    return chosen, [float(s[e]) for e in chosen], float(margin)
 
 
-def routed_experts(h, w, p, mlp, rnd=exact):
+class Routing:
+    """What a test wants to know of the routers' choices, or to settle about them.
+
+    ``margins[(layer, t)]``: how close the call was. ``forced[(layer, t)]``: the experts that
+    another implementation chose there; they replace the plain choice where the two differ and the
+    margin is below ``close`` (a computation in 16 bits may fall on either side of such a call);
+    where the margin is larger the difference is an error (unless ``strict`` is off)."""
+
+    def __init__(self, forced=None, close: float = 0.05, strict: bool = True):
+        self.forced, self.close, self.strict = forced or {}, close, strict
+        self.margins: Dict = {}
+
+    def settle(self, layer, t, chosen, weights, margin, z):
+        self.margins[(layer, t)] = margin
+        theirs = self.forced.get((layer, t))
+        if theirs is None or set(theirs) == set(chosen):
+            return chosen, weights
+        if self.strict and margin >= self.close:
+            raise AssertionError(f"layer {layer}, token {t}: experts {sorted(theirs)} were chosen, "
+                                 f"{sorted(chosen)} expected, at a margin of {margin:.3g}")
+        return list(theirs), [float(v) for v in sigmoid(z[list(theirs)])]
+
+
+def routed_experts(h, w, p, mlp, rnd=exact, routing: Optional[Routing] = None, layer: int = 0):
     r = mlp["router"]
     groups = r.get("groups") or {"count": 1, "keep": 1}
     z = h @ w[p + "router"].T
     out = np.zeros_like(h)
     for t in range(h.shape[0]):
-        chosen, weights = choose(z[t], w[p + "correction"], r["top"], groups["count"],
-                                 groups["keep"])
+        chosen, weights, margin = choose_with_margin(z[t], w[p + "correction"], r["top"],
+                                                     groups["count"], groups["keep"])
+        if routing is not None:
+            chosen, weights = routing.settle(layer, t, chosen, weights, margin, z[t])
         for e, s in zip(chosen, weights):
             q = f"{p}e{e}."
             a = rnd(silu(w[q + "gate"] @ h[t]) * (w[q + "up"] @ h[t]))
@@ -188,9 +226,9 @@ def routed_experts(h, w, p, mlp, rnd=exact):
 
 # ---------------------------------------------------------------------------- the model
 def forward(config, w: Dict[str, np.ndarray], tokens, rnd=exact,
-            states: Optional[list] = None) -> np.ndarray:
+            states: Optional[list] = None, routing: Optional[Routing] = None) -> np.ndarray:
     """Logits [T, vocab] of a whole sequence; ``states`` receives the residual after every
-    layer."""
+    layer; ``routing``: what a test knows or wants to know of the routers' choices."""
     eps = float(config["norm"]["eps"])
 
     def norm(x, name):
@@ -214,7 +252,7 @@ def forward(config, w: Dict[str, np.ndarray], tokens, rnd=exact,
             if mlp.get("kind", "dense") == "dense":
                 y = clamped_dense(h, w, l + "mlp.", float(mlp["limit"]), rnd)
             else:
-                y = routed_experts(h, w, l + "mlp.", mlp, rnd)
+                y = routed_experts(h, w, l + "mlp.", mlp, rnd, routing, i)
             x = x + norm(y, l + "norm2b")
         if states is not None:
             states.append(x.copy())

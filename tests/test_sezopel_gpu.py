@@ -353,7 +353,7 @@ def attention_of(hidden, heads, kv, dim, vdim, rot, softcap, scale, rt, shared=F
 
 
 ATTENTION_SIZES = [
-    (4, 2, 24, 40, {"base": 1e4, "dims": 16}, 7.0),     # the general kernel: value rows of 40
+    (4, 2, 24, 40, {"base": 1e4, "dims": 16}, 7.0),     # sizes that the kernel rounds up
     (3, 3, 10, 6, None, 0.0),                           # no rotation, no cap, no grouping
     (4, 1, 64, 64, {"base": 5e5, "dims": 64}, 3.0),     # tensor-core sizes
     (2, 1, 128, 128, {"base": 1e4, "dims": 64}, 12.0),
@@ -404,7 +404,7 @@ def test_attention_alone(dtype, heads, kv, dim, vdim, rot, softcap, monkeypatch)
     got2 = run_mixer(reader, hs, [(0, 131)], hidden, dtype, line=line, writes=False, store=True)
     for g, wnt in zip(got2, want2):
         check(g, wnt, dtype, "a reader of another mixer's keys and values")
-    fast = dtype == "bfloat16" and dim == vdim and dim in (64, 128)
+    fast = dtype == "bfloat16" and dim % 8 == 0 and vdim % 8 == 0 and max(dim, vdim) <= 128
     assert (len(general) == 0) == fast
 
 
@@ -415,7 +415,7 @@ def test_attention_finds_one_far_key_under_the_cap(dtype, past, dim, vdim, monke
     """One key far back is made loud for the last query (the first key, one at a page border,
     one in the middle): its raw score is far above the cap, so its weight is e^cap against
     e^(small) of the others, no more; the head's output is multiplied by the gate's sigmoid.
-    Heads of 64 and 128 values go to the tensor-core kernels in bfloat16."""
+    In bfloat16 these sizes go to the tensor-core kernels."""
     heads, kv, cap, scale = 2, 1, 6.0, 0.5
     rt = Runtime(TORCH[dtype])
     T = TORCH[dtype]
@@ -450,7 +450,7 @@ def test_attention_finds_one_far_key_under_the_cap(dtype, past, dim, vdim, monke
         # the cap counts: without it the loud key alone would be the output
         s0 = plain.soft_cap((k @ q[0]) * scale, cap)
         assert abs(s0[loud] - cap) < 1e-3 and np.exp(s0 - s0.max())[loud] / np.exp(s0 - s0.max()).sum() < 0.999
-    assert (len(general) == 0) == (dtype == "bfloat16" and dim == vdim)
+    assert (len(general) == 0) == (dtype == "bfloat16")
 
 
 # ---------------------------------------------------------------------------- the engine
