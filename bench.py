@@ -563,8 +563,9 @@ def tenusun_shapes(name):
 
 def tenusun_work(cfg, tokens, batch, held, experts_read=None):
     """As ``busavik_work`` for the Tenusun family: attention counts both products over the pairs
-    that the windows leave (a decode step the rows inside them, once), latent attention what its
-    kernel does (every head scores rows of kv_rank + rot_dim values and sums rows of kv_rank)."""
+    that the windows leave (a decode step the rows inside them, once), latent attention
+    what its kernels do (a prompt scores keys of dim + rot_dim values and sums rows of vdim, which
+    a product forms; a decode step reads the rows of the cache)."""
     out = {"prefill_flops": {"attention": 0.0, "products": 0.0},
            "decode_bytes": {"attention": 0.0, "products": 0.0}}
     w = cfg.width
@@ -577,7 +578,7 @@ def tenusun_work(cfg, tokens, batch, held, experts_read=None):
         if layer["type"] == "latent_attention":
             rd, kvr, qr = m["rot_dim"], m["kv_rank"], m["q_rank"]
             run = (qr + kvr + rd) * w + h * (dim + rd) * qr + h * (dim + vd) * kvr + h * vd * w
-            out["prefill_flops"]["attention"] += 2 * h * (kvr + rd + kvr) * pairs
+            out["prefill_flops"]["attention"] += 2 * h * (dim + rd + vd) * pairs
             out["decode_bytes"]["attention"] += 2 * batch * seen * (kvr + rd)
         else:
             kv = m["kv_heads"]

@@ -52,8 +52,8 @@ __device__ __forceinline__ void gate8(const bf16* g, float* v) {
 #pragma unroll
   for (int i = 0; i < 4; ++i) {
     const float2 f = __bfloat1622float2(*(const __nv_bfloat162*)&w[i]);
-    v[2 * i] *= sigmoid_f32(f.x);
-    v[2 * i + 1] *= sigmoid_f32(f.y);
+    v[2 * i] *= sigmoid_fast(f.x);
+    v[2 * i + 1] *= sigmoid_fast(f.y);
   }
 }
 

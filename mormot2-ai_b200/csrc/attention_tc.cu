@@ -320,8 +320,8 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ,
 #pragma unroll
         for (int i = 0; i < 8; ++i) {
           const float2 gv = __bfloat1622float2(*(const __nv_bfloat162*)&gw[i]);
-          o[2 * i] *= sigmoid_f32(gv.x);
-          o[2 * i + 1] *= sigmoid_f32(gv.y);
+          o[2 * i] *= sigmoid_fast(gv.x);
+          o[2 * i + 1] *= sigmoid_fast(gv.y);
         }
       }
       uint32_t w[8];

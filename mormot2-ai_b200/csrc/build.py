@@ -51,6 +51,7 @@ SOURCES = {
     "moe": "moe.cu",
     "moe_tc": "moe_tc.cu",
     "latent_mma": "latent_mma.cu",
+    "latent_tc": "latent_tc.cu",
     "streams": "streams.cu",
     "norm_step": "norm_step.cu",
     "recurrent": "recurrent.cu",
@@ -67,7 +68,8 @@ EXTRA_HEADERS = {"gemm_tc": ["tc_common.cuh"],
                  "latent": ["mma_common.cuh", "mma_tile.cuh"],
                  "moe": ["mma_common.cuh", "moe_act.cuh"],
                  "moe_tc": ["tc_common.cuh", "moe_act.cuh"],
-                 "latent_mma": ["mma_common.cuh"]}
+                 "latent_mma": ["mma_common.cuh"],
+                 "latent_tc": ["attention_tc.cuh", "tc_common.cuh"]}
 
 _lock = threading.Lock()
 _loaded: Dict[str, ctypes.CDLL] = {}

@@ -200,6 +200,10 @@ __device__ __forceinline__ float tanh_of_2xlog2e(float x2) {
 // 1 / (1 + e^(-g))
 __device__ __forceinline__ float sigmoid_f32(float g) { return 1.0f / (1.0f + expf(-g)); }
 
+// the same by the fast exponential and division (a few units of the last float32 place): for a
+// factor of something that is rounded to bfloat16 next
+__device__ __forceinline__ float sigmoid_fast(float g) { return __fdividef(1.0f, 1.0f + __expf(-g)); }
+
 __device__ __forceinline__ float warp_sum(float v) {
 #pragma unroll
   for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);

@@ -28,6 +28,22 @@ __global__ void embed_kernel(const TW* __restrict__ table, const int* __restrict
   }
 }
 
+// The same, four values a thread (rows of a multiple of four values on 16-byte boundaries).
+template <typename TW>
+__global__ void __launch_bounds__(256)
+embed4_kernel(const TW* __restrict__ table, const int* __restrict__ ids, float* __restrict__ x,
+              int H, int V, float scale, int copies, size_t copy_stride) {
+  mb_grid_wait();
+  mb_grid_launch_next();
+  const int t = blockIdx.x, c = 4 * (blockIdx.y * blockDim.x + threadIdx.x);
+  if (c >= H) return;
+  int id = ids[t];
+  if (id < 0 || id >= V) id = 0;
+  float4 v = load4<TW>(table + (size_t)id * H + c);
+  v.x *= scale; v.y *= scale; v.z *= scale; v.w *= scale;
+  for (int k = 0; k < copies; ++k) *(float4*)(x + k * copy_stride + (size_t)t * H + c) = v;
+}
+
 // x[k][t, :] = table[ids[t], :] * scale for each of `copies` residual streams (copy k starts
 // copy_stride floats after copy k - 1).
 MB_EXPORT int mb_embed(const void* table, int table_dtype, const int* ids, float* x, int T,
@@ -36,6 +52,16 @@ MB_EXPORT int mb_embed(const void* table, int table_dtype, const int* ids, float
   if (T <= 0) return 0;
   cudaStream_t s = (cudaStream_t)stream;
   const int threads = H >= 1024 ? 256 : 128;
+  if (H % 4 == 0 && copy_stride % 4 == 0 && (((uintptr_t)table | (uintptr_t)x) & 15) == 0) {
+    const dim3 grid(T, (H / 4 + threads - 1) / threads);
+    if (table_dtype == MB_F32)
+      mb_launch(embed4_kernel<float>, grid, dim3(threads), 0, s, (const float*)table, ids, x, H, V,
+                scale, copies, (size_t)copy_stride);
+    else
+      mb_launch(embed4_kernel<__nv_bfloat16>, grid, dim3(threads), 0, s,
+                (const __nv_bfloat16*)table, ids, x, H, V, scale, copies, (size_t)copy_stride);
+    MB_CHECK_LAUNCH("mb_embed");
+  }
   if (table_dtype == MB_F32)
     mb_launch(embed_kernel<float>, dim3(T), dim3(threads), 0, s, (const float*)table, ids, x, H, V, scale,
               copies, (size_t)copy_stride);

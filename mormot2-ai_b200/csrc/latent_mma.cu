@@ -15,8 +15,9 @@
 // bfloat16, and then each adds P · V for its half of the kv_rank output columns (V = the same
 // tile, read with ldmatrix.trans), with the output rows in registers (kv_rank / 4 floats a
 // thread). A decode step of few sequences deals the key tiles of a sequence out over `splits`
-// blocks that leave (max, sum, unnormalised output) in float32 scratch; the block that
-// finishes last (a ticket counter, no waiting) adds them up.
+// blocks that leave (max, sum, unnormalised output) in float32 scratch; a second kernel adds them
+// up, a block a row (the splits of all rows together are megabytes: one block a tile of rows would
+// read them at one SM's rate).
 //
 // Sizes: dk and kv_rank multiples of 16, kv_rank at most 512; other sizes use the kernel of
 // latent.cu. There is no wait on another block or on a barrier object, so nothing can hang.
@@ -58,8 +59,7 @@ latent_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, int q_stride,
                             const int* __restrict__ page_table, int max_pages, int ring_pages,
                             const int* __restrict__ seq_start, const int* __restrict__ seq_past,
                             const int* __restrict__ seq_slot, int B, int nh, int kv_rank, int dk,
-                            int window, float scale, int splits, float* __restrict__ scratch,
-                            unsigned int* __restrict__ tickets) {
+                            int window, float scale, int splits, float* __restrict__ scratch) {
   mb_grid_wait();
   mb_grid_launch_next();
   extern __shared__ __align__(16) unsigned char smem_raw[];
@@ -276,7 +276,7 @@ latent_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, int q_stride,
         if (i < nv)
           *(uint32_t*)(dst + 8 * i + 2 * t) = pack_bf16(o[i][2 * r] * inv, o[i][2 * r + 1] * inv);
     } else {
-      float* dst = scratch + ((size_t)((first + tok) * nh + head) * splits + split) * (kv_rank + 2);
+      float* dst = scratch + ((size_t)((first + tok) * nh + head) * splits + split) * (kv_rank + 4);
       if (cs == 0 && t == 0) {
         dst[0] = m_run[r];
         dst[1] = l;
@@ -284,82 +284,64 @@ latent_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, int q_stride,
 #pragma unroll
       for (int i = 0; i < NV; ++i)
         if (i < nv) {
-          dst[2 + col0 + 8 * i + 2 * t] = o[i][2 * r];
-          dst[2 + col0 + 8 * i + 2 * t + 1] = o[i][2 * r + 1];
+          *(float2*)(dst + 4 + col0 + 8 * i + 2 * t) = make_float2(o[i][2 * r], o[i][2 * r + 1]);
         }
     }
   }
-  if (splits == 1) return;
-  // ---- the block that finishes last of a tile's splits adds them up: out[row] =
-  // sum_s exp(m_s - M) O_s / sum_s exp(m_s - M) l_s. The ticket counter wraps to 0 by itself,
-  // so the next launch finds it as this one did; nobody waits for anybody.
-  __shared__ unsigned int ticket;
-  __threadfence();
-  __syncthreads();
-  if (tid == 0) ticket = atomicInc(&tickets[blockIdx.x], (unsigned)splits - 1);
-  __syncthreads();
-  if (ticket != (unsigned)splits - 1) return;
-  __threadfence();
-  const int width = kv_rank + 2;
-  // every row's weights exp(m_s - M) / sum first (a thread a row), then all threads add the
-  // splits' outputs up, a pair of columns each, with the splits' loads in flight together
-  float* wts = (float*)ks;                                   // [64][16]
-  const int rows_here = min(LM_ROWS, n_new * nh - row0);
-  if (tid < rows_here) {
-    const int row = row0 + tid;
-    const float* src = scratch + ((size_t)first * nh + row) * splits * width;
-    float m[16], l[16], M = -INFINITY;
+}
+
+// out[row] = sum_s exp(m_s - M) O_s / sum_s exp(m_s - M) l_s over the splits, in order; row = token
+// * nh + head. Four columns a thread, the splits' loads in flight together.
+__global__ void __launch_bounds__(128)
+latent_merge_kernel(const float* __restrict__ scratch, int splits, int kv_rank, int nh,
+                    __nv_bfloat16* __restrict__ out, int out_stride) {
+  mb_grid_wait();
+  mb_grid_launch_next();
+  const int row = blockIdx.x, width = kv_rank + 4;
+  const float* src = scratch + (size_t)row * splits * width;
+  float m[16], M = -INFINITY, total = 0.f;
 #pragma unroll
-    for (int sp = 0; sp < 16; ++sp) {
-      m[sp] = sp < splits ? __ldcg(src + (size_t)sp * width) : -INFINITY;
-      l[sp] = sp < splits ? __ldcg(src + (size_t)sp * width + 1) : 0.f;
-      M = fmaxf(M, m[sp]);
-    }
-    float total = 0.f;
-#pragma unroll
-    for (int sp = 0; sp < 16; ++sp) {
-      m[sp] = m[sp] == -INFINITY ? 0.f : expf(m[sp] - M);
-      total = fmaf(m[sp], l[sp], total);
-    }
-    const float inv = 1.0f / total;
-#pragma unroll
-    for (int sp = 0; sp < 16; ++sp) wts[tid * 16 + sp] = m[sp] * inv;
+  for (int sp = 0; sp < 16; ++sp) {
+    m[sp] = sp < splits ? src[(size_t)sp * width] : -INFINITY;
+    M = fmaxf(M, m[sp]);
   }
-  __syncthreads();
-  const int pairs = kv_rank / 2;
-  for (int e = tid; e < rows_here * pairs; e += LM_THREADS) {
-    const int r = e / pairs, c = 2 * (e - r * pairs);
-    const int row = row0 + r;
-    const float* src = scratch + ((size_t)first * nh + row) * splits * width + 2 + c;
-    float2 part[16];
+#pragma unroll
+  for (int sp = 0; sp < 16; ++sp) {
+    m[sp] = m[sp] == -INFINITY ? 0.f : expf(m[sp] - M);
+    if (sp < splits) total = fmaf(m[sp], src[(size_t)sp * width + 1], total);
+  }
+  const float inv = 1.0f / total;
+  const int tok = row / nh, head = row - tok * nh;
+  for (int c = 4 * threadIdx.x; c < kv_rank; c += 4 * blockDim.x) {
+    float4 part[16];
 #pragma unroll
     for (int sp = 0; sp < 16; ++sp)
-      part[sp] = sp < splits ? __ldcg((const float2*)(src + (size_t)sp * width))
-                             : make_float2(0.f, 0.f);
-    float v0 = 0.f, v1 = 0.f;
+      part[sp] = sp < splits ? *(const float4*)(src + (size_t)sp * width + 4 + c)
+                             : make_float4(0.f, 0.f, 0.f, 0.f);
+    float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
 #pragma unroll
     for (int sp = 0; sp < 16; ++sp) {
-      const float w = wts[r * 16 + sp];
-      v0 = fmaf(w, part[sp].x, v0);
-      v1 = fmaf(w, part[sp].y, v1);
+      v.x = fmaf(m[sp], part[sp].x, v.x);
+      v.y = fmaf(m[sp], part[sp].y, v.y);
+      v.z = fmaf(m[sp], part[sp].z, v.z);
+      v.w = fmaf(m[sp], part[sp].w, v.w);
     }
-    const int tok = row / nh, head = row - tok * nh;
-    *(uint32_t*)(out + (size_t)(first + tok) * out_stride + (size_t)head * kv_rank + c) =
-        pack_bf16(v0, v1);
+    uint32_t* dst = (uint32_t*)(out + (size_t)tok * out_stride + (size_t)head * kv_rank + c);
+    dst[0] = pack_bf16(v.x * inv, v.y * inv);
+    dst[1] = pack_bf16(v.z * inv, v.w * inv);
   }
 }
 
 // q [T, nh * dk] (row stride q_stride), out [T, nh * kv_rank]; `tiles` = the sum over the
 // step's sequences of ceil(new tokens * nh / 64), as the host counts it; `splits` > 1 needs
-// scratch of T * nh * splits * (kv_rank + 2) floats and `tickets`, `tiles` counters that are 0
-// (the kernel leaves them 0).
+// scratch of T * nh * splits * (kv_rank + 4) floats on a 16-byte boundary.
 MB_EXPORT int mb_latent_attention_mma(const void* q, int q_stride, void* out, int out_stride,
                                       const void* pool, const int* page_table, int max_pages,
                                       int ring_pages, const int* seq_start, const int* seq_past,
                                       const int* seq_slot, int B, int T, int tiles, int nh,
                                       int kv_rank, int rot_dim, int window, float scale,
                                       int splits, float* scratch, long long scratch_floats,
-                                      unsigned int* tickets, void* stream) {
+                                      void* stream) {
   if (T <= 0 || tiles <= 0) return 0;
   const int dk = kv_rank + rot_dim;
   if (dk % 16 || kv_rank % 16 || kv_rank > 512 || q_stride % 8 || out_stride % 2 ||
@@ -367,8 +349,8 @@ MB_EXPORT int mb_latent_attention_mma(const void* q, int q_stride, void* out, in
     MB_FAIL("mb_latent_attention_mma: sizes %d + %d or alignment not supported", kv_rank, rot_dim);
   if (splits < 1) splits = 1;
   if (splits > 16) MB_FAIL("mb_latent_attention_mma: at most 16 splits, not %d", splits);
-  if (splits > 1 && (scratch == nullptr || tickets == nullptr ||
-                     (long long)T * nh * splits * (kv_rank + 2) > scratch_floats))
+  if (splits > 1 && (scratch == nullptr ||
+                     (long long)T * nh * splits * (kv_rank + 4) > scratch_floats || ((uintptr_t)scratch & 15)))
     MB_FAIL("mb_latent_attention_mma: scratch for %d splits", splits);
   cudaStream_t s = (cudaStream_t)stream;
   const int pitch = dk + 8;
@@ -387,10 +369,12 @@ MB_EXPORT int mb_latent_attention_mma(const void* q, int q_stride, void* out, in
     mb_launch(latent_attention_mma_kernel<NV_>, grid, dim3(LM_THREADS), smem, s,              \
               (const __nv_bfloat16*)q, q_stride, (__nv_bfloat16*)out, out_stride,             \
               (const __nv_bfloat16*)pool, page_table, max_pages, ring_pages, seq_start,       \
-              seq_past, seq_slot, B, nh, kv_rank, dk, window, scale, splits, scratch,         \
-              tickets);                                                                       \
+              seq_past, seq_slot, B, nh, kv_rank, dk, window, scale, splits, scratch);        \
   }
   if (kv_rank <= 128) GO(8) else if (kv_rank <= 256) GO(16) else GO(32)
 #undef GO
+  if (splits > 1)
+    mb_launch(latent_merge_kernel, dim3(T * nh), dim3(128), 0, s, (const float*)scratch, splits,
+              kv_rank, nh, (__nv_bfloat16*)out, out_stride);
   MB_CHECK_LAUNCH("mb_latent_attention_mma");
 }

@@ -481,8 +481,11 @@ moe_gemm_kernel(const T* __restrict__ in, const TW* __restrict__ W, void* __rest
 // flight; the tokens' rows wait in shared memory. Within a step of 32 values of K a thread
 // holds values 8t .. 8t+7 of both operands: the products pair them up in another order than
 // the instruction's own, which is the same sum. K must be a multiple of 32.
+// GROUPS: how many groups of 16 features a warp of a product without a gate takes (two where there
+// are blocks enough: the tokens' rows and the look-ups ahead of the first weight then serve twice
+// as many weights).
 #define MR_WARPS 4
-template <int MODE>
+template <int MODE, int GROUPS>
 __global__ void __launch_bounds__(MR_WARPS * 32)
 moe_rows_mma_kernel(const __nv_bfloat16* __restrict__ in, const __nv_bfloat16* __restrict__ W,
                     void* __restrict__ out, const int* __restrict__ plan, int A, int E,
@@ -491,7 +494,7 @@ moe_rows_mma_kernel(const __nv_bfloat16* __restrict__ in, const __nv_bfloat16* _
   mb_grid_wait();
   mb_grid_launch_next();
   constexpr bool UP = MODE != MOE_DOWN;
-  constexpr int NB = MODE == MOE_GATED_UP ? 2 : 1;
+  constexpr int NB = MODE == MOE_GATED_UP ? 2 : GROUPS;
   const int tile = blockIdx.y;
   if (tile >= plan[0]) return;
   const int* offsets = plan + 1;
@@ -506,6 +509,18 @@ moe_rows_mma_kernel(const __nv_bfloat16* __restrict__ in, const __nv_bfloat16* _
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, t = lane & 3;
   if (tid < 8) src[tid] = tid < rows ? perm[r0 + tid] : -1;
   __syncthreads();
+  const int n0 = (blockIdx.x * MR_WARPS + warp) * (MODE == MOE_GATED_UP ? 16 : 16 * GROUPS);
+  const __nv_bfloat16* We = W + (size_t)e * (MODE == MOE_GATED_UP ? 2 : 1) * N * K;
+  // rows past N are read from row N - 1 and never stored
+  const __nv_bfloat16* wa[NB];
+  const __nv_bfloat16* wb[NB];
+#pragma unroll
+  for (int nb = 0; nb < NB; ++nb) {
+    const int row = n0 + (MODE == MOE_GATED_UP ? 0 : 16 * nb) + g;
+    const size_t up = MODE == MOE_GATED_UP ? (size_t)nb * N : 0;
+    wa[nb] = We + (up + min(row, N - 1)) * K + 8 * t;
+    wb[nb] = We + (up + min(row + 8, N - 1)) * K + 8 * t;
+  }
   for (int c = tid; c < 8 * (K / 8); c += MR_WARPS * 32) {
     const int r = c / (K / 8), kc = (c - r * (K / 8)) * 8;
     uint4 v = make_uint4(0u, 0u, 0u, 0u);
@@ -513,17 +528,7 @@ moe_rows_mma_kernel(const __nv_bfloat16* __restrict__ in, const __nv_bfloat16* _
     *(uint4*)(xs + r * pitch + kc) = v;
   }
   __syncthreads();
-  const int n0 = (blockIdx.x * MR_WARPS + warp) * 16;
   if (n0 >= N) return;
-  const __nv_bfloat16* We = W + (size_t)e * NB * N * K;
-  // rows past N are read from row N - 1 and never stored
-  const __nv_bfloat16* wa[NB];
-  const __nv_bfloat16* wb[NB];
-#pragma unroll
-  for (int nb = 0; nb < NB; ++nb) {
-    wa[nb] = We + ((size_t)nb * N + min(n0 + g, N - 1)) * K + 8 * t;
-    wb[nb] = We + ((size_t)nb * N + min(n0 + g + 8, N - 1)) * K + 8 * t;
-  }
   const __nv_bfloat16* xr = xs + g * pitch + 8 * t;
   float acc[NB][4];
 #pragma unroll
@@ -557,17 +562,19 @@ moe_rows_mma_kernel(const __nv_bfloat16* __restrict__ in, const __nv_bfloat16* _
   }
   // acc[.][0..1]: feature n0 + g, tokens 2t and 2t + 1; acc[.][2..3]: feature n0 + g + 8
 #pragma unroll
-  for (int el = 0; el < 4; ++el) {
-    const int gn = n0 + g + (el >= 2 ? 8 : 0), r = 2 * t + (el & 1);
-    if (gn >= N || r >= rows) continue;
-    if (UP) {
-      ((__nv_bfloat16*)out)[(size_t)(r0 + r) * N + gn] =
-          __float2bfloat16_rn(moe_act<MODE>(acc[0][el], acc[NB - 1][el], act, limit));
-    } else {
-      const int a_ = src[r];
-      ((float*)out)[(size_t)a_ * N + gn] = (weight ? weight[a_] : 1.0f) * acc[0][el];
+  for (int nb = 0; nb < (MODE == MOE_GATED_UP ? 1 : NB); ++nb)
+#pragma unroll
+    for (int el = 0; el < 4; ++el) {
+      const int gn = n0 + 16 * nb + g + (el >= 2 ? 8 : 0), r = 2 * t + (el & 1);
+      if (gn >= N || r >= rows) continue;
+      if (UP) {
+        ((__nv_bfloat16*)out)[(size_t)(r0 + r) * N + gn] = __float2bfloat16_rn(
+            moe_act<MODE>(acc[nb][el], acc[MODE == MOE_GATED_UP ? NB - 1 : nb][el], act, limit));
+      } else {
+        const int a_ = src[r];
+        ((float*)out)[(size_t)a_ * N + gn] = (weight ? weight[a_] : 1.0f) * acc[nb][el];
+      }
     }
-  }
 }
 
 MB_EXPORT int mb_moe_gemm(const void* in, int dtype, const void* W, int w_dtype, void* out,
@@ -586,22 +593,28 @@ MB_EXPORT int mb_moe_gemm(const void* in, int dtype, const void* W, int w_dtype,
       MB_FAIL("mb_moe_gemm: tiles of 8 rows are the decode kernel's (bfloat16, K %% 32 == 0)");
     const size_t smem = (size_t)8 * (K + 8) * 2;
     if (smem > 160 * 1024) MB_FAIL("mb_moe_gemm: rows of %d values", K);
-    dim3 g8((N + 16 * MR_WARPS - 1) / (16 * MR_WARPS), max_tiles);
-#define GO8(M_)                                                                               \
+    // two groups a warp while that still leaves two blocks an SM (as many experts as the step's
+    // assignments can name)
+    const int named = A < E ? A : E;
+    const bool two = up != MOE_GATED_UP &&
+                     (N + 32 * MR_WARPS - 1) / (32 * MR_WARPS) * named >= 2 * 148;
+    const int per_block = (two ? 32 : 16) * MR_WARPS;
+    dim3 g8((N + per_block - 1) / per_block, max_tiles);
+#define GO8(M_, G_)                                                                           \
   {                                                                                           \
     static bool configured = false;                                                           \
     if (!configured) {                                                                        \
-      cudaFuncSetAttribute(moe_rows_mma_kernel<M_>, cudaFuncAttributeMaxDynamicSharedMemorySize, \
-                           160 * 1024);                                                       \
+      cudaFuncSetAttribute(moe_rows_mma_kernel<M_, G_>,                                       \
+                           cudaFuncAttributeMaxDynamicSharedMemorySize, 160 * 1024);          \
       configured = true;                                                                      \
     }                                                                                         \
-    mb_launch(moe_rows_mma_kernel<M_>, g8, dim3(MR_WARPS * 32), smem, s,                     \
+    mb_launch(moe_rows_mma_kernel<M_, G_>, g8, dim3(MR_WARPS * 32), smem, s,                 \
               (const __nv_bfloat16*)in, (const __nv_bfloat16*)W, out, plan, A, E, max_tiles,  \
               top, N, K, act, weight, limit);                                                 \
   }
-    if (up == MOE_GATED_UP) GO8(MOE_GATED_UP)
-    else if (up == MOE_PLAIN_UP) GO8(MOE_PLAIN_UP)
-    else GO8(MOE_DOWN)
+    if (up == MOE_GATED_UP) GO8(MOE_GATED_UP, 1)
+    else if (up == MOE_PLAIN_UP) { if (two) GO8(MOE_PLAIN_UP, 2) else GO8(MOE_PLAIN_UP, 1) }
+    else { if (two) GO8(MOE_DOWN, 2) else GO8(MOE_DOWN, 1) }
 #undef GO8
     MB_CHECK_LAUNCH("mb_moe_gemm");
   }

@@ -71,7 +71,8 @@ CLASS_OF = {"mb_gemm_tc": "products", "mb_gemm_simt": "products",
             "mb_gated_act": "activation", "mb_scale": "activation", "mb_add_bias": "activation",
             "mb_gemm_tc_gated": "products", "mb_latent_prep": "rotary",
             "mb_heads_gemm": "products", "mb_latent_attention": "attention",
-            "mb_latent_attention_mma": "attention",
+            "mb_latent_attention_mma": "attention", "mb_latent_prefill_tc": "attention",
+            "mb_latent_gather": "rotary", "mb_latent_q_rope": "rotary",
             "mb_moe_route": "routing", "mb_moe_plan": "routing", "mb_moe_route_plan": "routing", "mb_moe_gemm": "products",
             "mb_moe_combine": "routing", "mb_moe_table_plan": "routing",
             "mb_moe_gather": "routing", "mb_moe_gemm_tc": "products",
@@ -875,26 +876,77 @@ def latent_attention(q: torch.Tensor, out: torch.Tensor, step, line, nh: int, kv
 
 def latent_attention_mma(q: torch.Tensor, out: torch.Tensor, step, line, nh: int, kv_rank: int,
                          rot_dim: int, window: int, scale: float, splits: int,
-                         scratch: Optional[torch.Tensor],
-                         tickets: Optional[torch.Tensor] = None) -> None:
+                         scratch: Optional[torch.Tensor]) -> None:
     """``latent_attention`` on the tensor cores (bfloat16; kv_rank and kv_rank + rot_dim
     multiples of 16, kv_rank at most 512). ``splits`` > 1: the key tiles of a sequence are
-    dealt out over that many blocks, whose partial results meet in ``scratch`` (float32);
-    ``tickets``: int32 zeros, one per 64 (token, head) rows of the step, left zero."""
+    dealt out over that many blocks, whose partial results meet in ``scratch`` (float32)."""
     T = out.shape[0]
     _contig(out, "out"), _contig(q, "q")
     assert q.dtype == out.dtype == line.k.dtype == torch.bfloat16
     tiles = sum(-(-n * nh // 64) for n in step.host_new)
-    if splits > 1:
-        assert tickets is not None and tickets.dtype == torch.int32 and tickets.numel() >= tiles
     _call("latent_mma", "mb_latent_attention_mma",
           [_vp, _i, _vp, _i, _vp, _vp, _i, _i, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _f, _i,
-           _vp, _ll, _vp, _vp],
+           _vp, _ll, _vp],
           _ptr(q), q.stride(0), _ptr(out), out.stride(0), _ptr(line.k), _ptr(line.page_table),
           line.max_pages, line.ring_pages, _ptr(step.seq_start), _ptr(step.seq_past),
           _ptr(step.seq_slot), step.B, T, tiles, nh, kv_rank, rot_dim, window, float(scale),
-          splits, _ptr(scratch), scratch.numel() if scratch is not None else 0,
-          _ptr(tickets), _stream())
+          splits, _ptr(scratch), scratch.numel() if scratch is not None else 0, _stream(),
+          launches=2 if splits > 1 else 1)
+
+
+def latent_gather(line, step, kv_rank: int, rot_dim: int, window: int, rows: int):
+    """The cache rows that the step's tokens can see, sequence by sequence (of each the positions
+    from its first new token's window on): their latents [rows, kv_rank] and their rotated parts,
+    filled up with zeros, [rows, 64]. ``rows`` as ``latent_rows`` counts them."""
+    dev = line.k.device
+    c = torch.empty((rows, kv_rank), dtype=line.k.dtype, device=dev)
+    r = torch.empty((rows, 64), dtype=line.k.dtype, device=dev)
+    assert line.k.dtype == torch.bfloat16 and line.head_dim == kv_rank + rot_dim
+    _call("latent_tc", "mb_latent_gather",
+          [_vp, _vp, _i, _i, _vp, _vp, _vp, _i, _i, _i, _i, _i, _vp, _vp, _vp],
+          _ptr(line.k), _ptr(line.page_table), line.max_pages, line.ring_pages,
+          _ptr(step.seq_start), _ptr(step.seq_past), _ptr(step.seq_slot), step.B, rows, kv_rank,
+          rot_dim, window, _ptr(c), _ptr(r), _stream())
+    return c, r
+
+
+def latent_rows(step, window: int) -> int:
+    """How many cache rows ``latent_gather`` collects for a step."""
+    return sum(past + new - (max(0, past + 1 - window) if window > 0 else 0)
+               for past, new in zip(step.host_past, step.host_new))
+
+
+def latent_q_rope(q: torch.Tensor, nh: int, dim: int, rot_dim: int, rot_dims: int,
+                  inv_freq: Optional[torch.Tensor], amplitude: float, step) -> None:
+    """The rotated part of every head of q [T, nh * (dim + rot_dim)] turns in place."""
+    assert q.dtype == torch.bfloat16 and q.stride(1) == 1 and q.shape[1] == nh * (dim + rot_dim)
+    if rot_dims == 0:
+        return
+    assert inv_freq.dtype == torch.float32 and inv_freq.numel() >= rot_dims // 2
+    _call("latent_tc", "mb_latent_q_rope", [_vp, _i, _i, _i, _i, _i, _i, _vp, _f, _vp, _vp],
+          _ptr(q), q.stride(0), q.shape[0], nh, dim, rot_dim, rot_dims, _ptr(inv_freq),
+          float(amplitude), _ptr(step.tok_pos), _stream())
+
+
+def latent_prefill_tc(q: torch.Tensor, kv: torch.Tensor, rot: torch.Tensor, out: torch.Tensor,
+                      step, nh: int, dim: int, rot_dim: int, vd: int, window: int, scale: float,
+                      error: torch.Tensor, gate: Optional[torch.Tensor] = None) -> None:
+    """Latent attention of a long step with keys and values per head on tcgen05 (dim and vd 64 or
+    128, rot_dim at most 64): q with its rotated parts turned, ``kv`` [rows, nh * (dim + vd)] the
+    keys of all heads and then their values for the gathered rows, ``rot`` their rotated parts,
+    ``gate`` (or None) [T, >= nh * vd] logits whose sigmoid multiplies the output."""
+    T = out.shape[0]
+    assert q.dtype == kv.dtype == rot.dtype == out.dtype == torch.bfloat16
+    assert q.stride(1) == kv.stride(1) == out.stride(1) == 1 and rot.is_contiguous()
+    assert kv.shape == (rot.shape[0], nh * (dim + vd)) and kv.shape[0] == latent_rows(step, window)
+    assert gate is None or (gate.dtype == torch.bfloat16 and gate.stride(1) == 1)
+    _call("latent_tc", "mb_latent_prefill_tc",
+          [_vp, _i, _vp, _i, _vp, _i, _vp, _i, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _i, _f, _vp,
+           _vp, _i, _vp],
+          _ptr(q), q.stride(0), _ptr(kv), kv.stride(0), _ptr(rot), kv.shape[0], _ptr(out),
+          out.stride(0), _ptr(step.seq_start), _ptr(step.seq_past), step.B, T, step.max_new, nh,
+          dim, rot_dim, vd, window, float(scale), _ptr(error), _ptr(gate),
+          gate.stride(0) if gate is not None else 0, _stream())
 
 
 # ------------------------------------------------------------------------------ routed experts

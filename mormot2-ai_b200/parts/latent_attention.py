@@ -8,10 +8,13 @@ per head.
     k_h = [W_uk,h c ; r],   v_h = W_uv,h c,   score = (q_h · k_h) · scale, causal softmax
     out = W_o (concat_h(sum_j p_j v_h,j) * sigmoid(W_g h))          (the gate is optional)
 
-The kernels never form k_h or v_h: q_h,plain is carried into the latent space
+Two forms. The kernels of a decode step never form k_h or v_h: q_h,plain is carried into the latent space
 (W_uk,hᵀ q_h,plain, a small product per head), every head attends over the same cache rows
 [c ; r], and the weighted latent is carried out through W_uv,h (``csrc/latent.cu``). The
-projections that read h (W_dq, W_dkv, W_g) are one product.
+projections that read h (W_dq, W_dkv, W_g) are one product. A long step in bfloat16 whose sizes
+``csrc/latent_tc.cu`` takes forms them: the latents that its tokens can see are gathered from the
+cache, one product makes every head's keys and values of them, and attention runs over those
+(``expands`` says when). The cache is the same for both.
 """
 from __future__ import annotations
 
@@ -23,6 +26,11 @@ from .. import kernels as K
 from ..errors import ConfigError
 from .base import MIXERS, CacheNeed, Part, TensorNeed
 from .linear import Linear, Pending
+
+
+EXPAND_TOKENS = 128        # new tokens of a step from which on keys and values are formed
+EXPAND_ROWS = 8            # and at most that many rows to form them for, for every new token
+EXPAND_VALUES = 1 << 29    # ... and so many values in all (a gigabyte)
 
 
 class LatentAttention(Part):
@@ -49,7 +57,23 @@ class LatentAttention(Part):
     can_store = True      # forward(..., store=True) writes its output into x instead of adding
 
     def libraries(self, rt) -> List[str]:
-        return ["latent", "latent_mma"] if rt.fast_kernels else ["latent"]
+        if not rt.fast_kernels:
+            return ["latent"]
+        return ["latent", "latent_mma"] + (["latent_tc"] if self.sizes_expand() else [])
+
+    def sizes_expand(self) -> bool:
+        """Whether the sizes allow the form with keys and values per head."""
+        return (self.dim in (64, 128) and self.vd in (64, 128) and self.rd <= 64
+                and self.rd % 8 == 0 and self.kvr % 8 == 0 and self.qr % 8 == 0 and self.scale > 0)
+
+    def expands(self, step) -> bool:
+        """Whether this step forms keys and values per head: many new tokens, for which that is
+        less work, and not too many rows."""
+        if not self.can_expand or step.decode or step.T < EXPAND_TOKENS:
+            return False
+        rows = K.latent_rows(step, self.window)
+        return (rows <= EXPAND_ROWS * step.T
+                and rows * self.nh * (self.dim + self.vd) <= EXPAND_VALUES)
 
     def tensors(self) -> List[TensorNeed]:
         n = self.names
@@ -93,6 +117,11 @@ class LatentAttention(Part):
         self.uk_t = (weights[n["uk"]].view(self.nh, self.dim, self.kvr).transpose(1, 2)
                      .contiguous())
         self.uv = weights[n["uv"]].view(self.nh, self.vd, self.kvr).contiguous()
+        self.can_expand = (rt.fast_kernels and self.sizes_expand() and self.uk_t.dtype == torch.bfloat16
+                           and self.uv.dtype == torch.bfloat16)
+        if self.can_expand:     # one product for every head's keys, then every head's values
+            self.ukv = Linear(torch.cat([weights[n["uk"]], weights[n["uv"]]], dim=0), rt)
+            self.can_expand = self.ukv.fast is not None
         self.o = Linear(weights[n["o"]], rt)
         self.q_norm, self.kv_norm = weights[n["dq_norm"]], weights[n["dkv_norm"]]
         if self.q_norm.dtype != self.kv_norm.dtype:
@@ -123,13 +152,20 @@ class LatentAttention(Part):
             K.latent_prep(f, 0, self.kv_col, qr, kvr, rd, self.q_norm, self.kv_norm, self.eps,
                           inv_freq, rot_dims, amplitude, step, line, cq, writes_cache)
         q = self.uq(cq)                                                # [T, nh (dim + rd)]
-        ql = torch.empty((T, nh * (kvr + rd)), dtype=dt, device=dev)
-        K.heads_gemm(q, dim + rd, self.uk_t, ql, kvr + rd, tail=rd, rot_dims=rot_dims,
-                     inv_freq=inv_freq, amplitude=amplitude, tok_pos=step.tok_pos)
-        ol = torch.empty((T, nh * kvr), dtype=dt, device=dev)
-        self.rt.latent_attention(ql, ol, step, line, nh, kvr, rd, self.window, self.scale)
         heads = torch.empty((T, nh * vd), dtype=dt, device=dev)
-        K.heads_gemm(ol, kvr, self.uv, heads, vd, gate=gate)
+        if self.expands(step) and (gate is None or gate.stride(0) % 8 == 0 and gate.data_ptr() % 16 == 0):
+            c, rot = K.latent_gather(line, step, kvr, rd, self.window,
+                                     K.latent_rows(step, self.window))
+            K.latent_q_rope(q, nh, dim, rd, rot_dims, inv_freq, amplitude, step)
+            K.latent_prefill_tc(q, self.ukv(c), rot, heads, step, nh, dim, rd, vd, self.window,
+                                self.scale, self.rt.error_word, gate)
+        else:
+            ql = torch.empty((T, nh * (kvr + rd)), dtype=dt, device=dev)
+            K.heads_gemm(q, dim + rd, self.uk_t, ql, kvr + rd, tail=rd, rot_dims=rot_dims,
+                         inv_freq=inv_freq, amplitude=amplitude, tok_pos=step.tok_pos)
+            ol = torch.empty((T, nh * kvr), dtype=dt, device=dev)
+            self.rt.latent_attention(ql, ol, step, line, nh, kvr, rd, self.window, self.scale)
+            K.heads_gemm(ol, kvr, self.uv, heads, vd, gate=gate)
         if store:       # stored into x, or left pending (x is then not touched)
             out = self.o(heads, out=x, defer="any")
         else:

@@ -6,8 +6,8 @@ A: sizes that are no multiples of four; fewer rotating values than a head has; w
    groups of experts of which one or two are kept; experts after latent attention too.
 B: no embedding scale, no window, no blended values; a layer that rotates nothing; one head, as
    many key/value heads as heads; one expert a token without groups; a layer without feed-forward.
-C: sizes that the tcgen05 prefill takes (heads of 128, value rows of 64 and 128) and the
-   tensor-core form of latent attention; windows longer than a page.
+C: sizes that the tcgen05 prefills take (heads of 128, value rows of 64 and 128; latent attention
+   with keys and values per head, and one that stays with the latents); windows longer than a page.
 D: sizes that the warp-level kernels round up (heads of 40, 64 and 72, value rows of 24 and 136:
    the last one beyond them); twenty heads on one key/value head; a single latent layer last.
 """
@@ -80,7 +80,7 @@ def _c():
                 _lat(4, 48, 32, 40, 72, 64, 0.12, 70, 1e4, _dense(192, 1.2)),
                 _att(2, 1, 128, 128, 0.06, _rot(128, 1e5), False, _moe(8, 2, 96, (4, 3))),
                 _att(6, 2, 128, 64, 0.07, _rot(32, 1e4, 2.0, 100), True, _dense(160, 0.9)),
-                _lat(2, 64, 16, 96, 40, 128, 0.1, 129, 1e5, _moe(12, 3, 32, (6, 4)))]}
+                _lat(2, 64, 16, 128, 40, 128, 0.1, 129, 1e5, _moe(12, 3, 32, (6, 4)))]}
 
 
 def _d():

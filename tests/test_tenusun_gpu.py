@@ -75,7 +75,7 @@ def expected(model, eng, slot, ids, dtype, states=None, alone=None):
 # a logit over the spread of the plain logits, bounded in the median, the ninth decile and the
 # worst position of a comparison, and never tighter than three times what the plain
 # implementation itself moves by when it rounds what a 16-bit run rounds.
-F32_TOL = 1e-5
+F32_TOL = 2e-5
 BF16_TOL = {"median": 0.04, "decile": 0.08, "worst": 0.2}
 
 
@@ -470,7 +470,11 @@ def test_attention_as_a_mixer_and_values_blended_across_layers(dtype, layer, hid
 
 
 LATENTS = [(_lat(3, 18, 10, 14, 26, 30, 0.25, 21, 90.0), 72), (_lat(4, 48, 32, 40, 72, 64, 0.12, 65, 1e4), 96),
-           (_lat(1, 16, 16, 8, 24, 48, 0.2, 64, 50.0), 64), (_lat(6, 24, 0, 32, 16, 32, 0.2, 0, 50.0), 64)]
+           (_lat(1, 16, 16, 8, 24, 48, 0.2, 64, 50.0), 64), (_lat(6, 24, 0, 32, 16, 32, 0.2, 0, 50.0), 64),
+           # sizes for which long steps form keys and values per head
+           (_lat(3, 64, 32, 64, 72, 64, 0.12, 65, 1e4), 96), (_lat(2, 128, 64, 128, 40, 48, 0.08, 200, 1e3), 64),
+           (_lat(5, 64, 0, 128, 32, 80, 0.15, 0, 50.0), 64), (_lat(1, 128, 8, 64, 24, 40, 0.1, 1, 90.0), 64),
+           (_lat(2, 64, 48, 64, 40, 128, 0.1, 300, 1e3), 64)]
 
 
 def loud_pair(w, m, hidden, eps, rng):
@@ -489,7 +493,7 @@ def loud_pair(w, m, hidden, eps, rng):
 
 @pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("layer,hidden", LATENTS, ids=[str(i) for i in range(len(LATENTS))])
-def test_latent_attention_in_a_window(dtype, layer, hidden):
+def test_latent_attention_in_a_window(dtype, layer, hidden, monkeypatch):
     """One key that some queries like more than all others: queries at the last position that sees
     it and at the first that does not."""
     m, eps = layer["mixer"], 1e-4
@@ -498,24 +502,34 @@ def test_latent_attention_in_a_window(dtype, layer, hidden):
     w, wp = part_weights(mixer, seed=5, std=0.25)
     mixer.bind(to_dev(w, dtype), rt)
     rng = np.random.default_rng(9)
-    hs = [rng.normal(size=(n, hidden)) for n in (150, 3, 67)]
+    formed = mixer.sizes_expand()
+    N = 600 if formed else 150          # long enough for several tiles of rows
+    hs = [rng.normal(size=(n, hidden)) for n in (N, 3, 67)]
     size = (m.get("mask") or {}).get("size")
     key, query = loud_pair(wp, m, hidden, eps, rng)
     hs[0][10] = key
     for n in (10 + (size or 70) - 1, 10 + (size or 70)):
-        hs[0][n] = query
+        if n != 10:
+            hs[0][n] = query
     hs = [rounded(h, dtype) for h in hs]
     want = [plain.latent_attention(h, wp, "x.mix.", m, eps) for h in hs]
     moved = [plain.latent_attention(h, wp, "x.mix.", m, eps, rnd=plain.bfloat16) for h in hs]
     if size:        # a window one position off would show
-        for other, at in ((size - 1, 10 + size - 1), (size + 1, 10 + size)):
+        for other, at in [(size + 1, 10 + size)] + [(size - 1, 10 + size - 1)] * (size > 1):
             off = plain.latent_attention(hs[0], wp, "x.mix.", dict(m, mask={"size": other}), eps)
             assert np.abs(off[at] - want[0][at]).max() > 0.2 * want[0].std(), (other, at)
-    for cuts in CUTS:
-        line = line_of(4, 192, 1, m["kv_rank"] + m["rot_dim"], m["kv_rank"] + m["rot_dim"], TORCH[dtype], seed=3)
+    calls, kernel = [], K.latent_prefill_tc
+    monkeypatch.setattr(K, "latent_prefill_tc", lambda *a, **k: (calls.append(1), kernel(*a, **k))[1])
+    cuts_of = CUTS if not formed else [
+        [(0, N)], [(0, 2), (2, 4), (4, 64), (64, 66), (66, N)], [(0, 300), (300, 429), (429, N)],
+        [(0, 560)] + [(t, t + 1) for t in range(560, 568)]]
+    for cuts in cuts_of:
+        line = line_of(4, N + 42, 1, m["kv_rank"] + m["rot_dim"], m["kv_rank"] + m["rot_dim"], TORCH[dtype], seed=3)
         got = run_mixer(mixer, hs, cuts, hidden, dtype, line)
         for g, wnt, mv in zip(got, want, moved):
             check(g, wnt[:len(g)], dtype, f"cuts {cuts[:4]}", mv[:len(g)] if dtype == "bfloat16" else None)
+    # two calls (stored, and added) for each of the six long portions
+    assert len(calls) == (12 if formed and dtype == "bfloat16" else 0)
     rt.check()
 
 
