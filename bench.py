@@ -873,16 +873,17 @@ def busavik_bench(a):
                     real = layer.feed_forward.experts      # ids from there on: identity experts
                     layer.feed_forward.probe = lambda part, step, ids, real=real: chosen.append(
                         int(ids[ids < real].unique().numel()))
-            dshares = {}
-            for k in range(6):
+            each = []
+            for k in range(8):
                 # a table of experts is read by token ids, and equal tokens choose alike: different
                 # ones in the batch
                 apart = 97 if a.design in ("lotirax", "tenusun") else 0
                 _, sh, _ = eng.timed_step([Entry(s, [1 + k + apart * i])
                                            for i, s in enumerate(slots)])
-                if k >= 2:
-                    for name, ms in sh.items():
-                        dshares[name] = dshares.get(name, 0.0) + ms / 4
+                if k >= 3:
+                    each.append(sh)
+            # the median of five steps: a kernel's first use now and then costs a step much time
+            dshares = {name: sorted(sh[name] for sh in each)[len(each) // 2] for name in each[0]}
             eng.rt.check()
             experts_read = sum(chosen) / len(chosen) if chosen else None
             work = busavik_work(cfg, tokens, batch, batch * (ctx - steps / 2.0), experts_read)

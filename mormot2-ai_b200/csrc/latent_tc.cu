@@ -117,6 +117,19 @@ latent_q_rope_kernel(bf16* __restrict__ q, int ld, int nh, int dim, int rot_dim,
   __syncthreads();
   mb_grid_wait();
   mb_grid_launch_next();
+  if ((half & 1) == 0) {   // two neighbouring pairs at a time (dim and rot_dim are multiples of 8)
+    const int quarter = half >> 1;
+    for (int n = threadIdx.x; n < nh * quarter; n += blockDim.x) {
+      const int h = n / quarter, i = 2 * (n - h * quarter);
+      __nv_bfloat162* p = (__nv_bfloat162*)(q + (size_t)t * ld + (size_t)h * (dim + rot_dim) + dim + i);
+      const float2 u = __bfloat1622float2(p[0]), v = __bfloat1622float2(p[quarter]);
+      const float c0 = lq_angles[i], s0 = lq_angles[half + i];
+      const float c1 = lq_angles[i + 1], s1 = lq_angles[half + i + 1];
+      p[0] = __floats2bfloat162_rn(u.x * c0 - v.x * s0, u.y * c1 - v.y * s1);
+      p[quarter] = __floats2bfloat162_rn(v.x * c0 + u.x * s0, v.y * c1 + u.y * s1);
+    }
+    return;
+  }
   for (int n = threadIdx.x; n < nh * half; n += blockDim.x) {
     const int h = n / half, i = n - h * half;
     bf16* p = q + (size_t)t * ld + (size_t)h * (dim + rot_dim) + dim + i;
@@ -131,7 +144,8 @@ MB_EXPORT int mb_latent_q_rope(void* q, int ld, int T, int nh, int dim, int rot_
                                const float* inv_freq, float amp, const int* tok_pos,
                                void* stream) {
   if (T <= 0 || rot_dims <= 0) return 0;
-  if (rot_dims > rot_dim || (rot_dims & 1) || inv_freq == nullptr)
+  if (rot_dims > rot_dim || (rot_dims & 1) || inv_freq == nullptr || dim % 8 || rot_dim % 8 ||
+      ld % 8 || ((uintptr_t)q & 15))
     MB_FAIL("mb_latent_q_rope: %d of %d values rotate", rot_dims, rot_dim);
   mb_launch(latent_q_rope_kernel, dim3(T), dim3(256), (size_t)rot_dims * sizeof(float),
             (cudaStream_t)stream, (bf16*)q, ld, nh, dim, rot_dim, rot_dims, inv_freq, amp, tok_pos);

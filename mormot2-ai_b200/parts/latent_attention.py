@@ -138,9 +138,10 @@ class LatentAttention(Part):
         amplitude = float(getattr(self.position, "amplitude", 1.0))
         if rot_dims > rd:
             raise ConfigError(f"{rot_dims} rotating values of a part of {rd}")
-        # [T, qr + kvr + rd (+ nh vd)], or (few tokens) the product's split sums, which the kernel
-        # that norms the latents adds up as it reads them
-        f = self.down(h, defer=True)
+        # [T, qr + kvr + rd (+ nh vd)], or the product's split sums, which the kernel that norms
+        # the latents adds up as it reads them (the gate's columns of a long step are wider than
+        # all that it reads: their sums are then added up by the product)
+        f = self.down(h, defer=True if self.gated else "any")
         cq = torch.empty((T, qr), dtype=dt, device=dev)
         if isinstance(f, Pending):
             gate = torch.empty((T, nh * vd), dtype=dt, device=dev) if self.gated else None
