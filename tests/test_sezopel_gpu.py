@@ -366,8 +366,8 @@ ATTENTION_SIZES = [
 def test_attention_alone(dtype, heads, kv, dim, vdim, rot, softcap, monkeypatch):
     """Prompts over a page border in portions and decoded tokens, with a batch mate; then a
     second mixer without keys and values of its own reads what the first one kept. In
-    bfloat16, heads of 64 and 128 values with value rows of the same size run on the
-    tensor-core kernels, cap and gates included; everything else on the general kernel."""
+    bfloat16, heads and value rows that are multiples of 8 up to 128 run on the tensor-core
+    kernels, cap and gates included; everything else on the general kernel."""
     hidden, scale = 72, 2.5
     rt = Runtime(TORCH[dtype])
     general = []
